@@ -2,8 +2,9 @@
  * qie_oracle.c -- CPU restatement (plain C99) of the Rafae1130/qwen_inference_engine
  * decode/prefill forward.  TEST INFRASTRUCTURE ONLY -- see qie_oracle.h.
  *
- * Build: gcc -O2 -ffp-contract=off (no implicit FMA; every FMA the reference's SASS
- * contains is written as fmaf() here, each one noted where it occurs).
+ * Build: gcc -O2 -ffp-contract=off (no implicit FMA; every FMA that nvcc's default
+ * contraction makes of the reference's source expressions is written as fmaf() here, each one noted where it occurs;
+ * tools/ubench/fma_contract.cu finds the placement from outputs).
  *
  * What cannot be restated bit-for-bit on a CPU: the reference GEMM accumulates through
  * legacy tensor-core HMMA.16816.F32.BF16 (wmma, src/matrix_mul.cu:199-256) whose
@@ -167,7 +168,7 @@ void orc_qknorm_eps(orc_bf16* qk, const orc_bf16* w, int head_dim, int n_tok, in
 }
 
 /* ------------------------------------------------------------------ RoPE
- * src/RoPE.cu:6-22.  Interleaved pairs.  SASS (nvcc 12.9, sm_100a, default -fmad):
+ * src/RoPE.cu:6-22.  Interleaved pairs.  With default -fmad (nvcc 12.9, sm_100a; tools/ubench/fma_contract.cu):
  *   v1 = fma(x0, c, -(x1*s));   v2 = fma(c, x1, x0*s). */
 void orc_rope(const float* cos_values, const float* sin_values, orc_bf16* x, int n_tok, int head_dim,
               int row_dim, int n_heads) {

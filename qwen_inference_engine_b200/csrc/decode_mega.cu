@@ -1604,7 +1604,7 @@ __device__ __forceinline__ void attention_phase(const MegaArgs& a, int layer, un
 //  * scores: thread = cached position, the query group's heads in turn (q as fp32 in shared memory);
 //  * softmax: one warp per head; the sum chain runs in lane 0 with its operands requested 16 positions ahead;
 //  * PV: warps 0..3 own heads w, w+4, w+8, w+12 with lane l on output dims 2l, 2l+1: one LDS.32 of a V row feeds
-//    the fma chains of all heads of the warp (packed FFMA2: two IEEE fp32 fmas per instruction), the four
+//    the fma chains of all heads of the warp (packed fma (fma.rn.f32x2): two IEEE fp32 fmas per instruction), the four
 //    probabilities of a head arrive with one broadcast LDS.128.  (r01: one warp per head re-read every V row
 //    7 times and the phase was bound by shared-memory wavefronts: 27 cycles per position, now ~8.)
 constexpr int AT = NTC;            // positions per K/V tile
@@ -1613,13 +1613,13 @@ __host__ __device__ inline int attn_score_pitch(int max_kv_len) { return ((max_k
 
 // PV of one V tile (tn cached positions, rows of 128 bytes, lane l = output dims 2l, 2l+1) for the NH heads of a warp:
 // o[h] = fma(p[h][k], v[k], o[h]) for k ascending -- the reference's chain (self_attension.cu:112-137), two IEEE fmas
-// per packed FFMA2.  Groups of 4 positions in two operand sets; a set is reloaded (for 8 positions ahead) right
+// per packed fma (fma.rn.f32x2).  Groups of 4 positions in two operand sets; a set is reloaded (for 8 positions ahead) right
 // after it has been consumed, so every load has the other set's chains to land.
 template <int NH>
 __device__ __forceinline__ void pv_tile(const unsigned char* __restrict__ vl, const float* __restrict__ sb, int hstride, int tn,
                                         float2 (&o)[2]) {
-  // bf16 pair -> two floats on the ALU pipe only (PRMT / LOP3): the shift form becomes IMAD.U32 every other time, which
-  // shares the FMA pipe with the FFMA2 chain (math-pipe throttle was 12 % of this loop's stall samples)
+  // bf16 pair -> two floats by byte permute and mask: timed faster than a shift and a mask beside the fma chain (ncu counted
+  // math-pipe throttle as 12 % of this loop's stall samples with the shift)
   auto cvt2 = [](uint32_t v) { return make_float2(__uint_as_float(__byte_perm(v, 0u, 0x1044)), __uint_as_float(v & 0xffff0000u)); };
   auto load4 = [&](uint32_t (&vv)[4], float4 (&pr)[NH], int kk) {
 #pragma unroll
@@ -1907,7 +1907,7 @@ __device__ __noinline__ void attention_group_phase(const MegaArgs& a, int layer,
 //  * softmax: one warp per head; exponentials of block j + 2 are computed by all lanes while every lane walks the
 //    reference's sequential sum over block j (broadcast LDS.128, no divergence), so the FADD chain (4 cycles per
 //    position) is the only cost.
-//  * PV: 4 warps own heads w and w + 4 (two FFMA2 chains per lane, one LDS.32 + one widening per V row for both); a
+//  * PV: 4 warps own heads w and w + 4 (two packed fma chains per lane, one LDS.32 + one widening per V row for both); a
 //    fifth warp keeps the V ring (7 slots of 64 positions) filled; mbarriers per slot, no CTA-wide barrier per tile.
 constexpr int AG = 64;              // cached positions per K slot (one slot per warp)
 constexpr int AG_BYTES = AG * 128;  // head_dim 64, bf16
@@ -2002,15 +2002,15 @@ __device__ __forceinline__ void dot_half2(float4 (&w)[4], const float4* __restri
   yb = x1;
 }
 
-__device__ __forceinline__ float2 bf2x_to_f2(uint32_t v) {  // ALU pipe only (PRMT / LOP3), see pv_tile
+__device__ __forceinline__ float2 bf2x_to_f2(uint32_t v) {  // byte permute and mask, see pv_tile
   return make_float2(__uint_as_float(__byte_perm(v, 0u, 0x1044)), __uint_as_float(v & 0xffff0000u));
 }
 
 // PV over one whole ring slot (AVG = 128 cached rows of V, swizzled: word `lane` of row r sits at (lane << 2) ^ ((r & 7) << 4)) for
 // the two heads of a warp: o[h] = fma(p[h][k], v[k], o[h]) for k ascending -- the reference's chain
-// (self_attension.cu:112-137), two IEEE fmas per packed FFMA2, lane l = output dims 2l, 2l + 1.  The body is PVU rows
+// (self_attension.cu:112-137), two IEEE fmas per packed fma (fma.rn.f32x2), lane l = output dims 2l, 2l + 1.  The body is PVU rows
 // unrolled (every address is one of 8 row registers + an immediate: a position costs one LDS.32, the widening and two
-// FFMA2, + a quarter of a broadcast LDS.128 per head); chunk c + 1 is loaded before the chains of chunk c.
+// packed fma, + a quarter of a broadcast LDS.128 per head); chunk c + 1 is loaded before the chains of chunk c.
 // ONE copy of the body serves every PV warp: a warp with a single head runs the second chain on a dummy probability
 // row (its scheduler has the slots to spare) -- the step executes ~120 KB of code per layer, right at the size of the
 // instruction cache, and every KB less shows up in ALL phases (cold code costs ~10 cycles per instruction).
@@ -2039,7 +2039,7 @@ __device__ __forceinline__ void pv_group(const unsigned char* __restrict__ slot,
       if (c + 1 < PVU / 8 || blk + 1 < AVG / PVU) load(c + 1);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        // low half through the FMA pipe (IMAD.SHL), high half through the ALU pipe (LOP3)
+        // low half by an integer product, high half by a mask: timed faster here than byte permute and mask
         const float2 vf = make_float2(__uint_as_float(v[c & 1][j] * 65536u), __uint_as_float(v[c & 1][j] & 0xffff0000u));
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {

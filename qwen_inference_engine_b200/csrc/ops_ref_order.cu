@@ -7,8 +7,9 @@
 //   RoPE           src/RoPE.cu:6-22            fma(x0,c,-(x1*s)) , fma(c,x1,x0*s)
 //   selfattention  src/self_attension.cu:10-149
 //   sampling       src/logit_decode.cu:149-274
-// This file is compiled with -fmad=false; every fused multiply-add the reference's SASS
-// contains is spelled __fmaf_rn here, everything else is an explicit _rn intrinsic.
+// This file is compiled with -fmad=false; every fused multiply-add that nvcc's default
+// contraction makes of the reference's source expressions is spelled __fmaf_rn here (tools/ubench/fma_contract.cu
+// finds the placement from outputs), everything else is an explicit _rn intrinsic.
 #include <curand_kernel.h>
 #include <math_constants.h>
 

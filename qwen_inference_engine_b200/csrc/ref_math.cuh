@@ -2,8 +2,9 @@
 // (citations relative to /root/reference/layers/).  Shared by the per-operator kernels
 // (ops_ref_order.cu, gemm_ref_order.cu) and the persistent decode kernel (decode_mega.cu).
 // Translation units including this header are compiled with -fmad=false: every fused
-// multiply-add the reference's SASS contains is spelled __fmaf_rn, everything else is an
-// explicit _rn intrinsic.
+// multiply-add that nvcc's default contraction makes of the reference's source expressions is
+// spelled __fmaf_rn (which product of a two-product sum it fuses: tools/ubench/fma_contract.cu
+// compares outputs), everything else is an explicit _rn intrinsic.
 #pragma once
 #include <math_constants.h>
 

@@ -1,5 +1,5 @@
 // microbenchmark: latency / throughput of the packed fp32x2 instructions the attention phase is built from
-// (FFMA2 chains of the PV product, FADD chain of the softmax sum, FMUL2/FFMA2/FADD2 trees of the scores).
+// (fma.f32x2 chains of the PV product, FADD chain of the softmax sum, mul.f32x2/fma.f32x2/add.f32x2 trees of the scores).
 // nvcc -gencode arch=compute_100a,code=sm_100a -O3 -o fp32x2_lat fp32x2_lat.cu && ./fp32x2_lat
 #include <cstdio>
 #include <cuda_runtime.h>
@@ -16,16 +16,16 @@ __global__ void k(float* out, long long* cyc, int n, float pin, uint32_t vin) {
   float s = 0.f;
   __syncthreads();
   const long long t0 = clock64();
-  if (V == 0) {  // one dependent FFMA2 chain
+  if (V == 0) {  // one dependent fma.f32x2 chain
 #pragma unroll 16
     for (int i = 0; i < n; ++i) o0 = __ffma2_rn(make_float2(p, p), v, o0);
-  } else if (V == 1) {  // two independent FFMA2 chains
+  } else if (V == 1) {  // two independent fma.f32x2 chains
 #pragma unroll 16
     for (int i = 0; i < n; ++i) {
       o0 = __ffma2_rn(make_float2(p, p), v, o0);
       o1 = __ffma2_rn(make_float2(p, p), v, o1);
     }
-  } else if (V == 2) {  // four independent FFMA2 chains
+  } else if (V == 2) {  // four independent fma.f32x2 chains
 #pragma unroll 16
     for (int i = 0; i < n; ++i) {
       o0 = __ffma2_rn(make_float2(p, p), v, o0);
@@ -42,7 +42,7 @@ __global__ void k(float* out, long long* cyc, int n, float pin, uint32_t vin) {
   } else if (V == 4) {  // dependent FADD chain
 #pragma unroll 16
     for (int i = 0; i < n; ++i) s = __fadd_rn(s, p);
-  } else if (V == 5) {  // one FFMA2 chain + widening of a bf16 pair per step (PRMT + LOP3)
+  } else if (V == 5) {  // one fma.f32x2 chain + widening of a bf16 pair per step (permute + mask)
 #pragma unroll 16
     for (int i = 0; i < n; ++i) {
       const float2 vv = cvt2(vw + i);
@@ -55,7 +55,7 @@ __global__ void k(float* out, long long* cyc, int n, float pin, uint32_t vin) {
       o0 = __ffma2_rn(make_float2(p, p), vv, o0);
       o1 = __ffma2_rn(make_float2(p, p), vv, o1);
     }
-  } else if (V == 7) {  // 8 independent FMUL2 + FFMA2 + FADD2 streams (throughput)
+  } else if (V == 7) {  // 8 independent mul.f32x2 + fma.f32x2 + add.f32x2 streams (throughput)
     float2 a[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) a[j] = make_float2(p + j, p - j);
@@ -109,15 +109,15 @@ void run(const char* name, int threads, double per) {
 
 int main() {
   for (int th : {32, 128, 256}) {
-    run<0>("FFMA2 one dependent chain", th, 1);
-    run<1>("FFMA2 two chains", th, 2);
-    run<2>("FFMA2 four chains", th, 4);
+    run<0>("fma.f32x2 one dependent chain", th, 1);
+    run<1>("fma.f32x2 two chains", th, 2);
+    run<2>("fma.f32x2 four chains", th, 4);
     run<3>("FFMA scalar pair chain (x,y)", th, 2);
     run<9>("FFMA scalar two pairs", th, 4);
     run<4>("FADD dependent chain", th, 1);
-    run<5>("FFMA2 chain + PRMT/LOP3 widening", th, 3);
-    run<6>("2 FFMA2 chains + PRMT/LOP3 widening", th, 4);
-    run<7>("8 streams FMUL2+FFMA2 (throughput)", th, 16);
+    run<5>("fma.f32x2 chain + permute/mask widening", th, 3);
+    run<6>("2 fma.f32x2 chains + permute/mask widening", th, 4);
+    run<7>("8 streams mul.f32x2+fma.f32x2 (throughput)", th, 16);
     run<8>("16 streams FMUL+FFMA scalar (throughput)", th, 32);
   }
   return 0;
