@@ -1,8 +1,9 @@
 // attn_gqa.cu -- grouped-query attention over paged key/value rows for the fp32-stream families (fosavik.h): the
-// store of new rows (optional per-head unit norm of queries and keys), and an attention whose mask, sink, number of
-// score maps and finishing step are arguments: causal or sliding window with kept first tokens, a unit sink in the
-// denominator, one or two softmax maps over shared values, and as the last step nothing, a sigmoid gate per head, or
-// the differential combination with a unit norm per head.  Softmax and accumulation are fp32; the cache rows are fp32
+// store of new rows (optional unit norm of queries and keys, per head or over the whole projection; mean rows of whole
+// blocks of tokens), and an attention whose mask, sink, number of score maps and finishing step are arguments: causal or
+// sliding window with kept first tokens or with the mean rows of the blocks before it, a unit sink in the denominator, one
+// or two softmax maps over shared values, and as the last step nothing, a sigmoid gate per head, the differential
+// combination with a unit norm per head, or a mix of the heads' softmax weights.  Softmax and accumulation are fp32; the cache rows are fp32
 // or bf16.  Keys are ALWAYS read from the cache (a row's own position is stored first), so a result does not depend
 // on how a prompt was cut or what else is in the batch.
 #include <stdlib.h>
@@ -11,6 +12,7 @@
 
 #include "fosavik.h"
 #include "launch.h"
+#include "pack.cuh"
 
 namespace qie {
 namespace {
@@ -24,6 +26,16 @@ __device__ __forceinline__ const char* kv_row_ptr(const KvRowCache& c, const int
   const size_t off = (size_t)page * c.page_elems + c.layer_off + (size_t)(pos % c.page_size) * (c.kw + c.vw);
   return static_cast<const char*>(c.pool) + off * c.elt_bytes;
 }
+
+// pooled row of block b (KvRowCache)
+__device__ __forceinline__ const char* kv_pool_ptr(const KvRowCache& c, const int* block_table, int max_pages, int slot, int b) {
+  const int pi = (b * c.block + c.block - 1) / c.page_size;
+  const int page = block_table[(size_t)slot * max_pages + pi];
+  const size_t off = (size_t)page * c.page_elems + c.pool_off + (size_t)(b - pi * c.page_size / c.block) * (c.kw + c.vw);
+  return static_cast<const char*>(c.pool) + off * c.elt_bytes;
+}
+// blocks that lie wholly before the window of position pos: (b + 1) * pool - 1 <= pos - window
+__host__ __device__ __forceinline__ int pooled_seen(int pos, int window, int pool) { return pool > 0 && pos >= window ? (pos - window + 1) / pool : 0; }
 
 __device__ __forceinline__ void store_elt(const KvRowCache& c, char* row, int i, float v) {
   if (c.elt_bytes == 4) reinterpret_cast<float*>(row)[i] = v;
@@ -107,34 +119,114 @@ __global__ void __launch_bounds__(128) kv_store_rows_kernel(const KvStoreArgs a)
   }
 }
 
-// CTA (row, kv head x head chunk, key split).  Shared memory: q [QV][dim] (scaled) | K tile [ATK][kd + 1] | V tile
-// [ATK][vd] | scores [QV][ATK] | corr [QV] | m [QV] | l [QV], QV = hpc * maps query vectors, kd = maps * dim.
-__global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnArgs a, int hpc, int chunks, int n_splits) {
+// the mean of a block's rows -> its pooled row, by the threads of one CTA
+__device__ __forceinline__ void pool_block(const KvRowCache& c, const int* block_table, int max_pages, int slot, int b) {
+  char* dst = const_cast<char*>(kv_pool_ptr(c, block_table, max_pages, slot, b));
+  const float inv = 1.0f / (float)c.block;
+  for (int i = threadIdx.x; i < c.kw + c.vw; i += blockDim.x) {
+    float s = 0.f;
+#pragma unroll 4
+    for (int t = 0; t < c.block; ++t) {
+      const char* row = kv_row_ptr(c, block_table, max_pages, slot, b * c.block + t);
+      s += c.elt_bytes == 4 ? reinterpret_cast<const float*>(row)[i] : bf2f(reinterpret_cast<const bf16*>(row)[i]);
+    }
+    store_elt(c, dst, i, s * inv);
+  }
+}
+// one CTA per row; only the rows at a block's end do something
+__global__ void __launch_bounds__(128) kv_pool_rows_kernel(const KvRowCache c, const int* __restrict__ pos, const int* __restrict__ slot,
+                                                           const int* __restrict__ block_table, int max_pages) {
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, p = pos[r];
+  if ((p + 1) % c.block == 0) pool_block(c, block_table, max_pages, slot[r], p / c.block);
+}
+
+// The store with the unit norm over the whole projection: one CTA per row, both reductions at once, then the rotation of
+// every head.  Neighbouring pairs move as 4- and 8-byte accesses when they can.
+__global__ void __launch_bounds__(256) kv_store_whole_kernel(const KvStoreArgs a) {
+  __shared__ float red[64];
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, p = a.pos[r], slot = a.slot[r], d = a.norm_dim, tid = threadIdx.x;
+  const int nq = a.q ? a.q_heads * d : 0, kw = a.c.kw, vw = a.c.vw;
+  const bool bf = a.k_bf != nullptr;
+  const bf16 *qb = a.q_bf + (size_t)r * a.ld_bf, *kb = a.k_bf + (size_t)r * a.ld_bf, *vb = a.v_bf + (size_t)r * a.ld_bf;
+  float* qf = a.q + (size_t)r * a.ldq;
+  const float *kf = a.k + (size_t)r * a.ldk, *vf = a.v + (size_t)r * a.ldv;
+  auto getq = [&](int i) { return (bf ? bf2f(qb[i]) : qf[i]) + (a.q_bias ? bf2f(a.q_bias[i]) : 0.f); };
+  auto getk = [&](int i) { return (bf ? bf2f(kb[i]) : kf[i]) + (a.k_bias ? bf2f(a.k_bias[i]) : 0.f); };
+  float sq = 0.f, sk = 0.f;
+  if (a.q_norm)
+    for (int i = tid; i < nq; i += blockDim.x) sq = fmaf(getq(i), getq(i), sq);
+  if (a.k_norm)
+    for (int i = tid; i < kw; i += blockDim.x) sk = fmaf(getk(i), getk(i), sk);
+  const float2 s2 = block_sum2_r(sq, sk, red);
+  const float rq = a.q_norm ? 1.0f / sqrtf(s2.x / (float)nq + a.eps) : 1.f, rk = a.k_norm ? 1.0f / sqrtf(s2.y / (float)kw + a.eps) : 1.f;
+  const int dims = a.rope.dims, half = dims / 2, rest = d - dims;
+  const int st1 = a.rope.half_layout ? 1 : 2, off2 = a.rope.half_layout ? half : 1;
+  const float *ct = a.rope.cos_t + (size_t)p * half, *sn = a.rope.sin_t + (size_t)p * half;
+  // every element is read and written by the same thread (with its pair), so put may overwrite get's source
+  auto emit = [&](int n, auto get, const bf16* w, float rstd, auto put) {
+    auto val = [&](int i) { return w ? get(i) * rstd * bf2f(w[i]) : get(i); };
+    for (int i = tid; i < n / d * half; i += blockDim.x) {
+      const int g = i / half, e = i - g * half, e0 = g * d + st1 * e, e1 = e0 + off2;
+      const float u = val(e0), v = val(e1), c = ct[e], s = sn[e];
+      put(e0, u * c - v * s);
+      put(e1, v * c + u * s);
+    }
+    if (rest > 0)
+      for (int i = tid; i < n / d * rest; i += blockDim.x) {
+        const int g = i / rest, e = g * d + dims + (i - g * rest);
+        put(e, val(e));
+      }
+  };
+  char* row = const_cast<char*>(kv_row_ptr(a.c, a.block_table, a.max_pages, slot, p));
+  emit(kw, getk, a.k_norm, rk, [&](int i, float x) { store_elt(a.c, row, i, x); });
+  if (nq) emit(nq, getq, a.q_norm, rq, [&](int i, float x) { qf[i] = x; });
+  if (bf && a.c.elt_bytes == 2 && !a.v_bias) {
+    for (int i = tid; i < vw; i += blockDim.x) reinterpret_cast<bf16*>(row)[kw + i] = vb[i];
+  } else {
+    for (int i = tid; i < vw; i += blockDim.x) store_elt(a.c, row, kw + i, (bf ? bf2f(vb[i]) : vf[i]) + (a.v_bias ? bf2f(a.v_bias[i]) : 0.f));
+  }
+  if (a.c.block > 0 && a.one_each && (p + 1) % a.c.block == 0) {
+    __syncthreads();  // this row's own elements come from the whole CTA
+    pool_block(a.c, a.block_table, a.max_pages, slot, p / a.c.block);
+  }
+}
+
+// CTA (row, kv head x head chunk x value chunk, key split).  Shared memory: q [QV][dim] (scaled) | K tile [ATK][kd + 1] | V tile
+// [ATK][nv] | scores [QV][ATK] | corr [QV] | m [QV] | l [QV], QV = hpc * maps query vectors, kd = maps * dim, nv <= vc the
+// value columns of this CTA: a head's own vdim, or (talk) a chunk of the values of all kv heads.
+__global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnArgs a, int hpc, int chunks, int n_splits, int vc, int nvc) {
   extern __shared__ float sm[];
   __shared__ const char* rowp[ATK];
   __shared__ int dist[ATK];  // pos - j of the tile's keys
   pdl_wait();
   pdl_trigger();
   const int r = blockIdx.x, split = blockIdx.z;
-  const int g = blockIdx.y / chunks, chunk = blockIdx.y % chunks;
+  const int vci = blockIdx.y % nvc, yc = blockIdx.y / nvc;
+  const int g = yc / chunks, chunk = yc % chunks;
   const int hpg = a.heads / a.kv_heads;
   const int h0 = g * hpg + chunk * hpc;                 // first head of this CTA
   const int nh = min(hpc, hpg - chunk * hpc);           // heads of this CTA
-  const int maps = a.maps, dim = a.dim, vd = a.vdim, kd = maps * dim;
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim, col0 = vci * vc;
+  const int maps = a.maps, dim = a.dim, vd = min(vc, vcols - col0), kd = maps * dim;
   const int QV = nh * maps;
   float* qs = sm;
   float* Kt = qs + hpc * maps * dim;
   float* Vt = Kt + ATK * (kd + 1);
-  float* sc = Vt + ATK * vd;
+  float* sc = Vt + ATK * vc;
   float* corr = sc + hpc * maps * ATK;
   float* mrun = corr + hpc * maps;
   float* lrun = mrun + hpc * maps;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pos = a.pos[r], slot = a.slot[r];
-  // visible keys as one virtual range: the kept first tokens below the window, then the window
+  // visible keys as one virtual range: the pooled blocks before the window, the kept first tokens below it, then the window
+  const int npool = a.c.block > 0 ? pooled_seen(pos, a.window, a.c.block) : 0;
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
   const int nfirst = a.window > 0 ? min(a.keep_first, lo) : 0;
-  const int nkeys = nfirst + (pos - lo + 1);
+  const int nkeys = npool + nfirst + (pos - lo + 1);
   int per = (nkeys + n_splits - 1) / n_splits;
   per = (per + ATK - 1) / ATK * ATK;
   const int i0 = split * per, i1 = min(nkeys, i0 + per);
@@ -147,16 +239,16 @@ __global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnAr
 #pragma unroll
   for (int i = 0; i < AMAXACC; ++i) acc[i] = 0.f;
   const int nacc = QV * vd;
-  const size_t koff = a.shared_keys ? 0 : (size_t)g * kd, voff = (size_t)a.c.kw + (size_t)g * vd;
+  const size_t koff = a.shared_keys ? 0 : (size_t)g * kd, voff = (size_t)a.c.kw + (a.talk ? (size_t)col0 : (size_t)g * vd);
   const bool vec8 = a.c.elt_bytes == 2 && (a.c.page_elems % 8 == 0) && (a.c.layer_off % 8 == 0) && ((a.c.kw + a.c.vw) % 8 == 0) && (kd % 8 == 0) &&
-                    (vd % 8 == 0) && (a.c.kw % 8 == 0);
+                    (vd % 8 == 0) && (a.c.kw % 8 == 0) && (!a.c.block || a.c.pool_off % 8 == 0);
   for (int t0 = i0; t0 < i1; t0 += ATK) {
     const int nk = min(ATK, i1 - t0);
     __syncthreads();  // the previous tile is consumed; q and m/l are written
     if (tid < nk) {
-      const int i = t0 + tid;
+      const int i = t0 + tid - npool;
       const int j = i < nfirst ? i : lo + (i - nfirst);
-      rowp[tid] = kv_row_ptr(a.c, a.block_table, a.max_pages, slot, j);
+      rowp[tid] = i < 0 ? kv_pool_ptr(a.c, a.block_table, a.max_pages, slot, t0 + tid) : kv_row_ptr(a.c, a.block_table, a.max_pages, slot, j);
       dist[tid] = pos - j;
     }
     __syncthreads();
@@ -248,14 +340,15 @@ __global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnAr
     if (idx < nacc) {
       const int qv = idx / vd, col = idx - qv * vd;
       const size_t rec = (((size_t)r * a.heads + h0) * maps + qv) * n_splits + split;
-      a.ws[rec * (vd + 2) + 2 + col] = acc[i];
+      a.ws[rec * (vcols + 2) + 2 + col0 + col] = acc[i];
     }
   }
-  for (int qv = tid; qv < QV; qv += ATHREADS) {
-    const size_t rec = (((size_t)r * a.heads + h0) * maps + qv) * n_splits + split;
-    a.ws[rec * (vd + 2)] = mrun[qv];
-    a.ws[rec * (vd + 2) + 1] = lrun[qv];
-  }
+  if (vci == 0)
+    for (int qv = tid; qv < QV; qv += ATHREADS) {
+      const size_t rec = (((size_t)r * a.heads + h0) * maps + qv) * n_splits + split;
+      a.ws[rec * (vcols + 2)] = mrun[qv];
+      a.ws[rec * (vcols + 2) + 1] = lrun[qv];
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -264,7 +357,9 @@ __global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnAr
 // CTA stages in shared memory once for all rows (the windows of neighbouring rows overlap almost completely).  Scores,
 // the online softmax and the accumulators stay in registers (the score accumulators are re-packed as the A operand of
 // the P V product); softmax, sink, gate and the differential finish are fp32.  Head sizes are padded with zeros to
-// DP / VP.  Two score maps run one after the other; the first map's result waits in the output rows.
+// DP / VP.  Two score maps run one after the other; the first map's result waits in the output rows.  With pooled rows the
+// blocks of 64 pooled rows that some row of the tile sees come before the key blocks.  With `talk` the CTA's value columns are
+// chunk blockIdx.z (vc columns) of the values of all kv heads, and its normalised result goes to the workspace record of (row, head).
 constexpr int PT_ROWS = 64, PT_KEYS = 64;
 
 __device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, uint32_t addr) {
@@ -273,7 +368,7 @@ __device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, ui
 
 template <int DP, int VP>
 __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs a, const int* __restrict__ seg_start,
-                                                              const int* __restrict__ seg_slot, int n_seg) {
+                                                              const int* __restrict__ seg_slot, int n_seg, int vc) {
   extern __shared__ __align__(16) unsigned char pt_smem[];  // two stages of a key block: K [2][64][DP + 8], V [2][64][VP + 8]
   typedef bf16 KTile[PT_KEYS][DP + 8];
   typedef bf16 VTile[PT_KEYS][VP + 8];
@@ -305,7 +400,9 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   __syncthreads();
   const int slot = tile_info[2];
   const int h = blockIdx.y, g = h / (a.heads / a.kv_heads);
-  const int dim = a.dim, vd = a.vdim, maps = a.maps, kd = maps * dim;
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim, col0 = a.talk ? (int)blockIdx.z * vc : 0;
+  const int dim = a.dim, vd = a.talk ? min(vc, vcols - col0) : a.vdim, maps = a.maps, kd = maps * dim;
+  const size_t voff = (size_t)a.c.kw + (a.talk ? (size_t)col0 : (size_t)g * vd);
   for (int which = 0; which < 2; ++which) {
   const int tile = tile_info[3 + which];
   if (tile < 0) break;
@@ -313,6 +410,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   const int pos0 = a.pos[row0];                       // rows of a segment are consecutive positions
   const int pmax = pos0 + nrows - 1;
   const int lo_min = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int nbmax = a.c.block > 0 ? pooled_seen(pmax, a.window, a.c.block) : 0, npb = (nbmax + PT_KEYS - 1) / PT_KEYS;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
   // soft cap of a scaled score: cap * tanh(s / cap) as cap * (1 - 2 / (exp(2 s / cap) + 1)); the weights become bf16 operands
   // below, far coarser than the fast exponential
@@ -324,7 +422,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   const int i0 = pos0 + wrow + qr, i1 = i0 + 8;       // positions of the thread's two rows
   // 16-byte staging when every cache row piece starts on a 16-byte boundary
   const bool vec = (a.c.page_elems % 8 == 0) && (a.c.layer_off % 8 == 0) && ((a.c.kw + a.c.vw) % 8 == 0) && (dim % 8 == 0) && (vd % 8 == 0) &&
-                   (a.c.kw % 8 == 0);
+                   (a.c.kw % 8 == 0) && (!a.c.block || a.c.pool_off % 8 == 0);
   for (int mp = 0; mp < maps; ++mp) {
     uint32_t qf[DP / 16][4];
     {
@@ -352,14 +450,23 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     // key blocks that some row of the tile sees: the blocks of the kept first tokens, then from the window's lower edge on
     auto skipped = [&](int j) { return a.window > 0 && j + PT_KEYS - 1 < lo_min && j >= a.keep_first; };
+    // a block's number j is its first position, or for the npb blocks of pooled rows -PT_KEYS * npb, ..., -PT_KEYS
     auto next_block = [&](int j) {
       j += PT_KEYS;
-      return skipped(j) ? lo_min / PT_KEYS * PT_KEYS : j;
+      return j >= 0 && skipped(j) ? lo_min / PT_KEYS * PT_KEYS : j;
     };
     // a key block -> stage `buf` (cp.async when every piece of a cache row starts on a 16-byte boundary); one commit group
     auto stage = [&](int jb, int buf) {
-      if (tid < PT_KEYS)  // one page lookup per key, not per 16-byte piece
-        krow[buf][tid] = jb + tid <= pmax ? reinterpret_cast<const bf16*>(kv_row_ptr(a.c, a.block_table, a.max_pages, slot, jb + tid)) : nullptr;
+      if (tid < PT_KEYS) {  // one page lookup per key, not per 16-byte piece
+        const char* kp = nullptr;
+        if (jb < 0) {
+          const int b = jb + npb * PT_KEYS + tid;
+          if (b < nbmax) kp = kv_pool_ptr(a.c, a.block_table, a.max_pages, slot, b);
+        } else if (jb + tid <= pmax) {
+          kp = kv_row_ptr(a.c, a.block_table, a.max_pages, slot, jb + tid);
+        }
+        krow[buf][tid] = reinterpret_cast<const bf16*>(kp);
+      }
       __syncthreads();
       for (int i = tid; i < PT_KEYS * (DP / 8); i += 128) {
         const int key = i / (DP / 8), c = (i % (DP / 8)) * 8;
@@ -379,7 +486,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
         bf16* dst = &Vs[buf][key][c];
         const bf16* row = krow[buf][key];
         if (row && c < vd) {
-          const bf16* src = row + a.c.kw + (size_t)g * vd + c;
+          const bf16* src = row + voff + c;
           if (vec) cp_async16(smem_u32(dst), src);
           else
             for (int e = 0; e < 8; ++e) dst[e] = c + e < vd ? src[e] : f2bf(0.f);
@@ -389,7 +496,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
       }
       cp_async_commit();
     };
-    int j0 = skipped(0) ? lo_min / PT_KEYS * PT_KEYS : 0, buf = 0;
+    int j0 = npb ? -npb * PT_KEYS : (skipped(0) ? lo_min / PT_KEYS * PT_KEYS : 0), buf = 0;
     stage(j0, 0);
     while (true) {
       const int jn = next_block(j0);
@@ -416,8 +523,18 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
       // mask, running maximum
       float mx0 = -INFINITY, mx1 = -INFINITY;
       // a block that every row of the warp sees whole (below the diagonal, inside the window) needs no mask
-      const bool whole = j0 + PT_KEYS - 1 <= pos0 + wrow && (a.window <= 0 || pos0 + wrow + 15 - j0 < a.window);
-      if (whole) {
+      const bool whole = j0 >= 0 && j0 + PT_KEYS - 1 <= pos0 + wrow && (a.window <= 0 || pos0 + wrow + 15 - j0 < a.window);
+      if (j0 < 0) {  // pooled rows: a prefix of the blocks, longer for later rows
+        const int b0 = j0 + npb * PT_KEYS + qc, n0 = pooled_seen(i0, a.window, a.c.block), n1 = pooled_seen(i1, a.window, a.c.block);
+#pragma unroll
+        for (int nb = 0; nb < PT_KEYS / 8; ++nb)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[nb][e] = b0 + nb * 8 + (e & 1) < ((e >> 1) ? n1 : n0) ? capped(s[nb][e] * a.scale) : -INFINITY;
+            if (e >> 1) mx1 = fmaxf(mx1, s[nb][e]);
+            else mx0 = fmaxf(mx0, s[nb][e]);
+          }
+      } else if (whole) {
         const float d0 = -slope * (float)(i0 - j0 - qc), d1 = -slope * (float)(i1 - j0 - qc);  // minus slope times the distance to the thread's first column
 #pragma unroll
         for (int nb = 0; nb < PT_KEYS / 8; ++nb)
@@ -499,6 +616,26 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
       f0 = l0 > 0.f ? 1.0f / l0 : 0.f;
       f1 = l1 > 0.f ? 1.0f / l1 : 0.f;
     }
+    if (a.talk) {  // the heads are mixed by gqa_talk_finish_kernel
+      const size_t rs = (size_t)(vcols + 2);
+      float* w0 = a.ws + ((size_t)(row0 + wrow + qr) * a.heads + h) * rs;
+      float* w1 = w0 + (size_t)8 * a.heads * rs;
+      if (blockIdx.z == 0 && (lane & 3) == 0) {
+        if (rv0) w0[0] = 0.f, w0[1] = 1.f;
+        if (rv1) w1[0] = 0.f, w1[1] = 1.f;
+      }
+#pragma unroll
+      for (int vb = 0; vb < VP / 8; ++vb) {
+        const int c = vb * 8 + qc;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (c + e >= vd) continue;
+          if (rv0) w0[2 + col0 + c + e] = o[vb][e] * f0;
+          if (rv1) w1[2 + col0 + c + e] = o[vb][2 + e] * f1;
+        }
+      }
+      continue;
+    }
     float* out0 = a.out + (size_t)(row0 + wrow + qr) * a.ldo + (size_t)h * vd;
     float* out1 = out0 + (size_t)8 * a.ldo;
     const bool last = mp == maps - 1;
@@ -563,19 +700,23 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
 template <int DP, int VP>
 cudaError_t launch_prefill_mma_dv(const GqaAttnArgs& a, const int* seg_start, const int* seg_slot, int n_seg, cudaStream_t st) {
   const int per_cta = a.window <= 0 ? 2 * PT_ROWS : PT_ROWS;
-  const dim3 grid((a.n + per_cta - 1) / per_cta + n_seg, a.heads), block(128);  // upper bound of the tiles / tile pairs
+  // talk: the values of all kv heads in equal chunks of at most VP columns, each a multiple of 8
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim, nvc = (vcols + VP - 1) / VP, vc = ((vcols + nvc - 1) / nvc + 7) / 8 * 8;
+  const dim3 grid((a.n + per_cta - 1) / per_cta + n_seg, a.heads, nvc), block(128);  // upper bound of the tiles / tile pairs
   const size_t smem = (size_t)2 * PT_KEYS * ((DP + 8) + (VP + 8)) * sizeof(bf16);
   if (smem > 48 * 1024) {
     cudaError_t r = cudaFuncSetAttribute(gqa_prefill_mma_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (r != cudaSuccess) return r;
   }
-  return launch_k(gqa_prefill_mma_kernel<DP, VP>, grid, block, smem, st, a, seg_start, seg_slot, n_seg);
+  return launch_k(gqa_prefill_mma_kernel<DP, VP>, grid, block, smem, st, a, seg_start, seg_slot, n_seg, vc);
 }
 
 template <int DP>
 cudaError_t launch_prefill_mma_v(const GqaAttnArgs& a, const int* seg_start, const int* seg_slot, int n_seg, cudaStream_t st) {
-  if (a.vdim <= 32) return launch_prefill_mma_dv<DP, 32>(a, seg_start, seg_slot, n_seg, st);
-  if (a.vdim <= 64) return launch_prefill_mma_dv<DP, 64>(a, seg_start, seg_slot, n_seg, st);
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim;
+  if (vcols <= 32) return launch_prefill_mma_dv<DP, 32>(a, seg_start, seg_slot, n_seg, st);
+  if (vcols <= 64) return launch_prefill_mma_dv<DP, 64>(a, seg_start, seg_slot, n_seg, st);
+  if (vcols > 128) return launch_prefill_mma_dv<DP, 256>(a, seg_start, seg_slot, n_seg, st);  // talk only
   return launch_prefill_mma_dv<DP, 128>(a, seg_start, seg_slot, n_seg, st);
 }
 
@@ -637,6 +778,50 @@ __global__ void __launch_bounds__(128) gqa_finish_kernel(const GqaAttnArgs a, in
   for (int c = threadIdx.x; c < vd; c += blockDim.x) out[c] = o[c] * rstd;
 }
 
+// CTA (row, kv head): merges the key splits of every head's attended values of this kv head, then mixes the heads:
+// out[h] = sum_g talk[h, g] a_g for the heads h of the kv head.  Shared memory: weights [heads][n_splits] | a [heads][vd]
+__global__ void __launch_bounds__(128) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits) {
+  extern __shared__ float tf_smem[];
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, c = blockIdx.y, vd = a.vdim, H = a.heads, hpg = H / a.kv_heads;
+  const size_t rs = (size_t)a.kv_heads * vd + 2;
+  const float* rec = a.ws + (size_t)r * H * n_splits * rs;
+  float* wt = tf_smem;
+  float* at = wt + H * n_splits;
+  for (int g = threadIdx.x; g < H; g += blockDim.x) {
+    const float* rg = rec + (size_t)g * n_splits * rs;
+    float M = -INFINITY, L = 0.f;
+    for (int s = 0; s < n_splits; ++s) M = fmaxf(M, rg[s * rs]);
+    for (int s = 0; s < n_splits; ++s) {
+      const float ms = rg[s * rs], w = ms > -INFINITY ? expf(ms - M) : 0.f;
+      wt[g * n_splits + s] = w;
+      L = fmaf(rg[s * rs + 1], w, L);
+    }
+    for (int s = 0; s < n_splits; ++s) wt[g * n_splits + s] /= L;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < H * vd; i += blockDim.x) {
+    const int g = i / vd, col = i - g * vd;
+    const float* rg = rec + (size_t)g * n_splits * rs + 2 + c * vd + col;
+    float v = 0.f;
+    for (int s = 0; s < n_splits; ++s) {
+      const float w = wt[g * n_splits + s];
+      if (w > 0.f) v = fmaf(rg[s * rs], w, v);
+    }
+    at[i] = v;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < hpg * vd; i += blockDim.x) {
+    const int h = c * hpg + i / vd, col = i % vd;
+    const bf16* t = a.talk + (size_t)h * H;
+    float v = 0.f;
+    for (int g = 0; g < H; ++g) v = fmaf(bf2f(t[g]), at[g * vd + col], v);
+    if (a.out_bf) a.out_bf[(size_t)r * a.ldo_bf + (size_t)h * vd + col] = f2bf(v);
+    else a.out[(size_t)r * a.ldo + (size_t)h * vd + col] = v;
+  }
+}
+
 }  // namespace
 
 static size_t talk_smem(const TalkQueries& t) { return ((size_t)t.heads * t.dim + (size_t)t.heads * t.heads) * sizeof(float); }
@@ -644,6 +829,13 @@ static size_t talk_smem(const TalkQueries& t) { return ((size_t)t.heads * t.dim 
 cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
   if (a.n <= 0) return cudaSuccess;
   if ((a.k_norm || a.rope.dims > 0) && (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2)) return cudaErrorInvalidValue;
+  if (a.c.block > 0 && !a.whole_norm) return cudaErrorInvalidValue;  // pooled rows are written by the whole-projection form
+  if (a.whole_norm) {
+    if (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2 || !a.c.pool || a.tq.talk || a.v_lam || a.v_keep ||
+        (a.q_bf && !a.q) || !(a.k_bf || a.k))
+      return cudaErrorInvalidValue;
+    return launch_k(kv_store_whole_kernel, dim3(a.n), dim3(256), 0, st, a);
+  }
   size_t smem = 0;
   if (a.tq.talk) {
     if (a.tq.heads <= 0 || a.tq.kv_heads <= 0 || a.tq.heads % a.tq.kv_heads) return cudaErrorInvalidValue;
@@ -657,46 +849,70 @@ cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
   return launch_k(kv_store_rows_kernel, dim3(a.n), dim3(128), smem, st, a);
 }
 
+cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st) {
+  if (n <= 0 || c.block <= 0) return cudaSuccess;
+  return launch_k(kv_pool_rows_kernel, dim3(n), dim3(128), 0, st, c, pos, slot, block_table, max_pages);
+}
+
+static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStream_t st) {
+  const size_t smem = ((size_t)a.heads * splits + (size_t)a.heads * a.vdim) * sizeof(float);
+  if (smem > 48 * 1024) {
+    if (smem > 200 * 1024) return cudaErrorInvalidValue;
+    cudaError_t r = cudaFuncSetAttribute(gqa_talk_finish_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (r != cudaSuccess) return r;
+  }
+  return launch_k(gqa_talk_finish_kernel, dim3(a.n, a.kv_heads), dim3(128), smem, st, a, splits);
+}
+
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches) {
   if (n_launches) *n_launches = 0;
   if (a.n <= 0) return cudaSuccess;
   if (a.shared_keys && (a.maps != 1 || a.dim != a.c.kw)) return cudaErrorInvalidValue;
   if (a.finish == 3 && !a.gate) return cudaErrorInvalidValue;
   if (a.out_bf && a.maps != 1 && !a.out) return cudaErrorInvalidValue;  // two maps: the first one's result waits in the fp32 rows
+  if (a.talk && (a.maps != 1 || a.finish || a.unit_sink || a.shared_keys)) return cudaErrorInvalidValue;
+  if (a.c.block > 0 && (a.window <= 0 || a.slopes || a.shared_keys || a.maps != 1)) return cudaErrorInvalidValue;
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim;
+  if (a.talk && gqa_ws_floats(a.n, a.heads, 1, vcols) > a.ws_floats) return cudaErrorInvalidValue;
   // prompt portions over a bf16 cache: the tensor-core kernel (one launch, no workspace); QIE_ATTN_MMA=0 keeps the per-row kernel (A/B)
   static const bool mma_on = [] { const char* v = getenv("QIE_ATTN_MMA"); return !(v && v[0] == '0'); }();
-  if (mma_on && a.seg_start && a.c.elt_bytes == 2 && a.n >= 64 && a.dim <= 128 && a.vdim <= 128 && a.maps <= 2 && a.heads % a.kv_heads == 0 &&
+  if (mma_on && a.seg_start && a.c.elt_bytes == 2 && a.n >= 64 && a.dim <= 128 && (a.talk || a.vdim <= 128) && a.maps <= 2 && a.heads % a.kv_heads == 0 &&
       (a.finish != 2 || a.maps == 2)) {
-    if (n_launches) *n_launches = 1;
-    if (a.dim <= 32) return launch_prefill_mma_v<32>(a, a.seg_start, a.seg_slot, a.n_seg, st);
-    if (a.dim <= 64) return launch_prefill_mma_v<64>(a, a.seg_start, a.seg_slot, a.n_seg, st);
-    return launch_prefill_mma_v<128>(a, a.seg_start, a.seg_slot, a.n_seg, st);
+    if (n_launches) *n_launches = a.talk ? 2 : 1;
+    cudaError_t r;
+    if (a.dim <= 32) r = launch_prefill_mma_v<32>(a, a.seg_start, a.seg_slot, a.n_seg, st);
+    else if (a.dim <= 64) r = launch_prefill_mma_v<64>(a, a.seg_start, a.seg_slot, a.n_seg, st);
+    else r = launch_prefill_mma_v<128>(a, a.seg_start, a.seg_slot, a.n_seg, st);
+    if (r != cudaSuccess || !a.talk) return r;
+    return launch_talk_finish(a, 1, st);
   }
-  if (a.maps < 1 || a.maps > 2 || a.heads % a.kv_heads || (a.finish == 2 && a.maps != 2) || a.maps * a.vdim > ATHREADS * AMAXACC)
+  if (a.maps < 1 || a.maps > 2 || a.heads % a.kv_heads || (a.finish == 2 && a.maps != 2) || (!a.talk && a.maps * a.vdim > ATHREADS * AMAXACC))
     return cudaErrorInvalidValue;
   const int hpg = a.heads / a.kv_heads;
-  const int hpc = std::max(1, std::min(hpg, ATHREADS * AMAXACC / (a.maps * a.vdim)));
+  const int vc = a.talk ? std::min(vcols, 512) : vcols, nvc = (vcols + vc - 1) / vc;  // value columns per CTA
+  const int hpc = std::max(1, std::min(hpg, ATHREADS * AMAXACC / (a.maps * vc)));
   const int chunks = (hpg + hpc - 1) / hpc;
   // key splits: fill the machine when there are few rows, within the workspace
   int splits = 1;
-  const long ctas = (long)a.n * a.kv_heads * chunks;
+  const long ctas = (long)a.n * a.kv_heads * chunks * nvc;
   if (ctas < 2L * a.num_sms && a.max_keys > 2 * ATK) {
     splits = (int)std::min<long>((2L * a.num_sms + ctas - 1) / ctas, (a.max_keys + 2 * ATK - 1) / (2 * ATK));
     splits = std::max(1, std::min(splits, 16));
   }
-  const size_t one = gqa_ws_floats(a.n, a.heads, a.maps, a.vdim);
+  const size_t one = gqa_ws_floats(a.n, a.heads, a.maps, vcols);
   if (one > a.ws_floats) return cudaErrorInvalidValue;
   splits = (int)std::min<size_t>(splits, a.ws_floats / one);
   const int kd = a.maps * a.dim, qvm = hpc * a.maps;
-  const size_t smem = ((size_t)qvm * a.dim + (size_t)ATK * (kd + 1) + (size_t)ATK * a.vdim + (size_t)qvm * ATK + 3 * (size_t)qvm) * sizeof(float);
+  const size_t smem = ((size_t)qvm * a.dim + (size_t)ATK * (kd + 1) + (size_t)ATK * vc + (size_t)qvm * ATK + 3 * (size_t)qvm) * sizeof(float);
   if (smem > 200 * 1024) return cudaErrorInvalidValue;
   if (smem > 48 * 1024) {
     cudaError_t r = cudaFuncSetAttribute(gqa_attention_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (r != cudaSuccess) return r;
   }
-  cudaError_t r = launch_k(gqa_attention_kernel, dim3(a.n, a.kv_heads * chunks, splits), dim3(ATHREADS), smem, st, a, hpc, chunks, splits);
+  cudaError_t r = launch_k(gqa_attention_kernel, dim3(a.n, a.kv_heads * chunks * nvc, splits), dim3(ATHREADS), smem, st, a, hpc, chunks, splits, vc, nvc);
   if (r != cudaSuccess) return r;
   if (n_launches) *n_launches = 2;
+  if (a.talk) return launch_talk_finish(a, splits, st);
   return launch_k(gqa_finish_kernel, dim3(a.n, a.heads), dim3(128), (size_t)a.vdim * sizeof(float), st, a, splits);
 }
 

@@ -398,7 +398,7 @@ static void engine_free(qie_engine* e) {
   if (e->fam) {
     e->fam->release();
     delete e->fam;
-    e->fam = nullptr, e->ng = nullptr, e->fv = nullptr, e->dx = nullptr, e->dd = nullptr;
+    e->fam = nullptr, e->ng = nullptr, e->fv = nullptr, e->dx = nullptr, e->dd = nullptr, e->gb = nullptr;
   }
   if (!e->blob_owned) e->blob = nullptr;
   void* dev[] = {e->blob, e->cos_d, e->sin_d, e->kv.pool, e->block_table_d, e->ids_d, e->pos_d, e->slot_d,
@@ -1443,7 +1443,7 @@ const char* qie_kernel_kind_name(int kind) {
   static const char* names[KK_COUNT] = {"embedding", "rmsnorm", "gemm_qkv", "qkv_post", "attention", "gemm_o",
                                         "gemm_gateup", "gemm_down", "lm_head", "sample", "advance", "f32_norm", "f32_proj", "latent_store",
                                         "latent_attn", "mlstm_scan", "moe_route", "moe_experts", "moe_shared", "moe_combine", "hyper_streams", "kv_store",
-                                        "gqa_attn", "causal_conv", "lru_scan", "ssd_scan", "glu_act"};
+                                        "gqa_attn", "causal_conv", "lru_scan", "ssd_scan", "glu_act", "linear_attn", "norm_gate"};
   return kind >= 0 && kind < KK_COUNT ? names[kind] : nullptr;
 }
 
@@ -1494,13 +1494,15 @@ const char* qie_model_families(void) { return registry_names(); }
 const char* qie_engine_family(const qie_engine* e) { return !e ? "" : (e->fam ? e->fam->family_name() : "qwen"); }
 
 static int create_family(qie_engine* e, int family, const std::string& arg, bool synthetic, uint64_t seed) {
-  if (family != FAMILY_NOGATAR && family != FAMILY_FOSAVIK && family != FAMILY_DITENEX && family != FAMILY_DEDUNEX) return fail(QIE_EINVAL, "family not handled here");
+  if (family != FAMILY_NOGATAR && family != FAMILY_FOSAVIK && family != FAMILY_DITENEX && family != FAMILY_DEDUNEX && family != FAMILY_GEBADRA)
+    return fail(QIE_EINVAL, "family not handled here");
   if (e->opts.tp_size > 1) return fail(QIE_EINVAL, "this family is not sharded (tp_size must be 1)");
   int code = QIE_EIO;
   std::string err;
   if (family == FAMILY_NOGATAR) err = synthetic ? nogatar_create_synthetic(e, arg, seed, &code) : nogatar_create(e, arg, &code);
   else if (family == FAMILY_FOSAVIK) err = synthetic ? fosavik_create_synthetic(e, arg, seed, &code) : fosavik_create(e, arg, &code);
   else if (family == FAMILY_DITENEX) err = synthetic ? ditenex_create_synthetic(e, arg, seed, &code) : ditenex_create(e, arg, &code);
+  else if (family == FAMILY_GEBADRA) err = synthetic ? gebadra_create_synthetic(e, arg, seed, &code) : gebadra_create(e, arg, &code);
   else err = synthetic ? dedunex_create_synthetic(e, arg, seed, &code) : dedunex_create(e, arg, &code);
   if (!err.empty()) return fail(code, "%s", err.c_str());
   return QIE_OK;

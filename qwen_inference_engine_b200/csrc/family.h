@@ -1,4 +1,4 @@
-// family.h -- what the model families with a general row forward share (Nogatar, Fosavik, Ditenex, Dedunex): the interface the engine
+// family.h -- what the model families with a general row forward share (Nogatar, Fosavik, Ditenex, Dedunex, Gebadra): the interface the engine
 // drives them through (forward over rows, slot reset, release), the weight blob helpers (tensor layout, safetensors
 // reader, synthetic fill), the rotary tables and the projection helper that puts a plain GEMM on the tcgen05 kernel when
 // precision and shape allow.  A row is (sequence slot, position); rows of one sequence are consecutive and in position order
@@ -78,15 +78,17 @@ std::string load_safetensors_blob(const std::string& path, const std::vector<Ten
 // Rotation angles of position p: a_i = p * f_i, f_i = base^(-2i / dims), i < dims / 2.  With `scaled` (YaRN) the
 // frequencies are blended: with corr(t) = dims * ln(original / (2 pi t)) / (2 ln base), lo = max(floor(corr(fast)), 0),
 // hi = min(ceil(corr(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is
-// f_i / factor * ramp_i + f_i * (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.
+// f_i / factor * ramp_i + f_i * (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.  `linear` divides every
+// frequency (linear position scaling).
 struct RotaryCfg {
   int dims = 0;
   double base = 10000.0;
   bool scaled = false;
   double factor = 1.0, original = 0.0, fast = 0.0, slow = 0.0;
+  double linear = 1.0;
   bool operator==(const RotaryCfg& o) const {
     return dims == o.dims && base == o.base && scaled == o.scaled && factor == o.factor && original == o.original && fast == o.fast &&
-           slow == o.slow;
+           slow == o.slow && linear == o.linear;
   }
 };
 // cos / sin tables [context, dims / 2], worked out in double, the magnitude factor folded in

@@ -124,7 +124,7 @@ void rotary_tables(const RotaryCfg& r, int context, std::vector<float>* c, std::
   const int half = r.dims / 2;
   std::vector<double> f(half);
   double mag = 1.0;
-  for (int i = 0; i < half; ++i) f[i] = pow(r.base, -2.0 * i / r.dims);
+  for (int i = 0; i < half; ++i) f[i] = pow(r.base, -2.0 * i / r.dims) / r.linear;
   if (r.scaled) {
     const double PI = 3.14159265358979323846;
     auto corr = [&](double turns) { return r.dims * log(r.original / (2.0 * PI * turns)) / (2.0 * log(r.base)); };

@@ -26,10 +26,14 @@ namespace qie {
 cudaError_t launch_embed_streams(float* X, const bf16* embed, const bf16* pos_table, const int* ids, const int* pos, int width, int streams,
                                  int n, cudaStream_t st);
 // One step over the streams of every row, both halves optional:
-//   write (y1 != null):  X'[t] = sum_s mix[s, t] X[s] + out[t] * (s1 * y1 + s2 * y2)      (all t at once from the old X)
-//   read  (h != null):   u = sum_s in[s] X'[s]  (in == null: plain sum);  h = u / sqrt(mean(u^2) + eps) * w
+//   write (y1 / y1_bf):  X'[t] = sum_s mix[s, t] X[s] + out[t] * (s1 * n(y1) + s2 * n(y2))      (all t at once from the old X)
+//                        n(y) = y, or with y1_norm / y2_norm y / sqrt(mean(y^2) + eps) * y*_norm
+//                        dump (optional) receives sum_t X'[t]
+//   read  (h / h_bf):    u = sum_s in[s] X'[s]  (in == null: plain sum);  h = u / sqrt(mean(u^2) + eps) * w, or with b the layer
+//                        norm (u - mean(u)) / sqrt(mean((u - mean(u))^2) + eps) * w + b
 //                        rows: src(r) = gather ? gather[r] : r;  sum_out (optional) receives u itself
-// A sublayer's write and the next sublayer's read are one launch.
+//   first (ids):         the streams do not exist yet: X[s] = embed[ids[r]] for every s, before the read half
+// A sublayer's write and the next sublayer's read are one launch.  Sublayer outputs and h are fp32 or dense bf16 rows.
 struct HyperStep {
   float* X = nullptr;
   int width = 0, streams = 0, n = 0;
@@ -38,12 +42,21 @@ struct HyperStep {
   const bf16* out = nullptr;  // [streams]
   const float* y1 = nullptr;
   const float* y2 = nullptr;
+  const bf16* y1_bf = nullptr;
+  const bf16* y2_bf = nullptr;
+  const bf16* y1_norm = nullptr;  // [width]
+  const bf16* y2_norm = nullptr;
   float s1 = 1.f, s2 = 0.f;
+  float* dump = nullptr;
   // read half
+  const int* ids = nullptr;
+  const bf16* embed = nullptr;
   const bf16* in = nullptr;  // [streams]
   const bf16* w = nullptr;   // [width] norm weight (null: no norm, h = u)
+  const bf16* b = nullptr;   // [width] norm bias: a layer norm instead of an RMS norm
   float eps = 0.f;
   float* h = nullptr;
+  bf16* h_bf = nullptr;
   float* sum_out = nullptr;
   const int* gather = nullptr;
 };
@@ -59,12 +72,23 @@ struct KvRowCache {
   size_t page_elems = 0;  // elements per page over all layers
   size_t layer_off = 0;
   int kw = 0, vw = 0;
+  // pooled rows (block > 0): one row [keys | values] per block of `block` consecutive positions, the mean of their rows; block b
+  // lies in the page that holds its last position, as that page's pooled row number b - floor(first position of the page / block)
+  int block = 0;
+  size_t pool_off = 0;  // elements into the page
 };
+// pooled rows that a page has room for
+inline int kv_pool_rows(int page_size, int block) { return block > 0 ? (page_size + block - 1) / block : 0; }
 // per row: keys k[r, 0:kw] (optionally unit-RMS normed per `norm_dim` consecutive elements, times k_norm) and values
 // v[r, 0:vw] -> cache row (slot, pos).  Rider: the row's queries q[r, 0:q_heads*norm_dim] normed in place with q_norm.
 // Optional: biases added to keys and values first; values blended with another layer's values of the same rows,
 // v = (1 - lam) v + lam v_other (lam one bf16 number on the device); the stored values also kept as fp32 rows (v_keep);
 // the head-mixed queries of the row (TalkQueries below) written in the same launch.
+// whole_norm: the unit RMS norm of the keys (and of the queries) goes over the row's whole key part (all its query heads)
+// at once, with weights k_norm [kw] and q_norm [q_heads * norm_dim]; norm_dim is then the head size that rotates.  In this form
+// the sources may be bf16 rows (*_bf, row stride ld_bf) and the queries go from q_bf to the fp32 rows q.
+// Pooled rows (c.block > 0): the row that holds a block's last position is followed by the block's mean row, in the same
+// launch when every row of the batch is another sequence's (one_each), else by launch_kv_pool_rows.
 // Rotary positions (rope.dims > 0): after the norm, the first rope.dims elements of every `norm_dim` consecutive elements
 // of the keys and of the queries are rotated by the row's position (with two score maps every map of every head is such a
 // group); q_bias is added to the queries before their norm.
@@ -96,6 +120,9 @@ struct KvStoreArgs {
   const bf16* v_bias = nullptr;  // [vw]
   const bf16* q_bias = nullptr;  // [q_heads * norm_dim]
   RopeTable rope;
+  int whole_norm = 0, one_each = 0;
+  const bf16 *q_bf = nullptr, *k_bf = nullptr, *v_bf = nullptr;
+  int ld_bf = 0;
   const bf16* v_lam = nullptr;
   const float* v_other = nullptr;
   int ld_vo = 0;
@@ -106,6 +133,8 @@ struct KvStoreArgs {
   int max_pages = 0, n = 0;
 };
 cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st);
+// pooled rows of every block whose last position is among the n rows (their keys and values are in the cache already)
+cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st);
 // out[r, h, :] over the keys j of row r's sequence with j <= pos and (window <= 0 or pos - j < window or j < keep_first).
 // `maps` score maps per head (queries [h][map][dim], keys [g][map][dim]) share the values [g][vdim]; head h reads kv
 // head h / (heads / kv_heads).  unit_sink adds 1 to every softmax denominator (as if one more key with a zero score and nothing to contribute took part).
@@ -116,6 +145,11 @@ cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st);
 // shared_keys: every head scores against the WHOLE key part of the cached row (dim = kw / maps elements: the keys of all
 // kv heads side by side) while its values stay those of kv head h / (heads / kv_heads); the queries are then
 // [h][map][kw / maps] (TalkQueries builds them).
+// c.block > 0 (with a window): beside the tokens of the window a row sees the pooled rows of the blocks that lie wholly before
+// it, block b when (b + 1) * block - 1 <= pos - window, in the same softmax.
+// talk (optional, [heads, heads]): the heads' softmax weights are mixed, weight_h <- sum_g talk[h, g] weight_g, before they meet
+// the values of head h's own kv head.  Computed as out_h = sum_g talk[h, g] (softmax_g . values of h's kv head): every
+// head attends to the values of all kv heads, and the heads are mixed when its result is complete.
 // The keys of a row may be split over CTAs; partial (max, sum, acc) go through ws and a second kernel finishes.
 struct GqaAttnArgs {
   KvRowCache c;
@@ -133,6 +167,7 @@ struct GqaAttnArgs {
   int ldg = 0;
   const float* slopes = nullptr;
   int shared_keys = 0;
+  const bf16* talk = nullptr;
   float lam = 0.f, post = 1.f, eps = 0.f;
   const int *pos = nullptr, *slot = nullptr, *block_table = nullptr;
   int max_pages = 0, n = 0, max_keys = 0;
@@ -146,6 +181,7 @@ struct GqaAttnArgs {
   int n_seg = 0;
 };
 // floats of workspace that n rows need with one split
+// (vdim: with `talk` the value elements of all kv heads together)
 inline size_t gqa_ws_floats(int n, int heads, int maps, int vdim) { return (size_t)n * heads * maps * (vdim + 2); }
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches = nullptr);
 

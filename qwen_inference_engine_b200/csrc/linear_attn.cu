@@ -1,0 +1,414 @@
+// linear_attn.cu -- linear attention with a fixed decay per head (gebadra.h): S = decay S + k v^T, o = S^T q, an fp32 matrix
+// per head and sequence slot.  Two forms of the same recurrence:
+//  * token by token: a CTA owns a block of 32 value columns of one head of one segment; its state columns live in registers
+//    (any head size, fp32 or bf16 sources) -- decode steps, short portions and 32-bit mode;
+//  * chunks of 64 rows on tensor cores (bf16 sources, prompt portions): every chunk's own contribution to the state
+//    U = sum_s decay^(L-1-s) k_s v_s^T, a carry pass S <- decay^L S + U over the chunks of a segment that leaves each chunk's
+//    entry state in place of its U, and the outputs o_t = decay^(t+1) S^T q_t + sum_(s<=t) decay^(t-s) (q_t . k_s) v_s.
+//    Everything that is not a projection stays fp32-like on the tensor cores: decayed keys, decayed scores and the entry
+//    state enter the products as bf16 hi + lo pairs (two MMAs), accumulators are fp32.
+#include <algorithm>
+
+#include "gebadra.h"
+#include "launch.h"
+
+namespace qie {
+namespace {
+
+constexpr int LA_TOK = 8;      // tokens staged at a time (token-by-token form)
+constexpr int LA_NR = 8;       // state rows per thread
+constexpr int LC = LINEAR_CHUNK;
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+
+// CTA (head, block of 32 value columns, segment); thread = (column, part of LA_NR state rows)
+__global__ void __launch_bounds__(1024) linear_scan_kernel(const LinearAttnArgs a, int parts) {
+  extern __shared__ float la_smem[];  // q [LA_TOK][DP] | k [LA_TOK][DP] | v [LA_TOK][32] | partial o [LA_TOK][parts][32]
+  pdl_wait();
+  pdl_trigger();
+  const int h = blockIdx.x, c0 = blockIdx.y * 32, seg = blockIdx.z;
+  const int dim = a.dim, vdim = a.vdim, DP = parts * LA_NR;
+  float* qs = la_smem;
+  float* ks = qs + LA_TOK * DP;
+  float* vs = ks + LA_TOK * DP;
+  float* po = vs + LA_TOK * 32;
+  const int tid = threadIdx.x, col = tid & 31, part = tid >> 5;
+  const int r0 = a.seg_start[seg], r1 = a.seg_start[seg + 1];
+  const float lam = a.decay_pow[h * (LC + 1) + 1];
+  float* st = a.state + (size_t)a.seg_slot[seg] * a.slot_stride + (size_t)h * dim * vdim;
+  const bool cv = c0 + col < vdim;
+  float S[LA_NR];
+#pragma unroll
+  for (int i = 0; i < LA_NR; ++i) {
+    const int d = part * LA_NR + i;
+    S[i] = cv && d < dim ? st[(size_t)d * vdim + c0 + col] : 0.f;
+  }
+  auto act = [&](float z) { return a.act ? silu_f(z) : z; };
+  for (int t0 = r0; t0 < r1; t0 += LA_TOK) {
+    const int nt = min(LA_TOK, r1 - t0);
+    __syncthreads();
+    for (int i = tid; i < nt * DP; i += blockDim.x) {
+      const int t = i / DP, d = i - t * DP;
+      float q = 0.f, k = 0.f;
+      if (d < dim) {
+        if (a.q_bf) {
+          const size_t o = (size_t)(t0 + t) * a.ld_bf + h * dim + d;
+          q = act(bf2f(a.q_bf[o])), k = act(bf2f(a.k_bf[o])) * a.k_scale;
+        } else {
+          const size_t o = (size_t)(t0 + t) * a.ld + h * dim + d;
+          q = act(a.q[o]), k = act(a.k[o]) * a.k_scale;
+        }
+      }
+      qs[i] = q, ks[i] = k;
+    }
+    for (int i = tid; i < nt * 32; i += blockDim.x) {
+      const int t = i >> 5, c = c0 + (i & 31);
+      float v = 0.f;
+      if (c < vdim) v = act(a.v_bf ? bf2f(a.v_bf[(size_t)(t0 + t) * a.ld_bf + h * vdim + c]) : a.v[(size_t)(t0 + t) * a.ld + h * vdim + c]);
+      vs[i] = v;
+    }
+    __syncthreads();
+    for (int t = 0; t < nt; ++t) {
+      const float v = vs[t * 32 + col];
+      const float4* q4 = reinterpret_cast<const float4*>(qs + t * DP + part * LA_NR);
+      const float4* k4 = reinterpret_cast<const float4*>(ks + t * DP + part * LA_NR);
+      float o = 0.f;
+#pragma unroll
+      for (int i = 0; i < LA_NR / 4; ++i) {
+        const float4 q = q4[i], k = k4[i];
+        S[4 * i] = fmaf(lam, S[4 * i], k.x * v), o = fmaf(S[4 * i], q.x, o);
+        S[4 * i + 1] = fmaf(lam, S[4 * i + 1], k.y * v), o = fmaf(S[4 * i + 1], q.y, o);
+        S[4 * i + 2] = fmaf(lam, S[4 * i + 2], k.z * v), o = fmaf(S[4 * i + 2], q.z, o);
+        S[4 * i + 3] = fmaf(lam, S[4 * i + 3], k.w * v), o = fmaf(S[4 * i + 3], q.w, o);
+      }
+      po[(t * parts + part) * 32 + col] = o;
+    }
+    __syncthreads();
+    for (int i = tid; i < nt * 32; i += blockDim.x) {
+      const int t = i >> 5, c = i & 31;
+      if (c0 + c >= vdim) continue;
+      float o = 0.f;
+      for (int p = 0; p < parts; ++p) o += po[(t * parts + p) * 32 + c];
+      a.out[(size_t)(t0 + t) * a.ldo + h * vdim + c0 + c] = o;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < LA_NR; ++i) {
+    const int d = part * LA_NR + i;
+    if (cv && d < dim) st[(size_t)d * vdim + c0 + col] = S[i];
+  }
+}
+
+// ---------------------------------------------------------------- chunks of 64 rows on tensor cores
+__device__ __forceinline__ void ldmatrix_x2_trans_la(uint32_t& r0, uint32_t& r1, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+
+// which chunk: {first row, rows, segment} of chunk number id (false: there is no such chunk)
+__device__ __forceinline__ bool find_chunk(const LinearAttnArgs& a, int id, int* info) {
+  for (int s = 0; s < a.n_seg; ++s) {
+    const int r0 = a.seg_start[s], len = a.seg_start[s + 1] - r0, nc = (len + LC - 1) / LC;
+    if (id < nc) {
+      info[0] = r0 + id * LC, info[1] = min(LC, len - id * LC), info[2] = s;
+      return true;
+    }
+    id -= nc;
+  }
+  return false;
+}
+
+// 64 rows x cols of a bf16 source (columns col0 ..) -> smem tile [64][P + 8], zeros beyond, silu where asked
+template <int P>
+__device__ __forceinline__ void load_tile(const bf16* src, int ld, int row0, int nrows, int cols, int act, bf16 (*dst)[P + 8]) {
+  const bool vec = cols % 8 == 0 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+  for (int i = threadIdx.x; i < LC * (P / 8); i += blockDim.x) {
+    const int r = i / (P / 8), c = (i % (P / 8)) * 8;
+    bf16* d = &dst[r][c];
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (r < nrows && c < cols) {
+      const bf16* s = src + (size_t)(row0 + r) * ld + c;
+      if (vec) {
+        v = *reinterpret_cast<const uint4*>(s);
+      } else {
+        bf16 t[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) t[e] = c + e < cols ? s[e] : f2bf(0.f);
+        v = make_uint4(pack2(t[0], t[1]), pack2(t[2], t[3]), pack2(t[4], t[5]), pack2(t[6], t[7]));
+      }
+      if (act) {
+        v.x = pack2(f2bf(silu_f(lo2f(v.x))), f2bf(silu_f(hi2f(v.x)))), v.y = pack2(f2bf(silu_f(lo2f(v.y))), f2bf(silu_f(hi2f(v.y))));
+        v.z = pack2(f2bf(silu_f(lo2f(v.z))), f2bf(silu_f(hi2f(v.z)))), v.w = pack2(f2bf(silu_f(lo2f(v.w))), f2bf(silu_f(hi2f(v.w))));
+      }
+    }
+    *reinterpret_cast<uint4*>(d) = v;
+  }
+}
+
+// CTA (chunk, head): U [dim, vdim] = sum_s decay^(L-1-s) k_scale k_s v_s^T -> ws.  Warp w owns the state rows 16 w .. (and 64 further).
+template <int DP, int VP>
+__global__ void __launch_bounds__(128) linear_chunk_state_kernel(const LinearAttnArgs a) {
+  extern __shared__ __align__(16) unsigned char lc_smem[];
+  typedef bf16 KT[DP + 8];
+  typedef bf16 VT[VP + 8];
+  KT* Kh = reinterpret_cast<KT*>(lc_smem);
+  KT* Kl = Kh + LC;
+  VT* Vs = reinterpret_cast<VT*>(Kl + LC);
+  __shared__ int info[3];
+  pdl_wait();
+  pdl_trigger();
+  if (threadIdx.x == 0 && !find_chunk(a, blockIdx.x, info)) info[0] = -1;
+  __syncthreads();
+  if (info[0] < 0) return;
+  const int h = blockIdx.y, row0 = info[0], L = info[1], dim = a.dim, vdim = a.vdim;
+  load_tile<DP>(a.k_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Kh);
+  load_tile<VP>(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim, a.act, Vs);
+  __syncthreads();
+  const float* pw = a.decay_pow + h * (LC + 1);
+  for (int i = threadIdx.x; i < L * DP; i += blockDim.x) {  // decayed keys as hi + lo pairs
+    const int s = i / DP, d = i - s * DP;
+    const float x = bf2f(Kh[s][d]) * (a.k_scale * pw[L - 1 - s]);
+    const bf16 hi = f2bf(x);
+    Kh[s][d] = hi;
+    Kl[s][d] = f2bf(x - bf2f(hi));
+  }
+  for (int i = L * DP + threadIdx.x; i < LC * DP; i += blockDim.x) Kl[i / DP][i % DP] = f2bf(0.f);
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* U = a.ws + ((size_t)blockIdx.x * a.heads + h) * dim * vdim;
+  for (int m0 = warp * 16; m0 < DP && m0 < dim; m0 += 64) {
+    float acc[VP / 8][4];
+#pragma unroll
+    for (int i = 0; i < VP / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+    for (int kb = 0; kb < LC / 16; ++kb) {
+      // A = K'^T: element (state row m, token k) lies at [k][m]
+      uint32_t ah[4], al[4];
+      const int tok = kb * 16 + (lane >> 4) * 8 + (lane & 7), dm = m0 + ((lane >> 3) & 1) * 8;
+      ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], smem_u32(&Kh[tok][dm]));
+      ldmatrix_x4_trans(al[0], al[1], al[2], al[3], smem_u32(&Kl[tok][dm]));
+#pragma unroll
+      for (int vb = 0; vb < VP / 8; ++vb) {
+        uint32_t b0, b1;
+        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][vb * 8]));
+        mma_bf16_16816(acc[vb], ah, b0, b1);
+        mma_bf16_16816(acc[vb], al, b0, b1);
+      }
+    }
+    const int r = m0 + (lane >> 2), c = (lane & 3) * 2;
+#pragma unroll
+    for (int vb = 0; vb < VP / 8; ++vb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int rr = r + (e >> 1) * 8, cc = vb * 8 + c + (e & 1);
+        if (rr < dim && cc < vdim) U[(size_t)rr * vdim + cc] = acc[vb][e];
+      }
+  }
+}
+
+// thread = state element of (segment, head): walks the segment's chunks; the chunk's U becomes its entry state
+__global__ void __launch_bounds__(256) linear_carry_kernel(const LinearAttnArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const int seg = blockIdx.y, per = a.dim * a.vdim, i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= a.heads * per) return;
+  int first = 0;
+  for (int s = 0; s < seg; ++s) first += (a.seg_start[s + 1] - a.seg_start[s] + LC - 1) / LC;
+  const int len = a.seg_start[seg + 1] - a.seg_start[seg], nc = (len + LC - 1) / LC, h = i / per;
+  const float* pw = a.decay_pow + h * (LC + 1);
+  const float full = pw[LC], last = pw[len - (nc - 1) * LC];
+  float* st = a.state + (size_t)a.seg_slot[seg] * a.slot_stride + i;
+  const size_t stride = (size_t)a.heads * per;
+  float* w = a.ws + (size_t)first * stride + i;
+  float S = *st;
+  constexpr int PF = 8;  // chunks whose loads are in flight
+  float u[PF];
+  for (int c0 = 0; c0 < nc; c0 += PF) {
+#pragma unroll
+    for (int j = 0; j < PF; ++j) u[j] = c0 + j < nc ? w[(size_t)(c0 + j) * stride] : 0.f;
+#pragma unroll
+    for (int j = 0; j < PF; ++j) {
+      if (c0 + j >= nc) break;
+      w[(size_t)(c0 + j) * stride] = S;
+      S = fmaf(c0 + j == nc - 1 ? last : full, S, u[j]);
+    }
+  }
+  *st = S;
+}
+
+// CTA (chunk, head): the outputs of the chunk's rows from its entry state and its own keys and values; warp w owns rows 16 w ..
+template <int DP, int VP>
+__global__ void __launch_bounds__(128) linear_chunk_out_kernel(const LinearAttnArgs a) {
+  extern __shared__ __align__(16) unsigned char lc_smem[];
+  typedef bf16 KT[DP + 8];
+  typedef bf16 VT[VP + 8];
+  KT* Qs = reinterpret_cast<KT*>(lc_smem);
+  KT* Ks = Qs + LC;
+  VT* Vs = reinterpret_cast<VT*>(Ks + LC);
+  VT* Sh = Vs + LC;   // [DP] entry state, hi
+  VT* Sl = Sh + DP;   // lo
+  __shared__ int info[3];
+  __shared__ float pw[LC + 1];
+  pdl_wait();
+  pdl_trigger();
+  if (threadIdx.x == 0 && !find_chunk(a, blockIdx.x, info)) info[0] = -1;
+  __syncthreads();
+  if (info[0] < 0) return;
+  const int h = blockIdx.y, row0 = info[0], L = info[1], dim = a.dim, vdim = a.vdim, tid = threadIdx.x;
+  for (int i = tid; i <= LC; i += 128) pw[i] = a.decay_pow[h * (LC + 1) + i];
+  load_tile<DP>(a.q_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Qs);
+  load_tile<DP>(a.k_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Ks);
+  load_tile<VP>(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim, a.act, Vs);
+  {
+    const float* S = a.ws + ((size_t)blockIdx.x * a.heads + h) * dim * vdim;
+    if (vdim % 4 == 0) {
+      for (int i = tid; i < DP * (VP / 4); i += 128) {
+        const int d = i / (VP / 4), c = (i % (VP / 4)) * 4;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d < dim && c < vdim) x = *reinterpret_cast<const float4*>(S + (size_t)d * vdim + c);
+        const bf16 h0 = f2bf(x.x), h1 = f2bf(x.y), h2 = f2bf(x.z), h3 = f2bf(x.w);
+        *reinterpret_cast<uint2*>(&Sh[d][c]) = make_uint2(pack2(h0, h1), pack2(h2, h3));
+        *reinterpret_cast<uint2*>(&Sl[d][c]) =
+            make_uint2(pack2(f2bf(x.x - bf2f(h0)), f2bf(x.y - bf2f(h1))), pack2(f2bf(x.z - bf2f(h2)), f2bf(x.w - bf2f(h3))));
+      }
+    } else {
+      for (int i = tid; i < DP * VP; i += 128) {
+        const int d = i / VP, c = i % VP;
+        const float x = d < dim && c < vdim ? S[(size_t)d * vdim + c] : 0.f;
+        const bf16 hi = f2bf(x);
+        Sh[d][c] = hi, Sl[d][c] = f2bf(x - bf2f(hi));
+      }
+    }
+  }
+  __syncthreads();
+  const int warp = tid >> 5, lane = tid & 31, w0 = warp * 16;
+  if (w0 >= L) return;
+  const int qr = lane >> 2, qc = (lane & 3) * 2;
+  const int t0 = w0 + qr, t1 = t0 + 8;  // this thread's two rows of the chunk
+  float o[VP / 8][4];
+#pragma unroll
+  for (int i = 0; i < VP / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float s[LC / 8][4];
+#pragma unroll
+  for (int i = 0; i < LC / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll
+  for (int kk = 0; kk < DP / 16; ++kk) {
+    uint32_t qf[4];
+    ldmatrix_x4(qf[0], qf[1], qf[2], qf[3], smem_u32(&Qs[w0 + (lane & 15)][kk * 16 + (lane >> 4) * 8]));
+#pragma unroll
+    for (int nb = 0; nb < LC / 8; ++nb) {
+      if (nb * 8 > w0 + 15) break;  // later than every row of the warp
+      uint32_t b0, b1;
+      ldmatrix_x2(b0, b1, smem_u32(&Ks[nb * 8 + (lane & 7)][kk * 16 + ((lane >> 3) & 1) * 8]));
+      mma_bf16_16816(s[nb], qf, b0, b1);
+    }
+#pragma unroll
+    for (int vb = 0; vb < VP / 8; ++vb) {
+      uint32_t b0, b1;
+      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sh[kk * 16 + (lane & 15)][vb * 8]));
+      mma_bf16_16816(o[vb], qf, b0, b1);
+      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sl[kk * 16 + (lane & 15)][vb * 8]));
+      mma_bf16_16816(o[vb], qf, b0, b1);
+    }
+  }
+  {
+    const float e0 = pw[t0 + 1], e1 = pw[t1 + 1];
+#pragma unroll
+    for (int vb = 0; vb < VP / 8; ++vb) o[vb][0] *= e0, o[vb][1] *= e0, o[vb][2] *= e1, o[vb][3] *= e1;
+  }
+#pragma unroll
+  for (int kb = 0; kb < LC / 16; ++kb) {
+    if (kb * 16 > w0 + 15) break;
+    uint32_t ph[4], pl[4];
+#pragma unroll
+    for (int f = 0; f < 4; ++f) {
+      const int nb = 2 * kb + (f >> 1), j = nb * 8 + qc, t = (f & 1) ? t1 : t0;
+      const float x0 = j <= t ? s[nb][(f & 1) * 2] * (a.k_scale * pw[t - j]) : 0.f;
+      const float x1 = j + 1 <= t ? s[nb][(f & 1) * 2 + 1] * (a.k_scale * pw[t - j - 1]) : 0.f;
+      const bf16 h0 = f2bf(x0), h1 = f2bf(x1);
+      ph[f] = pack2(h0, h1);
+      pl[f] = pack2(f2bf(x0 - bf2f(h0)), f2bf(x1 - bf2f(h1)));
+    }
+#pragma unroll
+    for (int vb = 0; vb < VP / 8; ++vb) {
+      uint32_t b0, b1;
+      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][vb * 8]));
+      mma_bf16_16816(o[vb], ph, b0, b1);
+      mma_bf16_16816(o[vb], pl, b0, b1);
+    }
+  }
+  const bool v0 = t0 < L, v1 = t1 < L;
+  float n0 = 1.f, n1 = 1.f;
+  if (a.norm_gate) {  // a row of a head lies in the four threads of a quad
+    float q0 = 0.f, q1 = 0.f;
+#pragma unroll
+    for (int vb = 0; vb < VP / 8; ++vb) q0 = fmaf(o[vb][0], o[vb][0], fmaf(o[vb][1], o[vb][1], q0)), q1 = fmaf(o[vb][2], o[vb][2], fmaf(o[vb][3], o[vb][3], q1));
+    q0 += __shfl_xor_sync(0xffffffffu, q0, 1), q1 += __shfl_xor_sync(0xffffffffu, q1, 1);
+    q0 += __shfl_xor_sync(0xffffffffu, q0, 2), q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
+    n0 = 1.0f / sqrtf(q0 / (float)vdim + a.eps), n1 = 1.0f / sqrtf(q1 / (float)vdim + a.eps);
+  }
+#pragma unroll
+  for (int vb = 0; vb < VP / 8; ++vb)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = vb * 8 + qc + e;
+      if (c >= vdim) continue;
+      const size_t ra = (size_t)(row0 + t0), rb = (size_t)(row0 + t1);
+      if (a.norm_gate) {
+        if (v0) a.out_bf[ra * a.ldo_bf + h * vdim + c] = f2bf(o[vb][e] * n0 * silu_f(bf2f(a.g_bf[ra * a.ld_bf + h * vdim + c])));
+        if (v1) a.out_bf[rb * a.ldo_bf + h * vdim + c] = f2bf(o[vb][2 + e] * n1 * silu_f(bf2f(a.g_bf[rb * a.ld_bf + h * vdim + c])));
+      } else {
+        if (v0) a.out[ra * a.ldo + h * vdim + c] = o[vb][e];
+        if (v1) a.out[rb * a.ldo + h * vdim + c] = o[vb][2 + e];
+      }
+    }
+}
+
+template <int DP, int VP>
+cudaError_t launch_chunked(const LinearAttnArgs& a, cudaStream_t st) {
+  const int chunks = a.n_rows / LC + a.n_seg;  // upper bound
+  const size_t s1 = ((size_t)2 * LC * (DP + 8) + (size_t)LC * (VP + 8)) * sizeof(bf16);
+  const size_t s2 = ((size_t)2 * LC * (DP + 8) + (size_t)(LC + 2 * DP) * (VP + 8)) * sizeof(bf16);
+  static PerDeviceOnce once;
+  if (once.need()) {
+    cudaError_t r;
+    if ((r = cudaFuncSetAttribute(linear_chunk_state_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1)) != cudaSuccess) return r;
+    if ((r = cudaFuncSetAttribute(linear_chunk_out_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2)) != cudaSuccess) return r;
+    once.done();
+  }
+  cudaError_t r = launch_k(linear_chunk_state_kernel<DP, VP>, dim3(chunks, a.heads), dim3(128), s1, st, a);
+  if (r != cudaSuccess) return r;
+  const int per = a.heads * a.dim * a.vdim;
+  if ((r = launch_k(linear_carry_kernel, dim3((per + 255) / 256, a.n_seg), dim3(256), 0, st, a)) != cudaSuccess) return r;
+  return launch_k(linear_chunk_out_kernel<DP, VP>, dim3(chunks, a.heads), dim3(128), s2, st, a);
+}
+
+}  // namespace
+
+bool linear_attention_chunked(const LinearAttnArgs& a) {
+  return a.q_bf && a.k_bf && a.v_bf && a.n_rows >= LC && a.dim <= 128 && a.vdim <= 128 && a.ws &&
+         linear_ws_floats(a.n_rows, a.n_seg, a.heads, a.dim, a.vdim) <= a.ws_floats;
+}
+
+cudaError_t launch_linear_attention(const LinearAttnArgs& a, cudaStream_t st, int* n_launches) {
+  if (n_launches) *n_launches = 0;
+  if (a.n_rows <= 0 || a.n_seg <= 0) return cudaSuccess;
+  if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || !a.decay_pow || !a.state || !(a.q_bf || a.q)) return cudaErrorInvalidValue;
+  const bool chunked = linear_attention_chunked(a);
+  if (a.norm_gate ? (!chunked || !a.g_bf || !a.out_bf) : !a.out) return cudaErrorInvalidValue;
+  if (chunked) {
+    if (n_launches) *n_launches = 3;
+    if (a.dim <= 64) return a.vdim <= 64 ? launch_chunked<64, 64>(a, st) : launch_chunked<64, 128>(a, st);
+    return a.vdim <= 64 ? launch_chunked<128, 64>(a, st) : launch_chunked<128, 128>(a, st);
+  }
+  const int parts = (a.dim + LA_NR - 1) / LA_NR;
+  if (parts > 32) return cudaErrorInvalidValue;  // head sizes up to 256
+  if (n_launches) *n_launches = 1;
+  const size_t smem = ((size_t)LA_TOK * 2 * parts * LA_NR + LA_TOK * 32 + (size_t)LA_TOK * parts * 32) * sizeof(float);
+  if (smem > 48 * 1024) {
+    cudaError_t r = cudaFuncSetAttribute(linear_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    if (r != cudaSuccess) return r;
+  }
+  return launch_k(linear_scan_kernel, dim3(a.heads, (a.vdim + 31) / 32, a.n_seg), dim3(32 * parts), smem, st, a, parts);
+}
+
+}  // namespace qie

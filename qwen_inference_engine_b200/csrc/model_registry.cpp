@@ -24,6 +24,7 @@ const Row kRegistry[] = {
     {"Fosavik", FAMILY_FOSAVIK},
     {"Ditenex", FAMILY_DITENEX},
     {"Dedunex", FAMILY_DEDUNEX},
+    {"Gebadra", FAMILY_GEBADRA},
     {"Qwen2ForCausalLM", FAMILY_QWEN},
     {"Qwen3ForCausalLM", FAMILY_QWEN},
 };

@@ -1,66 +1,19 @@
 // rmsnorm_f32.cu -- RMS norms of a model whose sublayers sit between two norms (ditenex.h): the output norm folded
 // into the residual add together with the next sublayer's input norm, and the input norm of a mixer that reads a blend
 // of each row with the row before it (token shift) with one carried row per sequence slot; and the grouped RMS norm of a
-// model of parallel blocks (dedunex.h): the residual add of the two sublayer outputs and the next block's norm in one kernel.
+// model of parallel blocks (dedunex.h): the residual add of the two sublayer outputs and the next block's norm in one kernel;
+// and the grouped norm with a gate behind it (gebadra.h).
 // All fp32, one CTA per row, every reduction in a fixed order per row, so a row's result does not depend on the rows it
 // shares a launch with.
 #include "dedunex.h"
 #include "ditenex.h"
+#include "gebadra.h"
 #include "launch.h"
 #include "moe_route.cuh"
+#include "pack.cuh"
 
 namespace qie {
 namespace {
-
-__device__ __forceinline__ float block_sum_r(float v, float* red) {
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
-  __syncthreads();  // red may still be read from the previous call
-  if (l == 0) red[w] = v;
-  __syncthreads();
-  float t = l < nw ? red[l] : 0.f;
-  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
-  return t;
-}
-
-// V consecutive elements per thread and step (V = 4: 16-byte fp32 and 8-byte bf16 accesses when the width and the
-// pointers allow it; V = 1 otherwise)
-template <int V>
-struct Pack {
-  float v[V];
-};
-template <int V>
-__device__ __forceinline__ Pack<V> ld_f32(const float* p) {
-  Pack<V> r;
-  if constexpr (V == 4) {
-    const float4 t = *reinterpret_cast<const float4*>(p);
-    r.v[0] = t.x, r.v[1] = t.y, r.v[2] = t.z, r.v[3] = t.w;
-  } else {
-    r.v[0] = p[0];
-  }
-  return r;
-}
-template <int V>
-__device__ __forceinline__ Pack<V> ld_bf16(const bf16* p) {
-  Pack<V> r;
-  if constexpr (V == 4) {
-    const uint2 t = *reinterpret_cast<const uint2*>(p);
-    r.v[0] = lo2f(t.x), r.v[1] = hi2f(t.x), r.v[2] = lo2f(t.y), r.v[3] = hi2f(t.y);
-  } else {
-    r.v[0] = bf2f(p[0]);
-  }
-  return r;
-}
-template <int V>
-__device__ __forceinline__ void st_f32(float* p, const Pack<V>& r) {
-  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-  else p[0] = r.v[0];
-}
-template <int V>
-__device__ __forceinline__ void st_bf16(bf16* p, const Pack<V>& r) {
-  if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack2(f2bf(r.v[0]), f2bf(r.v[1])), pack2(f2bf(r.v[2]), f2bf(r.v[3])));
-  else p[0] = f2bf(r.v[0]);
-}
 
 template <int V>
 __global__ void __launch_bounds__(256) rms_step_kernel(const RmsStep a) {
@@ -321,7 +274,51 @@ __global__ void __launch_bounds__(256) group_norm_step_kernel(const GroupNormSte
   }
 }
 
+template <int V>
+__global__ void __launch_bounds__(256) norm_gate_kernel(const NormGate a) {
+  extern __shared__ __align__(16) float row[];  // [width], then [groups] scales
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_trigger();
+  const size_t r = blockIdx.x;
+  const int W = a.width, gs = W / a.groups, t0 = threadIdx.x * V, step = blockDim.x * V;
+  float* scale = row + W;
+  for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_f32<V>(a.v + r * a.ldv + i));
+  __syncthreads();
+  group_rstd(row, W, a.groups, a.eps, red, scale);
+  for (int i = t0; i < W; i += step) {
+    Pack<V> x = ld_f32<V>(row + i), w;
+    const Pack<V> g = a.g_bf ? ld_bf16<V>(a.g_bf + r * a.ldg_bf + i) : ld_f32<V>(a.g + r * a.ldg + i);
+    if (a.w) w = ld_bf16<V>(a.w + i);
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+      const float sg = 1.0f / (1.0f + expf(-g.v[u]));
+      float y = x.v[u] * scale[(i + u) / gs];
+      if (a.w) y *= w.v[u];
+      x.v[u] = y * (a.act == 1 ? sg : g.v[u] * sg);
+    }
+    if (a.out) st_f32<V>(a.out + r * a.ldo + i, x);
+    if (a.out_bf) st_bf16<V>(a.out_bf + r * a.ldo_bf + i, x);
+  }
+}
+
 }  // namespace
+
+cudaError_t launch_norm_gate(const NormGate& a, cudaStream_t st) {
+  if (a.n <= 0) return cudaSuccess;
+  if (a.width <= 0 || a.groups <= 0 || a.width % a.groups || !a.v || !(a.g || a.g_bf) || !(a.out || a.out_bf)) return cudaErrorInvalidValue;
+  const size_t smem = ((size_t)a.width + a.groups) * sizeof(float);
+  auto al = [](const void* p, size_t b) { return (reinterpret_cast<uintptr_t>(p) & (b - 1)) == 0; };
+  const bool vec = a.width % 4 == 0 && a.ldv % 4 == 0 && a.ldg % 4 == 0 && a.ldg_bf % 4 == 0 && a.ldo % 4 == 0 && a.ldo_bf % 4 == 0 && al(a.v, 16) &&
+                   al(a.g, 16) && al(a.g_bf, 8) && al(a.w, 8) && al(a.out, 16) && al(a.out_bf, 8);
+  auto* kern = vec ? norm_gate_kernel<4> : norm_gate_kernel<1>;
+  if (smem > 48 * 1024) {
+    if (smem > 200 * 1024) return cudaErrorInvalidValue;
+    cudaError_t r = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (r != cudaSuccess) return r;
+  }
+  return launch_k(kern, dim3(a.n), dim3(256), smem, st, a);
+}
 
 cudaError_t launch_group_norm_step(const GroupNormStep& a, cudaStream_t st) {
   if (a.n <= 0) return cudaSuccess;
