@@ -520,6 +520,38 @@ def dedunex_macs_per_token(cfg):
     return mac
 
 
+def gebadra_config(z, vocab=32000):
+    """four layers: window attention with pooled blocks and mixed heads beside retention, lightning attention, the same
+    lightning weights again, a second parallel layer; gated feed-forwards of the compared Qwen model's width"""
+    W = z["width"]
+    ff = {"ff": z["top"] * z["ff"] + z["sff"], "kind": "dense"}
+
+    def decay(n):
+        return [1.0 - 2.0 ** (-1.0 - 6.0 * i / max(1, n - 1)) for i in range(n)]
+    left = {"dim": 64, "heads": W // 64, "kv_heads": 4, "mask": {"pool": 16, "size": z["window"]}, "scale": 0.125, "vdim": 64,
+            "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 2.0}}}
+    par = {"left": left, "right": {"decay": decay(W // 128), "dim": 64, "heads": W // 128, "vdim": 128}}
+    lig = {"decay": decay(W // 64), "dim": 64, "heads": W // 64, "vdim": 64}
+    layers = [{"type": "parallel", "mixer": par, "mlp": ff}, {"type": "lightning", "mixer": lig, "mlp": ff},
+              {"type": "lightning", "mixer": lig, "mlp": ff, "weights_of": 1}, {"type": "parallel", "mixer": par, "mlp": ff}]
+    return {"architecture": "Gebadra", "layers": layers, "norm": {"eps": 1e-6}, "streams": 4, "vocab": vocab, "width": W}
+
+
+def gebadra_macs_per_token(cfg):
+    """multiply-adds of the projections of one token (attention scores and the recurrences not counted)"""
+    W, mac = cfg["width"], 0
+    for ly in cfg["layers"]:
+        mx = ly["mixer"]
+        lin = mx if ly["type"] == "lightning" else mx["right"]
+        mac += W * lin["heads"] * (2 * lin["dim"] + 3 * lin["vdim"])
+        if ly["type"] == "parallel":
+            lf = mx["left"]
+            mac += W * (lf["heads"] * lf["dim"] + lf["kv_heads"] * (lf["dim"] + lf["vdim"]) + lf["heads"] * lf["vdim"])
+        if ly.get("mlp"):
+            mac += 3 * W * ly["mlp"]["ff"]
+    return mac
+
+
 def run_family_compare(args):
     import numpy as np
     import torch
@@ -600,7 +632,7 @@ def run_family_compare(args):
                                   head_dim=128, vocab=vocab), context=8192)
         pages = (ctx + 64 + 15) // 16 * 9 + (T + 15) // 16 + 8
         rec = {}
-        if args.family in ("fosavik", "dedunex"):
+        if args.family in ("fosavik", "dedunex", "gebadra"):
             fv = fosavik_config(z, vocab)
             fv_cfg = json.dumps(fv)
             rec["fosavik"] = measure(lambda rows, seqs: q.Engine(config_json=fv_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
@@ -609,6 +641,11 @@ def run_family_compare(args):
             dd = dedunex_config(z, vocab)
             dd_cfg = json.dumps(dd)
             rec["dedunex"] = measure(lambda rows, seqs: q.Engine(config_json=dd_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
+                                                                 max_seqs=seqs, max_batch_tokens=rows, context=8192), vocab, False)
+        if args.family == "gebadra":
+            gb = gebadra_config(z, vocab)
+            gb_cfg = json.dumps(gb)
+            rec["gebadra"] = measure(lambda rows, seqs: q.Engine(config_json=gb_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
                                                                  max_seqs=seqs, max_batch_tokens=rows, context=8192), vocab, False)
         if args.family == "ditenex":
             dx = ditenex_config(z, vocab)
@@ -632,7 +669,10 @@ def run_family_compare(args):
         if args.family == "dedunex":
             rec["macs_per_token"]["dedunex"] = dedunex_macs_per_token(dd)
             fams.append(("dedunex", rec["macs_per_token"]["dedunex"]))
-        if args.family in ("fosavik", "dedunex"):
+        if args.family == "gebadra":
+            rec["macs_per_token"]["gebadra"] = gebadra_macs_per_token(gb)
+            fams.append(("gebadra", rec["macs_per_token"]["gebadra"]))
+        if args.family in ("fosavik", "dedunex", "gebadra"):
             rec["macs_per_token"]["fosavik"] = fosavik_macs_per_token(fv)
             fams.append(("fosavik", rec["macs_per_token"]["fosavik"]))
         if args.family == "ditenex":
@@ -664,9 +704,9 @@ def main():
     ap.add_argument("--family-compare", action="store_true",
                     help="side measurement (not the contract line): prefill / decode throughput of the Nogatar family beside the "
                          "Qwen family at equal size, with per-kernel-class device times")
-    ap.add_argument("--family", default="nogatar", choices=["nogatar", "fosavik", "ditenex", "dedunex"],
+    ap.add_argument("--family", default="nogatar", choices=["nogatar", "fosavik", "ditenex", "dedunex", "gebadra"],
                     help="with --family-compare: which fp32-stream family is measured beside the Qwen family (fosavik and ditenex also run "
-                         "nogatar; dedunex also runs fosavik and nogatar, the families whose mixers are closest to its own)")
+                         "nogatar; dedunex and gebadra also run fosavik, the family whose mixers are closest to their own)")
     ap.add_argument("--family-size", default="", help="one of " + ", ".join(FAMILY_SIZES) + " (default: all)")
     ap.add_argument("--family-tokens", type=int, default=2048)
     ap.add_argument("--family-ctx", type=int, default=1024)
