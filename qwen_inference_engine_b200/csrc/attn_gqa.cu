@@ -11,6 +11,7 @@
 #include <algorithm>
 
 #include "fosavik.h"
+#include "kv_rows.cuh"
 #include "launch.h"
 #include "pack.cuh"
 
@@ -20,22 +21,6 @@ namespace {
 constexpr int ATK = 32;       // keys per tile
 constexpr int ATHREADS = 128;
 constexpr int AMAXACC = 16;   // accumulators per thread: query vectors x value columns of a CTA <= 2048
-
-__device__ __forceinline__ const char* kv_row_ptr(const KvRowCache& c, const int* block_table, int max_pages, int slot, int pos) {
-  const int page = block_table[(size_t)slot * max_pages + pos / c.page_size];
-  const size_t off = (size_t)page * c.page_elems + c.layer_off + (size_t)(pos % c.page_size) * (c.kw + c.vw);
-  return static_cast<const char*>(c.pool) + off * c.elt_bytes;
-}
-
-// pooled row of block b (KvRowCache)
-__device__ __forceinline__ const char* kv_pool_ptr(const KvRowCache& c, const int* block_table, int max_pages, int slot, int b) {
-  const int pi = (b * c.block + c.block - 1) / c.page_size;
-  const int page = block_table[(size_t)slot * max_pages + pi];
-  const size_t off = (size_t)page * c.page_elems + c.pool_off + (size_t)(b - pi * c.page_size / c.block) * (c.kw + c.vw);
-  return static_cast<const char*>(c.pool) + off * c.elt_bytes;
-}
-// blocks that lie wholly before the window of position pos: (b + 1) * pool - 1 <= pos - window
-__host__ __device__ __forceinline__ int pooled_seen(int pos, int window, int pool) { return pool > 0 && pos >= window ? (pos - window + 1) / pool : 0; }
 
 __device__ __forceinline__ void store_elt(const KvRowCache& c, char* row, int i, float v) {
   if (c.elt_bytes == 4) reinterpret_cast<float*>(row)[i] = v;
@@ -133,13 +118,16 @@ __device__ __forceinline__ void pool_block(const KvRowCache& c, const int* block
     store_elt(c, dst, i, s * inv);
   }
 }
-// one CTA per row; only the rows at a block's end do something
+// one CTA per POOL_ROWS rows; only the rows at a block's end do something
+constexpr int POOL_ROWS = 16;
 __global__ void __launch_bounds__(128) kv_pool_rows_kernel(const KvRowCache c, const int* __restrict__ pos, const int* __restrict__ slot,
-                                                           const int* __restrict__ block_table, int max_pages) {
+                                                           const int* __restrict__ block_table, int max_pages, int n) {
   pdl_wait();
   pdl_trigger();
-  const int r = blockIdx.x, p = pos[r];
-  if ((p + 1) % c.block == 0) pool_block(c, block_table, max_pages, slot[r], p / c.block);
+  for (int r = blockIdx.x * POOL_ROWS; r < min(n, (int)(blockIdx.x + 1) * POOL_ROWS); ++r) {
+    const int p = pos[r];
+    if ((p + 1) % c.block == 0) pool_block(c, block_table, max_pages, slot[r], p / c.block);
+  }
 }
 
 // The store with the unit norm over the whole projection: one CTA per row, both reductions at once, then the rotation of
@@ -156,10 +144,26 @@ __global__ void __launch_bounds__(256) kv_store_whole_kernel(const KvStoreArgs a
   const float *kf = a.k + (size_t)r * a.ldk, *vf = a.v + (size_t)r * a.ldv;
   auto getq = [&](int i) { return (bf ? bf2f(qb[i]) : qf[i]) + (a.q_bias ? bf2f(a.q_bias[i]) : 0.f); };
   auto getk = [&](int i) { return (bf ? bf2f(kb[i]) : kf[i]) + (a.k_bias ? bf2f(a.k_bias[i]) : 0.f); };
+  // neighbouring pairs, bf16 sources: a thread moves a pair per access (pair j holds elements 2j and 2j + 1, and d is even)
+  const bool pairs = bf && !a.rope.half_layout && d % 2 == 0 && a.ld_bf % 2 == 0 && a.ldq % 2 == 0 && !a.q_bias && !a.k_bias &&
+                     ((reinterpret_cast<uintptr_t>(a.q_bf) | reinterpret_cast<uintptr_t>(a.k_bf)) & 3) == 0 && (a.c.kw + vw) % 2 == 0 && a.c.layer_off % 2 == 0 &&
+                     a.c.page_elems % 2 == 0;
   float sq = 0.f, sk = 0.f;
-  if (a.q_norm)
+  if (pairs) {
+    if (a.q_norm)
+      for (int j = tid; j < nq / 2; j += blockDim.x) {
+        const uint32_t x = reinterpret_cast<const uint32_t*>(qb)[j];
+        sq = fmaf(lo2f(x), lo2f(x), fmaf(hi2f(x), hi2f(x), sq));
+      }
+    if (a.k_norm)
+      for (int j = tid; j < kw / 2; j += blockDim.x) {
+        const uint32_t x = reinterpret_cast<const uint32_t*>(kb)[j];
+        sk = fmaf(lo2f(x), lo2f(x), fmaf(hi2f(x), hi2f(x), sk));
+      }
+  }
+  if (a.q_norm && !pairs)
     for (int i = tid; i < nq; i += blockDim.x) sq = fmaf(getq(i), getq(i), sq);
-  if (a.k_norm)
+  if (a.k_norm && !pairs)
     for (int i = tid; i < kw; i += blockDim.x) sk = fmaf(getk(i), getk(i), sk);
   const float2 s2 = block_sum2_r(sq, sk, red);
   const float rq = a.q_norm ? 1.0f / sqrtf(s2.x / (float)nq + a.eps) : 1.f, rk = a.k_norm ? 1.0f / sqrtf(s2.y / (float)kw + a.eps) : 1.f;
@@ -182,8 +186,25 @@ __global__ void __launch_bounds__(256) kv_store_whole_kernel(const KvStoreArgs a
       }
   };
   char* row = const_cast<char*>(kv_row_ptr(a.c, a.block_table, a.max_pages, slot, p));
-  emit(kw, getk, a.k_norm, rk, [&](int i, float x) { store_elt(a.c, row, i, x); });
-  if (nq) emit(nq, getq, a.q_norm, rq, [&](int i, float x) { qf[i] = x; });
+  if (pairs) {
+    auto turn = [&](uint32_t x, const bf16* w, float rstd, int j) {
+      float u = lo2f(x), v = hi2f(x);
+      if (w) u *= rstd * bf2f(w[2 * j]), v *= rstd * bf2f(w[2 * j + 1]);
+      const int e = j % (d / 2);
+      if (e >= half) return make_float2(u, v);
+      const float c = ct[e], s = sn[e];
+      return make_float2(u * c - v * s, v * c + u * s);
+    };
+    for (int j = tid; j < kw / 2; j += blockDim.x) {
+      const float2 y = turn(reinterpret_cast<const uint32_t*>(kb)[j], a.k_norm, rk, j);
+      if (a.c.elt_bytes == 2) reinterpret_cast<uint32_t*>(row)[j] = pack2(f2bf(y.x), f2bf(y.y));
+      else reinterpret_cast<float2*>(row)[j] = y;
+    }
+    for (int j = tid; j < nq / 2; j += blockDim.x)
+      reinterpret_cast<float2*>(qf)[j] = turn(reinterpret_cast<const uint32_t*>(qb)[j], a.q_norm, rq, j);
+  }
+  if (!pairs) emit(kw, getk, a.k_norm, rk, [&](int i, float x) { store_elt(a.c, row, i, x); });
+  if (nq && !pairs) emit(nq, getq, a.q_norm, rq, [&](int i, float x) { qf[i] = x; });
   if (bf && a.c.elt_bytes == 2 && !a.v_bias) {
     for (int i = tid; i < vw; i += blockDim.x) reinterpret_cast<bf16*>(row)[kw + i] = vb[i];
   } else {
@@ -851,7 +872,7 @@ cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
 
 cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st) {
   if (n <= 0 || c.block <= 0) return cudaSuccess;
-  return launch_k(kv_pool_rows_kernel, dim3(n), dim3(128), 0, st, c, pos, slot, block_table, max_pages);
+  return launch_k(kv_pool_rows_kernel, dim3((n + POOL_ROWS - 1) / POOL_ROWS), dim3(128), 0, st, c, pos, slot, block_table, max_pages, n);
 }
 
 static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStream_t st) {
@@ -874,6 +895,13 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
   if (a.c.block > 0 && (a.window <= 0 || a.slopes || a.shared_keys || a.maps != 1)) return cudaErrorInvalidValue;
   const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim;
   if (a.talk && gqa_ws_floats(a.n, a.heads, 1, vcols) > a.ws_floats) return cudaErrorInvalidValue;
+  // mixed heads over a bf16 cache: the tcgen05 kernel for prompt portions (QIE_ATTN_TC=0: the kernels below)
+  static const bool tc_on = [] { const char* v = getenv("QIE_ATTN_TC"); return !(v && v[0] == '0'); }();
+  if (tc_on && gqa_talk_tc_fits(a)) {
+    if (n_launches) *n_launches = 2;
+    cudaError_t r = launch_gqa_talk_tc(a, st);
+    return r != cudaSuccess ? r : launch_talk_finish(a, 1, st);
+  }
   // prompt portions over a bf16 cache: the tensor-core kernel (one launch, no workspace); QIE_ATTN_MMA=0 keeps the per-row kernel (A/B)
   static const bool mma_on = [] { const char* v = getenv("QIE_ATTN_MMA"); return !(v && v[0] == '0'); }();
   if (mma_on && a.seg_start && a.c.elt_bytes == 2 && a.n >= 64 && a.dim <= 128 && (a.talk || a.vdim <= 128) && a.maps <= 2 && a.heads % a.kv_heads == 0 &&

@@ -1,0 +1,399 @@
+// attn_gqa_tc.cu -- prompt attention over paged bf16 key/value rows on the 5th-gen tensor cores (tcgen05 + TMEM), for grouped
+// queries whose softmax weights are mixed over the heads (GqaAttnArgs::talk), a sliding window or a causal mask, and pooled
+// rows.  Mixing after the softmax is linear, so every head attends to the values of ALL kv heads -- one product with up to
+// 256 value columns, which is what the tensor cores are good at -- and gqa_talk_finish_kernel mixes the results.
+//
+// A CTA owns 128 consecutive rows of one segment, one query head and one chunk of value columns, and walks tiles of 64 keys: first
+// the tiles of pooled rows that some row sees, then the tokens from the first window's lower edge on.  12 warps:
+//   warps 9-11  copy the tile's key and value rows into the swizzled operand layout (cp.async, ring of stages)
+//   warp 8      issues the products: S = Q K^T (128 x 64, two TMEM buffers, one tile ahead of the softmax) and O += P V (TMEM)
+//   warps 0-7   softmax, two threads per row: S from TMEM, mask, reference maximum, weights as bf16 hi + lo pairs into shared
+//               memory (two buffers, two products per tile, so a weight keeps ~16 bits)
+// O stays in TMEM over all tiles.  Instead of scaling it whenever a row's maximum grows, a row keeps its reference maximum until a
+// score exceeds it by RESCALE (weights then stay below 2^RESCALE); only then the warp that owns the row scales its part of O.
+// Every wait has a limit; when one runs out the CTA finishes without waiting and marks its results as not a number.
+#include <algorithm>
+
+#include "common.cuh"
+#include "fosavik.h"
+#include "kernels.h"
+#include "kv_rows.cuh"
+#include "launch.h"
+
+namespace qie {
+namespace {
+
+constexpr int TQ = 128, TK = 64;
+constexpr int NSOFT = 256, NLOAD = 96, NTHR = NSOFT + 32 + NLOAD;
+constexpr int LROWS = NLOAD / 8, LPASS = (TK + LROWS - 1) / LROWS;  // rows a pass of the copying threads covers
+constexpr int KBLK = TK * 128;   // [64 keys][64 columns] bf16, 8-row swizzle atoms: 8 KiB
+constexpr int QBLK = TQ * 128;   // [128 rows][64 columns]: 16 KiB
+constexpr float RESCALE = 8.0f;  // in powers of two
+
+__device__ __forceinline__ void mbar_init_tc(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count)); }
+__device__ __forceinline__ void mbar_arrive_tc(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
+// waits for the phase of this parity; after the limit it sets *dead, and from then on no wait of the CTA waits
+__device__ __forceinline__ void mbar_wait_tc(uint32_t bar, uint32_t parity, volatile int* dead) {
+  for (int i = 0; i < 2000000; ++i) {
+    uint32_t done = 0;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done)
+        : "r"(bar), "r"(parity)
+        : "memory");
+    if (done) return;
+    if ((i & 63) == 63 && *dead) return;
+  }
+  *dead = 1;
+}
+__device__ __forceinline__ void umma_tc(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(acc)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_tc(uint32_t bar) {
+  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+__device__ __forceinline__ void tmem_ld32_tc(uint32_t taddr, uint32_t (&r)[32]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
+      "%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
+        "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
+        "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+      : "r"(taddr));
+}
+__device__ __forceinline__ void tmem_st32_tc(uint32_t taddr, const uint32_t (&r)[32]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%32], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
+      "%23,%24,%25,%26,%27,%28,%29,%30,%31};"
+      ::"r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
+      "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]),
+      "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]), "r"(taddr)
+      : "memory");
+}
+// K-major operand, SWIZZLE_128B, 8-row atoms 1024 bytes apart
+__device__ __forceinline__ uint64_t desc_k_tc(uint32_t smem_addr) {
+  return (uint64_t)((smem_addr >> 4) & 0x3FFF) | (uint64_t)1 << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+// MN-major operand (values as stored: [key][column]), SWIZZLE_128B: blocks of 64 columns KBLK bytes apart, groups of 8 keys 1024
+__device__ __forceinline__ uint64_t desc_mn_tc(uint32_t smem_addr) {
+  return (uint64_t)((smem_addr >> 4) & 0x3FFF) | (uint64_t)(KBLK >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+// D = F32, A = B = BF16, N >> 3 at [17,23), M >> 4 at [24,29), bit 16: B is MN-major
+__device__ __forceinline__ uint32_t idesc_tc(int m, int n, bool b_mn) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
+}
+__device__ __forceinline__ float ex2_tc(float x) {  // 2^x; 2^(-inf) = 0
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// byte offset of 16-byte chunk ch (0..7) of row r in a block of 64 columns
+__device__ __forceinline__ uint32_t blk_off(int r, int ch) { return (uint32_t)(r * 128 + ((ch ^ (r & 7)) << 4)); }
+
+struct TcLayout {  // byte offsets from the 1024-aligned base
+  int dblk, vblk, nst, q, p, st, stage, bar, total;
+};
+__host__ __device__ inline TcLayout tc_layout(int dblk, int vblk, int nst) {
+  TcLayout l;
+  l.dblk = dblk, l.vblk = vblk, l.nst = nst;
+  l.q = 0;
+  l.p = l.q + dblk * QBLK;        // P [buffer 2][hi, lo]
+  l.st = l.p + 4 * QBLK;          // stages: K blocks | V blocks
+  l.stage = (dblk + vblk) * KBLK;
+  l.bar = l.st + nst * l.stage;   // mbarriers, flags, row maxima
+  l.total = l.bar + 256 + 4 * TQ * 4;
+  return l;
+}
+
+__global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc) {
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
+  __shared__ int info[4];  // first row, rows, slot
+  __shared__ int dead_s;
+  pdl_wait();
+  pdl_trigger();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    int left = blockIdx.y, found = 0;
+    for (int s = 0; s < a.n_seg && !found; ++s) {
+      const int r0 = a.seg_start[s], len = a.seg_start[s + 1] - r0, nt = (len + TQ - 1) / TQ;
+      if (left < nt) info[0] = r0 + left * TQ, info[1] = min(TQ, len - left * TQ), info[2] = a.seg_slot[s], found = 1;
+      left -= nt;
+    }
+    if (!found) info[1] = 0;
+    dead_s = 0;
+  }
+  __syncthreads();
+  const int row0 = info[0], nrows = info[1], slot = info[2];
+  if (nrows == 0) return;
+  volatile int* dead = &dead_s;
+  const TcLayout L = tc_layout(dblk, vblk, nst);
+  const uint32_t s0 = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  unsigned char* sg = smem_raw + (s0 - smem_u32(smem_raw));
+  const uint32_t b0 = s0 + L.bar;
+  const uint32_t bar_full = b0, bar_empty = b0 + 32, bar_s = b0 + 64, bar_p = b0 + 80, bar_o = b0 + 96, tslot = b0 + 112;
+  float* xmax = reinterpret_cast<float*>(sg + L.bar + 256);  // [tile parity][half][row]; the sums use the first half at the end
+  const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), dim = a.dim;
+  const int vcols = a.kv_heads * a.vdim, col0 = blockIdx.z * vc, nv = min(vc, vcols - col0);
+  const int pos0 = a.pos[row0], pmax = pos0 + nrows - 1;
+  const int lo_min = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int nbmax = a.c.block > 0 ? pooled_seen(pmax, a.window, a.c.block) : 0, npt = (nbmax + TK - 1) / TK;
+  const int tt0 = lo_min / TK, nt = npt + pmax / TK - tt0 + 1;  // tiles: npt of pooled rows, then tokens from tile tt0 on
+  if (tid == 0) {
+    for (int i = 0; i < nst; ++i) mbar_init_tc(bar_full + 8 * i, NLOAD), mbar_init_tc(bar_empty + 8 * i, 1);
+    for (int i = 0; i < 2; ++i) mbar_init_tc(bar_s + 8 * i, 1), mbar_init_tc(bar_p + 8 * i, NSOFT), mbar_init_tc(bar_o + 8 * i, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 8) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tslot), "r"(512u) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  // Q rows as bf16, zeros beyond the head size and the last row
+  for (int i = tid; i < TQ * dblk * 8; i += NTHR) {
+    const int r = i / (dblk * 8), c = (i - r * dblk * 8) * 8;
+    uint32_t w[4] = {0u, 0u, 0u, 0u};
+    if (r < nrows) {
+      const float* q = a.q + (size_t)(row0 + r) * a.ldq + (size_t)h * dim + c;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + 2 * e < dim) w[e] = pack2(f2bf(q[2 * e]), f2bf(q[2 * e + 1]));  // dim is a multiple of 8
+    }
+    *reinterpret_cast<uint4*>(sg + L.q + (c >> 6) * QBLK + blk_off(r, (c >> 3) & 7)) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+  uint32_t tmem;
+  asm volatile("ld.shared.b32 %0, [%1];" : "=r"(tmem) : "r"(tslot));
+  const uint32_t t_o = tmem + 128;  // S: columns 0..127 (two buffers), O: 128 ..
+  const int vcp = vblk * 64;        // columns of O
+
+  if (warp >= 9) {
+    // ---- copies
+    const int lt = tid - (NSOFT + 32), ch = lt & 7, rr = lt >> 3;  // chunk of a 64-column block, rows rr + LROWS k
+    const size_t koff = (size_t)g * dim, voff = (size_t)a.c.kw + col0;
+    auto announce = [&](int t) {  // the copies of tile t are complete: visible to the tensor core
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      mbar_arrive_tc(bar_full + 8 * (t % nst));
+    };
+    for (int t = 0; t < nt; ++t) {
+      const int s = t % nst;
+      if (t > 0 && nst == 2) {  // the stage that this tile waits for is only given back behind the scores of the tile before
+        cp_async_wait<0>();
+        announce(t - 1);
+      }
+      if (t >= nst) mbar_wait_tc(bar_empty + 8 * s, (uint32_t)((t / nst - 1) & 1), dead);
+      const bf16* rowp[LPASS];
+#pragma unroll
+      for (int k = 0; k < LPASS; ++k) {
+        const int r = rr + LROWS * k;
+        const char* p = nullptr;
+        if (t < npt) {
+          if (r < TK && t * TK + r < nbmax) p = kv_pool_ptr(a.c, a.block_table, a.max_pages, slot, t * TK + r);
+        } else {
+          const int j = (tt0 + t - npt) * TK + r;
+          if (r < TK && j <= pmax) p = kv_row_ptr(a.c, a.block_table, a.max_pages, slot, j);
+        }
+        rowp[k] = reinterpret_cast<const bf16*>(p);
+      }
+      const uint32_t base = s0 + L.st + s * L.stage;
+      for (int b = 0; b < dblk + vblk; ++b) {
+        const bool isv = b >= dblk;
+        const int c = (isv ? b - dblk : b) * 64 + ch * 8;
+        const bool in = c < (isv ? nv : dim);
+#pragma unroll
+        for (int k = 0; k < LPASS; ++k) {
+          const int r = rr + LROWS * k;
+          if (r >= TK) break;
+          const uint32_t dst = base + b * KBLK + blk_off(r, ch);
+          if (in && rowp[k]) cp_async16(dst, rowp[k] + (isv ? voff : koff) + c);
+          else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0u) : "memory");
+        }
+      }
+      cp_async_commit();
+      if (t > 0 && nst > 2) {
+        cp_async_wait<1>();
+        announce(t - 1);
+      }
+    }
+    cp_async_wait<0>();
+    announce(nt - 1);
+  } else if (warp == 8) {
+    // ---- products
+    if (lane == 0) {
+      const uint32_t id_s = idesc_tc(TQ, TK, false), id_o = idesc_tc(TQ, vcp, true);
+      auto issue_s = [&](int t) {
+        const int s = t % nst;
+        mbar_wait_tc(bar_full + 8 * s, (uint32_t)((t / nst) & 1), dead);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        const uint32_t kb = s0 + L.st + s * L.stage;
+        for (int kk = 0; kk < dblk * 4; ++kk)
+          umma_tc(tmem + (uint32_t)((t & 1) * TK), desc_k_tc(s0 + L.q + (kk >> 2) * QBLK + (kk & 3) * 32), desc_k_tc(kb + (kk >> 2) * KBLK + (kk & 3) * 32),
+                  id_s, kk != 0);
+        umma_commit_tc(bar_s + 8 * (t & 1));
+      };
+      issue_s(0);
+      for (int t = 0; t < nt; ++t) {
+        if (t + 1 < nt) issue_s(t + 1);  // its buffer was read before the weights of tile t - 1 were announced
+        mbar_wait_tc(bar_p + 8 * (t & 1), (uint32_t)((t >> 1) & 1), dead);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        const uint32_t vb = s0 + L.st + (t % nst) * L.stage + dblk * KBLK, ph = s0 + L.p + (t & 1) * 2 * QBLK;
+        for (int part = 0; part < 2; ++part)  // hi, lo
+          for (int kk = 0; kk < TK / 16; ++kk)
+            umma_tc(t_o, desc_k_tc(ph + part * QBLK + kk * 32), desc_mn_tc(vb + kk * 16 * 128), id_o, t > 0 || part > 0 || kk > 0);
+        umma_commit_tc(bar_empty + 8 * (t % nst));
+        umma_commit_tc(bar_o + 8 * (t & 1));
+      }
+    }
+    __syncwarp();
+  } else {
+    // ---- softmax: row (TMEM lane), half of the tile's keys and of O's columns
+    const int row = (warp & 3) * 32 + lane, hf = warp >> 2;
+    const int my_pos = pos0 + row, my_lo = a.window > 0 ? my_pos - a.window + 1 : 0, my_seen = a.c.block > 0 ? pooled_seen(my_pos, a.window, a.c.block) : 0;
+    const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+    const float sl2 = a.scale * 1.4426950408889634f;
+    float m_ref = -INFINITY, l_run = 0.f;
+    for (int t = 0; t < nt; ++t) {
+      mbar_wait_tc(bar_s + 8 * (t & 1), (uint32_t)((t >> 1) & 1), dead);
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      uint32_t r[32];
+      tmem_ld32_tc(tmem + lane_addr + (uint32_t)((t & 1) * TK + 32 * hf), r);
+      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+      // visible keys of this thread: first .. last (relative to its 32)
+      int first, last;
+      if (t < npt) first = 0, last = my_seen - 1 - (t * TK + 32 * hf);
+      else first = my_lo - ((tt0 + t - npt) * TK + 32 * hf), last = my_pos - ((tt0 + t - npt) * TK + 32 * hf);
+      float mx = -INFINITY;
+      if (first > 0 || last < 31) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+          if (j < first || j > last) r[j] = 0xff800000u;  // -inf
+      }
+#pragma unroll
+      for (int j = 0; j < 32; ++j) mx = fmaxf(mx, __uint_as_float(r[j]));
+      float* xm = xmax + (t & 1) * 2 * TQ;
+      xm[hf * TQ + row] = mx;
+      asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp & 3)) : "memory");  // the two warps that share these 32 rows
+      mx = fmaxf(mx, xm[(hf ^ 1) * TQ + row]) * sl2;
+      const bool grow = mx > m_ref + RESCALE;
+      if (__any_sync(0xffffffffu, grow)) {
+        const float m_new = fmaxf(m_ref, mx), f = m_new > -INFINITY ? ex2_tc(m_ref - m_new) : 1.f;
+        m_ref = m_new, l_run *= f;
+        if (t > 0) {  // scale this thread's columns of O once the product of the tile before is in
+          mbar_wait_tc(bar_o + 8 * ((t - 1) & 1), (uint32_t)(((t - 1) >> 1) & 1), dead);
+          asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+          for (int c = hf * (vcp / 2); c < (hf + 1) * (vcp / 2); c += 32) {
+            uint32_t o[32];
+            tmem_ld32_tc(t_o + lane_addr + c, o);
+            asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+            for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * f);
+            tmem_st32_tc(t_o + lane_addr + c, o);
+          }
+          asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+        }
+      }
+      const float nm = m_ref > -INFINITY ? -m_ref : 0.f;
+      if (t >= 2) mbar_wait_tc(bar_o + 8 * (t & 1), (uint32_t)(((t >> 1) - 1) & 1), dead);  // the product that read this P buffer
+      const uint32_t pd = s0 + L.p + (t & 1) * 2 * QBLK;
+      float rs = 0.f;
+#pragma unroll
+      for (int q8 = 0; q8 < 4; ++q8) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float e0 = ex2_tc(fmaf(__uint_as_float(r[q8 * 8 + 2 * e]), sl2, nm)), e1 = ex2_tc(fmaf(__uint_as_float(r[q8 * 8 + 2 * e + 1]), sl2, nm));
+          rs += e0 + e1;
+          const bf16 h0 = f2bf(e0), h1 = f2bf(e1);
+          hi[e] = pack2(h0, h1);
+          lo[e] = pack2(f2bf(e0 - bf2f(h0)), f2bf(e1 - bf2f(h1)));
+        }
+        const uint32_t o = blk_off(row, 4 * hf + q8);
+        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + o), "r"(hi[0]), "r"(hi[1]), "r"(hi[2]), "r"(hi[3]) : "memory");
+        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + QBLK + o), "r"(lo[0]), "r"(lo[1]), "r"(lo[2]), "r"(lo[3]) : "memory");
+      }
+      l_run += rs;
+      asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      mbar_arrive_tc(bar_p + 8 * (t & 1));
+    }
+    mbar_wait_tc(bar_o + 8 * ((nt - 1) & 1), (uint32_t)(((nt - 1) >> 1) & 1), dead);
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    float* xs = xmax + (nt & 1) * 2 * TQ;  // the buffer that the last tile did not use
+    xs[hf * TQ + row] = l_run;
+    asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp & 3)) : "memory");
+    const float l = l_run + xs[(hf ^ 1) * TQ + row];
+    const float inv = *dead ? __int_as_float(0x7fffffff) : (l > 0.f ? 1.0f / l : 0.f);
+    float* rec = a.ws + ((size_t)(row0 + row) * a.heads + h) * (vcols + 2);
+    if (row < nrows && hf == 0 && blockIdx.z == 0) rec[0] = 0.f, rec[1] = 1.f;
+    for (int c = hf * (vcp / 2); c < (hf + 1) * (vcp / 2); c += 32) {
+      uint32_t o[32];
+      tmem_ld32_tc(t_o + lane_addr + c, o);
+      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+      if (row < nrows) {
+        float* d = rec + 2 + col0 + c;
+        if (c + 32 <= nv) {  // records are 8-byte aligned
+#pragma unroll
+          for (int j = 0; j < 32; j += 2) *reinterpret_cast<float2*>(d + j) = make_float2(__uint_as_float(o[j]) * inv, __uint_as_float(o[j + 1]) * inv);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            if (c + j < nv) d[j] = __uint_as_float(o[j]) * inv;
+        }
+      }
+    }
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  if (warp == 8) {
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+  }
+}
+
+constexpr int SMEM_MAX = 226 * 1024;
+struct TcPlan {
+  int dblk, vblk, nst, vc, nvc;
+  size_t smem;
+};
+TcPlan tc_plan(const GqaAttnArgs& a) {
+  TcPlan p;
+  const int vcols = a.kv_heads * a.vdim;
+  p.dblk = (a.dim + 63) / 64;
+  p.nvc = (vcols + 255) / 256;
+  p.vc = ((vcols + p.nvc - 1) / p.nvc + 7) / 8 * 8;
+  p.vblk = (p.vc + 63) / 64;
+  p.nst = tc_layout(p.dblk, p.vblk, 3).total + 1024 <= SMEM_MAX ? 3 : 2;
+  p.smem = (size_t)tc_layout(p.dblk, p.vblk, p.nst).total + 1024;
+  return p;
+}
+
+}  // namespace
+
+bool gqa_talk_tc_fits(const GqaAttnArgs& a) {
+  return a.talk && a.c.elt_bytes == 2 && a.seg_start && a.n >= 128 && a.n / a.n_seg >= 64 && a.dim <= 128 && a.dim % 8 == 0 && (a.kv_heads * a.vdim) % 8 == 0 &&
+         a.maps == 1 && a.scale > 0.f && a.keep_first == 0 && a.softcap == 0.f && !a.slopes && !a.shared_keys && a.c.page_elems % 8 == 0 && a.c.layer_off % 8 == 0 &&
+         (a.c.kw + a.c.vw) % 8 == 0 && a.c.kw % 8 == 0 && (!a.c.block || (a.c.pool_off % 8 == 0 && a.window > 0)) &&
+         (reinterpret_cast<uintptr_t>(a.c.pool) & 15) == 0 && a.heads <= 65535;
+}
+
+cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st) {
+  const TcPlan p = tc_plan(a);
+  static PerDeviceOnce once;
+  if (once.need()) {
+    cudaError_t r = cudaFuncSetAttribute(gqa_talk_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
+    if (r != cudaSuccess) return r;
+    once.done();
+  }
+  return launch_k(gqa_talk_tc_kernel, dim3(a.heads, a.n / TQ + a.n_seg, p.nvc), dim3(NTHR), p.smem, st, a, p.dblk, p.vblk, p.nst, p.vc);
+}
+
+}  // namespace qie

@@ -184,6 +184,10 @@ struct GqaAttnArgs {
 // (vdim: with `talk` the value elements of all kv heads together)
 inline size_t gqa_ws_floats(int n, int heads, int maps, int vdim) { return (size_t)n * heads * maps * (vdim + 2); }
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches = nullptr);
+// the tcgen05 form of a prompt portion's attention with `talk` (attn_gqa_tc.cu), without the mix of the heads: the normalised result
+// of every head over the values of all kv heads goes to its workspace record (max 0, sum 1); launch_gqa_attention picks it
+bool gqa_talk_tc_fits(const GqaAttnArgs& a);
+cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st);
 
 // ---------------------------------------------------------------- short convolution and recurrences (recurrent.cu)
 // Causal per-channel convolution over the rows of each segment: out[t, c] = act(b[c] + sum_i w[c, i] * in(t - (taps-1-i), c)),
