@@ -105,22 +105,42 @@ __global__ void __launch_bounds__(128) kv_store_rows_kernel(const KvStoreArgs a)
 }
 
 // the mean of a block's rows -> its pooled row, by the threads of one CTA
+constexpr int POOL_SRC = 32;  // rows whose addresses are worked out at a time
 __device__ __forceinline__ void pool_block(const KvRowCache& c, const int* block_table, int max_pages, int slot, int b) {
+  __shared__ const char* src[POOL_SRC];
   char* dst = const_cast<char*>(kv_pool_ptr(c, block_table, max_pages, slot, b));
   const float inv = 1.0f / (float)c.block;
-  for (int i = threadIdx.x; i < c.kw + c.vw; i += blockDim.x) {
-    float s = 0.f;
+  const int w = c.kw + c.vw;
+  const bool pairs = c.elt_bytes == 2 && w % 2 == 0 && c.layer_off % 2 == 0 && c.pool_off % 2 == 0 && c.page_elems % 2 == 0;
+  const int ne = pairs ? w / 2 : w;  // what a thread handles: a pair of bf16 elements, else one element
+  for (int e0 = 0; e0 < ne; e0 += blockDim.x) {
+    const int i = e0 + threadIdx.x;
+    float s0 = 0.f, s1 = 0.f;
+    for (int t0 = 0; t0 < c.block; t0 += POOL_SRC) {
+      const int nt = min(POOL_SRC, c.block - t0);
+      __syncthreads();
+      if (threadIdx.x < nt) src[threadIdx.x] = kv_row_ptr(c, block_table, max_pages, slot, b * c.block + t0 + threadIdx.x);
+      __syncthreads();
+      if (i >= ne) continue;
+      if (pairs) {
+#pragma unroll 16
+        for (int t = 0; t < nt; ++t) {
+          const uint32_t v = reinterpret_cast<const uint32_t*>(src[t])[i];
+          s0 += lo2f(v), s1 += hi2f(v);
+        }
+      } else {
 #pragma unroll 4
-    for (int t = 0; t < c.block; ++t) {
-      const char* row = kv_row_ptr(c, block_table, max_pages, slot, b * c.block + t);
-      s += c.elt_bytes == 4 ? reinterpret_cast<const float*>(row)[i] : bf2f(reinterpret_cast<const bf16*>(row)[i]);
+        for (int t = 0; t < nt; ++t) s0 += c.elt_bytes == 4 ? reinterpret_cast<const float*>(src[t])[i] : bf2f(reinterpret_cast<const bf16*>(src[t])[i]);
+      }
     }
-    store_elt(c, dst, i, s * inv);
+    if (i >= ne) continue;
+    if (pairs) reinterpret_cast<uint32_t*>(dst)[i] = pack2f(s0 * inv, s1 * inv);
+    else store_elt(c, dst, i, s0 * inv);
   }
 }
 // one CTA per POOL_ROWS rows; only the rows at a block's end do something
 constexpr int POOL_ROWS = 16;
-__global__ void __launch_bounds__(128) kv_pool_rows_kernel(const KvRowCache c, const int* __restrict__ pos, const int* __restrict__ slot,
+__global__ void __launch_bounds__(256) kv_pool_rows_kernel(const KvRowCache c, const int* __restrict__ pos, const int* __restrict__ slot,
                                                            const int* __restrict__ block_table, int max_pages, int n) {
   pdl_wait();
   pdl_trigger();
@@ -213,6 +233,75 @@ __global__ void __launch_bounds__(256) kv_store_whole_kernel(const KvStoreArgs a
   if (a.c.block > 0 && a.one_each && (p + 1) % a.c.block == 0) {
     __syncthreads();  // this row's own elements come from the whole CTA
     pool_block(a.c, a.block_table, a.max_pages, slot, p / a.c.block);
+  }
+}
+
+// The same for rows of bf16 sources whose parts are whole 16-byte pieces: a warp per row, the row's queries and keys stay in
+// registers between the reduction and the rotation (neighbouring pairs, a piece holds four of them).  NQ, NK: pieces per lane.
+template <int NQ, int NK>
+__global__ void __launch_bounds__(256) kv_store_whole_warp_kernel(const KvStoreArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= a.n) return;
+  const int p = a.pos[r], d = a.norm_dim, dims = a.rope.dims, half = dims / 2;
+  const int q8 = a.q_heads * d / 8, k8 = a.c.kw / 8, v8 = a.c.vw / 8;
+  const uint4* qb = reinterpret_cast<const uint4*>(a.q_bf + (size_t)r * a.ld_bf);
+  const uint4* kb = reinterpret_cast<const uint4*>(a.k_bf + (size_t)r * a.ld_bf);
+  const uint4* vb = reinterpret_cast<const uint4*>(a.v_bf + (size_t)r * a.ld_bf);
+  bf16* row = reinterpret_cast<bf16*>(const_cast<char*>(kv_row_ptr(a.c, a.block_table, a.max_pages, a.slot[r], p)));
+  uint4 q[NQ], k[NK];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) q[i] = lane + 32 * i < q8 ? qb[lane + 32 * i] : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+  for (int i = 0; i < NK; ++i) k[i] = lane + 32 * i < k8 ? kb[lane + 32 * i] : make_uint4(0u, 0u, 0u, 0u);
+  for (int i = lane; i < v8; i += 32) reinterpret_cast<uint4*>(row + a.c.kw)[i] = vb[i];
+  auto sq8 = [](const uint4& x, float s) {
+    s = fmaf(lo2f(x.x), lo2f(x.x), fmaf(hi2f(x.x), hi2f(x.x), s)), s = fmaf(lo2f(x.y), lo2f(x.y), fmaf(hi2f(x.y), hi2f(x.y), s));
+    return fmaf(lo2f(x.z), lo2f(x.z), fmaf(hi2f(x.z), hi2f(x.z), fmaf(lo2f(x.w), lo2f(x.w), fmaf(hi2f(x.w), hi2f(x.w), s))));
+  };
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) sq = sq8(q[i], sq);
+#pragma unroll
+  for (int i = 0; i < NK; ++i) sk = sq8(k[i], sk);
+  const float rq = a.q_norm ? 1.0f / sqrtf(warp_sum(sq) / (float)(8 * q8) + a.eps) : 1.f;
+  const float rk = a.k_norm ? 1.0f / sqrtf(warp_sum(sk) / (float)(8 * k8) + a.eps) : 1.f;
+  const float *ct = a.rope.cos_t + (size_t)p * half, *sn = a.rope.sin_t + (size_t)p * half;
+  auto turn = [&](const uint4& x, const bf16* w, float rstd, int i, float (&y)[8]) {
+    const uint32_t u[4] = {x.x, x.y, x.z, x.w};
+    uint4 wv = make_uint4(0u, 0u, 0u, 0u);
+    if (w) wv = reinterpret_cast<const uint4*>(w)[i];
+    const uint32_t ww[4] = {wv.x, wv.y, wv.z, wv.w};
+    const int e = 8 * i % d;
+    float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (e < dims) c = *reinterpret_cast<const float4*>(ct + e / 2), s = *reinterpret_cast<const float4*>(sn + e / 2);
+    const float cc[4] = {c.x, c.y, c.z, c.w}, ss[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      float f0 = lo2f(u[j]), f1 = hi2f(u[j]);
+      if (w) f0 *= rstd * lo2f(ww[j]), f1 *= rstd * hi2f(ww[j]);
+      y[2 * j] = f0 * cc[j] - f1 * ss[j];
+      y[2 * j + 1] = f1 * cc[j] + f0 * ss[j];
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < NK; ++i) {
+    const int idx = lane + 32 * i;
+    if (idx >= k8) break;
+    float y[8];
+    turn(k[i], a.k_norm, rk, idx, y);
+    reinterpret_cast<uint4*>(row)[idx] = make_uint4(pack2f(y[0], y[1]), pack2f(y[2], y[3]), pack2f(y[4], y[5]), pack2f(y[6], y[7]));
+  }
+  float* qf = a.q + (size_t)r * a.ldq;
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int idx = lane + 32 * i;
+    if (idx >= q8) break;
+    float y[8];
+    turn(q[i], a.q_norm, rq, idx, y);
+    *reinterpret_cast<float4*>(qf + 8 * idx) = make_float4(y[0], y[1], y[2], y[3]);
+    *reinterpret_cast<float4*>(qf + 8 * idx + 4) = make_float4(y[4], y[5], y[6], y[7]);
   }
 }
 
@@ -799,47 +888,66 @@ __global__ void __launch_bounds__(128) gqa_finish_kernel(const GqaAttnArgs a, in
   for (int c = threadIdx.x; c < vd; c += blockDim.x) out[c] = o[c] * rstd;
 }
 
-// CTA (row, kv head): merges the key splits of every head's attended values of this kv head, then mixes the heads:
-// out[h] = sum_g talk[h, g] a_g for the heads h of the kv head.  Shared memory: weights [heads][n_splits] | a [heads][vd]
-__global__ void __launch_bounds__(128) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits) {
+// CTA of `rows` rows: merges the key splits of every head's attended values and mixes the heads.  Thread = (kv head c, value
+// column): out[h] = sum_g talk[h, g] a_g[c] for the heads h of kv head c, eight of them at a time.  Shared memory: the mix
+// [g][h] as fp32 | split weights [heads][n_splits]
+__global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits, int rows) {
   extern __shared__ float tf_smem[];
   pdl_wait();
   pdl_trigger();
-  const int r = blockIdx.x, c = blockIdx.y, vd = a.vdim, H = a.heads, hpg = H / a.kv_heads;
-  const size_t rs = (size_t)a.kv_heads * vd + 2;
-  const float* rec = a.ws + (size_t)r * H * n_splits * rs;
-  float* wt = tf_smem;
-  float* at = wt + H * n_splits;
-  for (int g = threadIdx.x; g < H; g += blockDim.x) {
-    const float* rg = rec + (size_t)g * n_splits * rs;
-    float M = -INFINITY, L = 0.f;
-    for (int s = 0; s < n_splits; ++s) M = fmaxf(M, rg[s * rs]);
-    for (int s = 0; s < n_splits; ++s) {
-      const float ms = rg[s * rs], w = ms > -INFINITY ? expf(ms - M) : 0.f;
-      wt[g * n_splits + s] = w;
-      L = fmaf(rg[s * rs + 1], w, L);
+  const int vd = a.vdim, H = a.heads, hpg = H / a.kv_heads, ncol = a.kv_heads * vd;
+  const size_t rs = (size_t)ncol + 2;
+  float* tk = tf_smem;
+  float* wt = tk + H * H;
+  for (int i = threadIdx.x; i < H * H; i += blockDim.x) tk[(i % H) * H + i / H] = bf2f(a.talk[i]);
+  for (int r = blockIdx.x * rows; r < min(a.n, (int)(blockIdx.x + 1) * rows); ++r) {
+    const float* rec = a.ws + (size_t)r * H * n_splits * rs;
+    __syncthreads();
+    for (int g = threadIdx.x; g < H; g += blockDim.x) {
+      const float* rg = rec + (size_t)g * n_splits * rs;
+      float M = -INFINITY, L = 0.f;
+      for (int s = 0; s < n_splits; ++s) M = fmaxf(M, rg[s * rs]);
+      for (int s = 0; s < n_splits; ++s) {
+        const float ms = rg[s * rs], w = ms > -INFINITY ? expf(ms - M) : 0.f;
+        wt[g * n_splits + s] = w;
+        L = fmaf(rg[s * rs + 1], w, L);
+      }
+      for (int s = 0; s < n_splits; ++s) wt[g * n_splits + s] /= L;
     }
-    for (int s = 0; s < n_splits; ++s) wt[g * n_splits + s] /= L;
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < H * vd; i += blockDim.x) {
-    const int g = i / vd, col = i - g * vd;
-    const float* rg = rec + (size_t)g * n_splits * rs + 2 + c * vd + col;
-    float v = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-      const float w = wt[g * n_splits + s];
-      if (w > 0.f) v = fmaf(rg[s * rs], w, v);
+    __syncthreads();
+    for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
+      const int c = i / vd, col = i - c * vd;
+      const float* ri = rec + 2 + i;
+      for (int h0 = 0; h0 < hpg; h0 += 8) {
+        float acc[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) acc[k] = 0.f;
+        for (int g0 = 0; g0 < H; g0 += 8) {  // eight heads' values in flight
+          float v[8];
+#pragma unroll
+          for (int u = 0; u < 8; ++u) v[u] = g0 + u < H ? ri[(size_t)(g0 + u) * n_splits * rs] * wt[(g0 + u) * n_splits] : 0.f;
+          for (int s = 1; s < n_splits; ++s)
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+              if (g0 + u < H) v[u] = fmaf(ri[((size_t)(g0 + u) * n_splits + s) * rs], wt[(g0 + u) * n_splits + s], v[u]);
+#pragma unroll
+          for (int u = 0; u < 8; ++u) {
+            if (g0 + u >= H) break;
+            const float* t = tk + (g0 + u) * H + c * hpg + h0;
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              if (h0 + k < hpg) acc[k] = fmaf(t[k], v[u], acc[k]);
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          if (h0 + k >= hpg) break;
+          const size_t o = (size_t)(c * hpg + h0 + k) * vd + col;
+          if (a.out_bf) a.out_bf[(size_t)r * a.ldo_bf + o] = f2bf(acc[k]);
+          else a.out[(size_t)r * a.ldo + o] = acc[k];
+        }
+      }
     }
-    at[i] = v;
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < hpg * vd; i += blockDim.x) {
-    const int h = c * hpg + i / vd, col = i % vd;
-    const bf16* t = a.talk + (size_t)h * H;
-    float v = 0.f;
-    for (int g = 0; g < H; ++g) v = fmaf(bf2f(t[g]), at[g * vd + col], v);
-    if (a.out_bf) a.out_bf[(size_t)r * a.ldo_bf + (size_t)h * vd + col] = f2bf(v);
-    else a.out[(size_t)r * a.ldo + (size_t)h * vd + col] = v;
   }
 }
 
@@ -855,6 +963,17 @@ cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
     if (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2 || !a.c.pool || a.tq.talk || a.v_lam || a.v_keep ||
         (a.q_bf && !a.q) || !(a.k_bf || a.k))
       return cudaErrorInvalidValue;
+    auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int nq = a.q ? a.q_heads * a.norm_dim : 0;
+    if (a.q_bf && a.k_bf && a.v_bf && a.c.elt_bytes == 2 && !(a.c.block > 0 && a.one_each) && !a.rope.half_layout && !a.q_bias && !a.k_bias && !a.v_bias &&
+        a.norm_dim % 8 == 0 && a.rope.dims % 8 == 0 && a.c.vw % 8 == 0 && a.ld_bf % 8 == 0 && a.ldq % 4 == 0 && a.c.layer_off % 8 == 0 && a.c.page_elems % 8 == 0 &&
+        nq <= 4096 && a.c.kw <= 2048 && al(a.q_bf) && al(a.k_bf) && al(a.v_bf) && al(a.q) && al(a.q_norm) && al(a.k_norm) && al(a.c.pool) &&
+        al(a.rope.cos_t) && al(a.rope.sin_t)) {
+      const dim3 grid((a.n + 7) / 8);
+      if (nq <= 1024 && a.c.kw <= 512) return launch_k(kv_store_whole_warp_kernel<4, 2>, grid, dim3(256), 0, st, a);
+      if (nq <= 2048 && a.c.kw <= 1024) return launch_k(kv_store_whole_warp_kernel<8, 4>, grid, dim3(256), 0, st, a);
+      return launch_k(kv_store_whole_warp_kernel<16, 8>, grid, dim3(256), 0, st, a);
+    }
     return launch_k(kv_store_whole_kernel, dim3(a.n), dim3(256), 0, st, a);
   }
   size_t smem = 0;
@@ -872,17 +991,18 @@ cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
 
 cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st) {
   if (n <= 0 || c.block <= 0) return cudaSuccess;
-  return launch_k(kv_pool_rows_kernel, dim3((n + POOL_ROWS - 1) / POOL_ROWS), dim3(128), 0, st, c, pos, slot, block_table, max_pages, n);
+  return launch_k(kv_pool_rows_kernel, dim3((n + POOL_ROWS - 1) / POOL_ROWS), dim3(256), 0, st, c, pos, slot, block_table, max_pages, n);
 }
 
 static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStream_t st) {
-  const size_t smem = ((size_t)a.heads * splits + (size_t)a.heads * a.vdim) * sizeof(float);
+  const size_t smem = ((size_t)a.heads * splits + (size_t)a.heads * a.heads) * sizeof(float);
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return cudaErrorInvalidValue;
     cudaError_t r = cudaFuncSetAttribute(gqa_talk_finish_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (r != cudaSuccess) return r;
   }
-  return launch_k(gqa_talk_finish_kernel, dim3(a.n, a.kv_heads), dim3(128), smem, st, a, splits);
+  const int rows = a.n >= 1024 ? 2 : 1;
+  return launch_k(gqa_talk_finish_kernel, dim3((a.n + rows - 1) / rows), dim3(256), smem, st, a, splits, rows);
 }
 
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches) {

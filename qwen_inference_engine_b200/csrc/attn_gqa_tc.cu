@@ -4,14 +4,17 @@
 // 256 value columns, which is what the tensor cores are good at -- and gqa_talk_finish_kernel mixes the results.
 //
 // A CTA owns 128 consecutive rows of one segment, one query head and one chunk of value columns, and walks tiles of 64 keys: first
-// the tiles of pooled rows that some row sees, then the tokens from the first window's lower edge on.  12 warps:
-//   warps 9-11  copy the tile's key and value rows into the swizzled operand layout (cp.async, ring of stages)
-//   warp 8      issues the products: S = Q K^T (128 x 64, two TMEM buffers, one tile ahead of the softmax) and O += P V (TMEM)
-//   warps 0-7   softmax, two threads per row: S from TMEM, mask, reference maximum, weights as bf16 hi + lo pairs into shared
+// the tiles of pooled rows that some row sees, then the tokens from the first window's lower edge on.  20 warps:
+//   the last 3  bring the tile's key and value rows into the swizzled operand layout, a ring of stages: token rows by TMA boxes of
+//               a page, pooled rows (and token rows of pages that do not divide a tile) by cp.async
+//   warp 16     issues the products: S = Q K^T (128 x 64, two TMEM buffers, one tile ahead of the softmax) and O += P V (TMEM)
+//   warps 0-15  softmax, four threads per row: S from TMEM, mask, reference maximum, weights as bf16 hi + lo pairs into shared
 //               memory (two buffers, two products per tile, so a weight keeps ~16 bits)
 // O stays in TMEM over all tiles.  Instead of scaling it whenever a row's maximum grows, a row keeps its reference maximum until a
 // score exceeds it by RESCALE (weights then stay below 2^RESCALE); only then the warp that owns the row scales its part of O.
 // Every wait has a limit; when one runs out the CTA finishes without waiting and marks its results as not a number.
+#include <cuda.h>
+
 #include <algorithm>
 
 #include "common.cuh"
@@ -24,7 +27,7 @@ namespace qie {
 namespace {
 
 constexpr int TQ = 128, TK = 64;
-constexpr int NSOFT = 256, NLOAD = 96, NTHR = NSOFT + 32 + NLOAD;
+constexpr int NSOFT = 512, NLOAD = 96, MMA_WARP = NSOFT / 32, NTHR = NSOFT + 32 + NLOAD;
 constexpr int LROWS = NLOAD / 8, LPASS = (TK + LROWS - 1) / LROWS;  // rows a pass of the copying threads covers
 constexpr int KBLK = TK * 128;   // [64 keys][64 columns] bf16, 8-row swizzle atoms: 8 KiB
 constexpr int QBLK = TQ * 128;   // [128 rows][64 columns]: 16 KiB
@@ -59,23 +62,18 @@ __device__ __forceinline__ void umma_tc(uint32_t d_tmem, uint64_t adesc, uint64_
 __device__ __forceinline__ void umma_commit_tc(uint32_t bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
 }
-__device__ __forceinline__ void tmem_ld32_tc(uint32_t taddr, uint32_t (&r)[32]) {
+__device__ __forceinline__ void tmem_ld16_tc(uint32_t taddr, uint32_t (&r)[16]) {
   asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
-      "%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
       : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-        "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-        "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
       : "r"(taddr));
 }
-__device__ __forceinline__ void tmem_st32_tc(uint32_t taddr, const uint32_t (&r)[32]) {
+__device__ __forceinline__ void tmem_st16_tc(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%32], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
-      "%23,%24,%25,%26,%27,%28,%29,%30,%31};"
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};"
       ::"r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
-      "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]),
-      "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]), "r"(taddr)
+      "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
       : "memory");
 }
 // K-major operand, SWIZZLE_128B, 8-row atoms 1024 bytes apart
@@ -109,11 +107,12 @@ __host__ __device__ inline TcLayout tc_layout(int dblk, int vblk, int nst) {
   l.st = l.p + 4 * QBLK;          // stages: K blocks | V blocks
   l.stage = (dblk + vblk) * KBLK;
   l.bar = l.st + nst * l.stage;   // mbarriers, flags, row maxima
-  l.total = l.bar + 256 + 4 * TQ * 4;
+  l.total = l.bar + 256 + 8 * TQ * 4;
   return l;
 }
 
-__global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc) {
+__global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc,
+                                                               const __grid_constant__ CUtensorMap rows_map, int use_tma) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   __shared__ int info[4];  // first row, rows, slot
   __shared__ int dead_s;
@@ -139,7 +138,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   unsigned char* sg = smem_raw + (s0 - smem_u32(smem_raw));
   const uint32_t b0 = s0 + L.bar;
   const uint32_t bar_full = b0, bar_empty = b0 + 32, bar_s = b0 + 64, bar_p = b0 + 80, bar_o = b0 + 96, tslot = b0 + 112;
-  float* xmax = reinterpret_cast<float*>(sg + L.bar + 256);  // [tile parity][half][row]; the sums use the first half at the end
+  float* xmax = reinterpret_cast<float*>(sg + L.bar + 256);  // [tile parity][quarter][row]; the sums use the parity that the last tile did not
   const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), dim = a.dim;
   const int vcols = a.kv_heads * a.vdim, col0 = blockIdx.z * vc, nv = min(vc, vcols - col0);
   const int pos0 = a.pos[row0], pmax = pos0 + nrows - 1;
@@ -151,7 +150,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
     for (int i = 0; i < 2; ++i) mbar_init_tc(bar_s + 8 * i, 1), mbar_init_tc(bar_p + 8 * i, NSOFT), mbar_init_tc(bar_o + 8 * i, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 8) {
+  if (warp == MMA_WARP) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tslot), "r"(512u) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
@@ -176,7 +175,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   const uint32_t t_o = tmem + 128;  // S: columns 0..127 (two buffers), O: 128 ..
   const int vcp = vblk * 64;        // columns of O
 
-  if (warp >= 9) {
+  if (warp > MMA_WARP) {
     // ---- copies
     const int lt = tid - (NSOFT + 32), ch = lt & 7, rr = lt >> 3;  // chunk of a 64-column block, rows rr + LROWS k
     const size_t koff = (size_t)g * dim, voff = (size_t)a.c.kw + col0;
@@ -184,13 +183,35 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       mbar_arrive_tc(bar_full + 8 * (t % nst));
     };
+    bool prev_cp = false;  // the tile before was copied by cp.async and is not announced yet
     for (int t = 0; t < nt; ++t) {
       const int s = t % nst;
-      if (t > 0 && nst == 2) {  // the stage that this tile waits for is only given back behind the scores of the tile before
+      const bool tma = use_tma && t >= npt;
+      if (prev_cp && (nst == 2 || tma)) {  // (two stages: the stage that this tile waits for is only given back behind the scores of the tile before)
         cp_async_wait<0>();
         announce(t - 1);
+        prev_cp = false;
       }
       if (t >= nst) mbar_wait_tc(bar_empty + 8 * s, (uint32_t)((t / nst - 1) & 1), dead);
+      const uint32_t base = s0 + L.st + s * L.stage;
+      if (tma) {  // boxes of up to 64 rows of a page and 64 columns; rows behind the last position and columns behind a part are
+                  // other cache contents, finite numbers that meet zero weights, zero queries or columns nobody reads
+        if (lt == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar_full + 8 * s), "r"((uint32_t)L.stage) : "memory");
+        else mbar_arrive_tc(bar_full + 8 * s);
+        if (warp == MMA_WARP + 1) {
+          __syncwarp();
+          const int br = min(a.c.page_size, TK), nbx = TK / br, j0 = (tt0 + t - npt) * TK;
+          for (int i = lane; i < nbx * (dblk + vblk); i += 32) {
+            const int b = i / nbx, pg = i - b * nbx;
+            const int x = b < dblk ? g * dim + b * 64 : a.c.kw + col0 + (b - dblk) * 64;
+            const int page = a.block_table[(size_t)slot * a.max_pages + min(j0 + pg * br, pmax) / a.c.page_size];
+            asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+                         ::"r"(base + b * KBLK + pg * br * 128), "l"(&rows_map), "r"(bar_full + 8 * s), "r"(x), "r"(j0 % a.c.page_size), "r"(page)
+                         : "memory");
+          }
+        }
+        continue;
+      }
       const bf16* rowp[LPASS];
 #pragma unroll
       for (int k = 0; k < LPASS; ++k) {
@@ -204,7 +225,6 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
         }
         rowp[k] = reinterpret_cast<const bf16*>(p);
       }
-      const uint32_t base = s0 + L.st + s * L.stage;
       for (int b = 0; b < dblk + vblk; ++b) {
         const bool isv = b >= dblk;
         const int c = (isv ? b - dblk : b) * 64 + ch * 8;
@@ -219,14 +239,17 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
         }
       }
       cp_async_commit();
-      if (t > 0 && nst > 2) {
+      if (prev_cp) {
         cp_async_wait<1>();
         announce(t - 1);
       }
+      prev_cp = true;
     }
-    cp_async_wait<0>();
-    announce(nt - 1);
-  } else if (warp == 8) {
+    if (prev_cp) {
+      cp_async_wait<0>();
+      announce(nt - 1);
+    }
+  } else if (warp == MMA_WARP) {
     // ---- products
     if (lane == 0) {
       const uint32_t id_s = idesc_tc(TQ, TK, false), id_o = idesc_tc(TQ, vcp, true);
@@ -255,34 +278,35 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
     }
     __syncwarp();
   } else {
-    // ---- softmax: row (TMEM lane), half of the tile's keys and of O's columns
-    const int row = (warp & 3) * 32 + lane, hf = warp >> 2;
+    // ---- softmax: row (TMEM lane), quarter of the tile's keys and of O's columns
+    const int row = (warp & 3) * 32 + lane, qt = warp >> 2;
     const int my_pos = pos0 + row, my_lo = a.window > 0 ? my_pos - a.window + 1 : 0, my_seen = a.c.block > 0 ? pooled_seen(my_pos, a.window, a.c.block) : 0;
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const float sl2 = a.scale * 1.4426950408889634f;
+    const int oc0 = qt * (vcp / 4), oc1 = oc0 + vcp / 4;
     float m_ref = -INFINITY, l_run = 0.f;
     for (int t = 0; t < nt; ++t) {
       mbar_wait_tc(bar_s + 8 * (t & 1), (uint32_t)((t >> 1) & 1), dead);
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      uint32_t r[32];
-      tmem_ld32_tc(tmem + lane_addr + (uint32_t)((t & 1) * TK + 32 * hf), r);
+      uint32_t r[16];
+      tmem_ld16_tc(tmem + lane_addr + (uint32_t)((t & 1) * TK + 16 * qt), r);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-      // visible keys of this thread: first .. last (relative to its 32)
+      // visible keys of this thread: first .. last (relative to its 16)
       int first, last;
-      if (t < npt) first = 0, last = my_seen - 1 - (t * TK + 32 * hf);
-      else first = my_lo - ((tt0 + t - npt) * TK + 32 * hf), last = my_pos - ((tt0 + t - npt) * TK + 32 * hf);
-      float mx = -INFINITY;
-      if (first > 0 || last < 31) {
+      if (t < npt) first = 0, last = my_seen - 1 - (t * TK + 16 * qt);
+      else first = my_lo - ((tt0 + t - npt) * TK + 16 * qt), last = my_pos - ((tt0 + t - npt) * TK + 16 * qt);
+      if (first > 0 || last < 15) {
 #pragma unroll
-        for (int j = 0; j < 32; ++j)
+        for (int j = 0; j < 16; ++j)
           if (j < first || j > last) r[j] = 0xff800000u;  // -inf
       }
+      float mx = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < 32; ++j) mx = fmaxf(mx, __uint_as_float(r[j]));
-      float* xm = xmax + (t & 1) * 2 * TQ;
-      xm[hf * TQ + row] = mx;
-      asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp & 3)) : "memory");  // the two warps that share these 32 rows
-      mx = fmaxf(mx, xm[(hf ^ 1) * TQ + row]) * sl2;
+      for (int j = 0; j < 16; ++j) mx = fmaxf(mx, __uint_as_float(r[j]));
+      float* xm = xmax + (t & 1) * 4 * TQ + row;
+      xm[qt * TQ] = mx;
+      asm volatile("bar.sync %0, 128;" ::"r"(1 + (warp & 3)) : "memory");  // the four warps that share these 32 rows
+      mx = fmaxf(fmaxf(xm[0], xm[TQ]), fmaxf(xm[2 * TQ], xm[3 * TQ])) * sl2;
       const bool grow = mx > m_ref + RESCALE;
       if (__any_sync(0xffffffffu, grow)) {
         const float m_new = fmaxf(m_ref, mx), f = m_new > -INFINITY ? ex2_tc(m_ref - m_new) : 1.f;
@@ -290,70 +314,69 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
         if (t > 0) {  // scale this thread's columns of O once the product of the tile before is in
           mbar_wait_tc(bar_o + 8 * ((t - 1) & 1), (uint32_t)(((t - 1) >> 1) & 1), dead);
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-          for (int c = hf * (vcp / 2); c < (hf + 1) * (vcp / 2); c += 32) {
-            uint32_t o[32];
-            tmem_ld32_tc(t_o + lane_addr + c, o);
+          for (int c = oc0; c < oc1; c += 16) {
+            uint32_t o[16];
+            tmem_ld16_tc(t_o + lane_addr + c, o);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-            for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * f);
-            tmem_st32_tc(t_o + lane_addr + c, o);
+            for (int j = 0; j < 16; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * f);
+            tmem_st16_tc(t_o + lane_addr + c, o);
           }
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
       const float nm = m_ref > -INFINITY ? -m_ref : 0.f;
-      if (t >= 2) mbar_wait_tc(bar_o + 8 * (t & 1), (uint32_t)(((t >> 1) - 1) & 1), dead);  // the product that read this P buffer
-      const uint32_t pd = s0 + L.p + (t & 1) * 2 * QBLK;
       float rs = 0.f;
+      uint32_t hi[8], lo[8];
 #pragma unroll
-      for (int q8 = 0; q8 < 4; ++q8) {
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float e0 = ex2_tc(fmaf(__uint_as_float(r[q8 * 8 + 2 * e]), sl2, nm)), e1 = ex2_tc(fmaf(__uint_as_float(r[q8 * 8 + 2 * e + 1]), sl2, nm));
-          rs += e0 + e1;
-          const bf16 h0 = f2bf(e0), h1 = f2bf(e1);
-          hi[e] = pack2(h0, h1);
-          lo[e] = pack2(f2bf(e0 - bf2f(h0)), f2bf(e1 - bf2f(h1)));
-        }
-        const uint32_t o = blk_off(row, 4 * hf + q8);
-        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + o), "r"(hi[0]), "r"(hi[1]), "r"(hi[2]), "r"(hi[3]) : "memory");
-        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + QBLK + o), "r"(lo[0]), "r"(lo[1]), "r"(lo[2]), "r"(lo[3]) : "memory");
+      for (int e = 0; e < 8; ++e) {
+        const float e0 = ex2_tc(fmaf(__uint_as_float(r[2 * e]), sl2, nm)), e1 = ex2_tc(fmaf(__uint_as_float(r[2 * e + 1]), sl2, nm));
+        rs += e0 + e1;
+        hi[e] = pack2f(e0, e1);
+        lo[e] = pack2f(e0 - lo2f(hi[e]), e1 - hi2f(hi[e]));
       }
       l_run += rs;
+      if (t >= 2) mbar_wait_tc(bar_o + 8 * (t & 1), (uint32_t)(((t >> 1) - 1) & 1), dead);  // the product that read this P buffer
+      const uint32_t pd = s0 + L.p + (t & 1) * 2 * QBLK;
+#pragma unroll
+      for (int q8 = 0; q8 < 2; ++q8) {
+        const uint32_t o = blk_off(row, 2 * qt + q8);
+        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + o), "r"(hi[4 * q8]), "r"(hi[4 * q8 + 1]), "r"(hi[4 * q8 + 2]), "r"(hi[4 * q8 + 3]) : "memory");
+        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + QBLK + o), "r"(lo[4 * q8]), "r"(lo[4 * q8 + 1]), "r"(lo[4 * q8 + 2]), "r"(lo[4 * q8 + 3]) : "memory");
+      }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       mbar_arrive_tc(bar_p + 8 * (t & 1));
     }
     mbar_wait_tc(bar_o + 8 * ((nt - 1) & 1), (uint32_t)(((nt - 1) >> 1) & 1), dead);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    float* xs = xmax + (nt & 1) * 2 * TQ;  // the buffer that the last tile did not use
-    xs[hf * TQ + row] = l_run;
-    asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp & 3)) : "memory");
-    const float l = l_run + xs[(hf ^ 1) * TQ + row];
+    float* xs = xmax + (nt & 1) * 4 * TQ + row;
+    xs[qt * TQ] = l_run;
+    asm volatile("bar.sync %0, 128;" ::"r"(1 + (warp & 3)) : "memory");
+    const float l = (xs[0] + xs[TQ]) + (xs[2 * TQ] + xs[3 * TQ]);
     const float inv = *dead ? __int_as_float(0x7fffffff) : (l > 0.f ? 1.0f / l : 0.f);
-    float* rec = a.ws + ((size_t)(row0 + row) * a.heads + h) * (vcols + 2);
-    if (row < nrows && hf == 0 && blockIdx.z == 0) rec[0] = 0.f, rec[1] = 1.f;
-    for (int c = hf * (vcp / 2); c < (hf + 1) * (vcp / 2); c += 32) {
-      uint32_t o[32];
-      tmem_ld32_tc(t_o + lane_addr + c, o);
+    const size_t rs_rec = (size_t)vcols + 2;
+    float* rec = a.ws + ((size_t)(row0 + (warp & 3) * 32) * a.heads + h) * rs_rec;  // record of the warp's first row
+    const size_t row_step = (size_t)a.heads * rs_rec;
+    const int wrows = min(32, nrows - (warp & 3) * 32);
+    if (lane < wrows && qt == 0 && blockIdx.z == 0) rec[lane * row_step] = 0.f, rec[lane * row_step + 1] = 1.f;
+    float* tr = reinterpret_cast<float*>(sg + L.p) + warp * (32 * 17);  // every product is done: P is free to turn the rows around
+    for (int c = oc0; c < oc1; c += 16) {
+      uint32_t o[16];
+      tmem_ld16_tc(t_o + lane_addr + c, o);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-      if (row < nrows) {
-        float* d = rec + 2 + col0 + c;
-        if (c + 32 <= nv) {  // records are 8-byte aligned
+      __syncwarp();
 #pragma unroll
-          for (int j = 0; j < 32; j += 2) *reinterpret_cast<float2*>(d + j) = make_float2(__uint_as_float(o[j]) * inv, __uint_as_float(o[j + 1]) * inv);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 32; ++j)
-            if (c + j < nv) d[j] = __uint_as_float(o[j]) * inv;
-        }
-      }
+      for (int j = 0; j < 16; ++j) tr[lane * 17 + j] = __uint_as_float(o[j]) * inv;
+      __syncwarp();
+      const int cc = c + (lane & 15);
+      if (cc < nv)
+        for (int i = lane >> 4; i < wrows; i += 2) rec[i * row_step + 2 + col0 + cc] = tr[i * 17 + (lane & 15)];
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();
-  if (warp == 8) {
+  if (warp == MMA_WARP) {
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
   }
@@ -393,7 +416,14 @@ cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st) {
     if (r != cudaSuccess) return r;
     once.done();
   }
-  return launch_k(gqa_talk_tc_kernel, dim3(a.heads, a.n / TQ + a.n_seg, p.nvc), dim3(NTHR), p.smem, st, a, p.dblk, p.vblk, p.nst, p.vc);
+  // token rows by TMA where a tile of 64 positions is whole pages or lies in one (pages of 8, 16, 32 or a multiple of 64 positions)
+  TensorMap2D tm{};
+  const int ps = a.c.page_size, row = a.c.kw + a.c.vw;
+  const int use_tma = a.c.n_pages > 0 && row >= 64 && (ps % TK == 0 || (TK % ps == 0 && ps >= 8)) &&
+                      make_tensor_map_pages(&tm, static_cast<const bf16*>(a.c.pool) + a.c.layer_off, row, ps, a.c.n_pages, a.c.page_elems,
+                                            std::min(ps, TK)) == cudaSuccess;
+  return launch_k(gqa_talk_tc_kernel, dim3(a.heads, a.n / TQ + a.n_seg, p.nvc), dim3(NTHR), p.smem, st, a, p.dblk, p.vblk, p.nst, p.vc,
+                  *reinterpret_cast<const CUtensorMap*>(&tm), use_tma);
 }
 
 }  // namespace qie

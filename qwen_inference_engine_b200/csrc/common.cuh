@@ -17,6 +17,11 @@ __device__ __forceinline__ float hi2f(uint32_t p) { return __uint_as_float(p & 0
 __device__ __forceinline__ uint32_t pack2(bf16 a, bf16 b) {
   return (uint32_t)__bfloat16_as_ushort(a) | ((uint32_t)__bfloat16_as_ushort(b) << 16);
 }
+// the same of two floats, rounded to nearest even
+__device__ __forceinline__ uint32_t pack2f(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
 
 // ---- cp.async (LDGSTS) 16-byte global->shared -------------------------------------
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {

@@ -76,6 +76,7 @@ struct KvRowCache {
   // lies in the page that holds its last position, as that page's pooled row number b - floor(first position of the page / block)
   int block = 0;
   size_t pool_off = 0;  // elements into the page
+  int n_pages = 0;      // pages of the pool (0: unknown; then no kernel describes the pool as a tensor)
 };
 // pooled rows that a page has room for
 inline int kv_pool_rows(int page_size, int block) { return block > 0 ? (page_size + block - 1) / block : 0; }

@@ -458,7 +458,7 @@ cudaError_t GbModel::forward(qie_engine* e, int n, int n_seg, int n_out, int max
       const int H = L.heads, G = L.kv_heads, d = L.dim, vd = L.vdim;
       KvRowCache c;
       c.pool = m->kv_pool, c.elt_bytes = m->f32 ? 4 : 2, c.page_size = e->kv.page_size, c.page_elems = m->page_elems;
-      c.layer_off = L.kv_off, c.kw = G * d, c.vw = G * vd, c.block = L.pool, c.pool_off = L.pool_off;
+      c.layer_off = L.kv_off, c.kw = G * d, c.vw = G * vd, c.block = L.pool, c.pool_off = L.pool_off, c.n_pages = e->kv.n_pages;
       const float* q = m->p0 + L.o_q;
       int ldq = ld;
       {  // keys (norm over all kv heads, rotation) and values -> cache rows; the queries alike

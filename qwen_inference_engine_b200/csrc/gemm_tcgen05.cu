@@ -795,6 +795,20 @@ cudaError_t make_tensor_map_kv(TensorMap2D* out, const bf16* pool, unsigned long
   return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
 }
 
+cudaError_t make_tensor_map_pages(TensorMap2D* out, const bf16* base, int row_elems, int page_size, int n_pages, size_t page_elems, int box_rows) {
+  EncodeTiledFn enc = get_encode();
+  if (!enc) return cudaErrorNotSupported;
+  if (row_elems % 8 || page_elems % 8 || box_rows < 1 || box_rows > 256 || (reinterpret_cast<uintptr_t>(base) & 15)) return cudaErrorInvalidValue;
+  cuuint64_t dims[3] = {(cuuint64_t)row_elems, (cuuint64_t)page_size, (cuuint64_t)n_pages};
+  cuuint64_t strides[2] = {(cuuint64_t)row_elems * 2, (cuuint64_t)page_elems * 2};
+  cuuint32_t box[3] = {64, (cuuint32_t)box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(reinterpret_cast<CUtensorMap*>(out), CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, (void*)base, dims, strides, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
+}
+
 template <int BN>
 static cudaError_t launch_bn(const TcGemm& t, const TcArgs& g, int token_tiles, cudaStream_t st) {
   constexpr int STAGE_BYTES = BM * BK * 2 + BN * BK * 2;

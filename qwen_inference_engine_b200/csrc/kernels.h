@@ -140,6 +140,9 @@ cudaError_t make_tensor_map_2d(TensorMap2D* out, const bf16* base, int rows, int
 cudaError_t make_tensor_map_w3d(TensorMap2D* out, const bf16* base, int rows, int K, int kc, int ld = 0, int box_rows = 8);  // ld: row stride in elements (0 = K)
 // KV pool as a 2-D tensor {head_dim 64, every (page, layer, K|V, head, slot) row}: box = box_rows slots x 128 bytes, 128-byte swizzle
 cudaError_t make_tensor_map_kv(TensorMap2D* out, const bf16* pool, unsigned long long rows, int hd, int box_rows);
+// cache rows of one layer as a 3-D tensor {row elements, positions of a page, pages} (page stride page_elems): box = 64 elements x box_rows
+// positions of one page, 128-byte swizzle
+cudaError_t make_tensor_map_pages(TensorMap2D* out, const bf16* base, int row_elems, int page_size, int n_pages, size_t page_elems, int box_rows);
 int tc_token_tile(int M);
 struct TcGemm {
   const TensorMap2D* w[3];  // weight maps, box rows = 128

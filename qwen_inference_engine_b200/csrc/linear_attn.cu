@@ -104,12 +104,14 @@ __device__ __forceinline__ void ldmatrix_x2_trans_la(uint32_t& r0, uint32_t& r1,
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
 
-// which chunk: {first row, rows, segment} of chunk number id (false: there is no such chunk)
-__device__ __forceinline__ bool find_chunk(const LinearAttnArgs& a, int id, int* info) {
+constexpr int LT = 256;  // threads of the chunk kernels
+
+// which chunk: first row, rows and segment of chunk number id (false: there is no such chunk); every thread reads the same few words
+__device__ __forceinline__ bool find_chunk(const LinearAttnArgs& a, int id, int* row0, int* rows) {
   for (int s = 0; s < a.n_seg; ++s) {
     const int r0 = a.seg_start[s], len = a.seg_start[s + 1] - r0, nc = (len + LC - 1) / LC;
     if (id < nc) {
-      info[0] = r0 + id * LC, info[1] = min(LC, len - id * LC), info[2] = s;
+      *row0 = r0 + id * LC, *rows = min(LC, len - id * LC);
       return true;
     }
     id -= nc;
@@ -117,68 +119,96 @@ __device__ __forceinline__ bool find_chunk(const LinearAttnArgs& a, int id, int*
   return false;
 }
 
-// 64 rows x cols of a bf16 source (columns col0 ..) -> smem tile [64][P + 8], zeros beyond, silu where asked
+// 64 rows x cols of a bf16 source -> registers (every load in flight at once) -> smem tile [64][P + 8], zeros beyond, silu where asked
 template <int P>
-__device__ __forceinline__ void load_tile(const bf16* src, int ld, int row0, int nrows, int cols, int act, bf16 (*dst)[P + 8]) {
-  const bool vec = cols % 8 == 0 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
-  for (int i = threadIdx.x; i < LC * (P / 8); i += blockDim.x) {
-    const int r = i / (P / 8), c = (i % (P / 8)) * 8;
-    bf16* d = &dst[r][c];
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < nrows && c < cols) {
+struct TileRegs {
+  static constexpr int N = LC * (P / 8) / LT;
+  uint4 v[N];
+  __device__ __forceinline__ void load(const bf16* src, int ld, int row0, int nrows, int cols) {
+    const bool vec = cols % 8 == 0 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int i = threadIdx.x + k * LT, r = i / (P / 8), c = (i % (P / 8)) * 8;
+      v[k] = make_uint4(0u, 0u, 0u, 0u);
+      if (r >= nrows || c >= cols) continue;
       const bf16* s = src + (size_t)(row0 + r) * ld + c;
       if (vec) {
-        v = *reinterpret_cast<const uint4*>(s);
+        v[k] = *reinterpret_cast<const uint4*>(s);
       } else {
         bf16 t[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) t[e] = c + e < cols ? s[e] : f2bf(0.f);
-        v = make_uint4(pack2(t[0], t[1]), pack2(t[2], t[3]), pack2(t[4], t[5]), pack2(t[6], t[7]));
-      }
-      if (act) {
-        v.x = pack2(f2bf(silu_f(lo2f(v.x))), f2bf(silu_f(hi2f(v.x)))), v.y = pack2(f2bf(silu_f(lo2f(v.y))), f2bf(silu_f(hi2f(v.y))));
-        v.z = pack2(f2bf(silu_f(lo2f(v.z))), f2bf(silu_f(hi2f(v.z)))), v.w = pack2(f2bf(silu_f(lo2f(v.w))), f2bf(silu_f(hi2f(v.w))));
+        v[k] = make_uint4(pack2(t[0], t[1]), pack2(t[2], t[3]), pack2(t[4], t[5]), pack2(t[6], t[7]));
       }
     }
-    *reinterpret_cast<uint4*>(d) = v;
   }
-}
+  __device__ __forceinline__ void store(bf16 (*dst)[P + 8], int act) {
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int i = threadIdx.x + k * LT, r = i / (P / 8), c = (i % (P / 8)) * 8;
+      uint4 x = v[k];
+      if (act) {
+        x.x = pack2f(silu_f(lo2f(x.x)), silu_f(hi2f(x.x))), x.y = pack2f(silu_f(lo2f(x.y)), silu_f(hi2f(x.y)));
+        x.z = pack2f(silu_f(lo2f(x.z)), silu_f(hi2f(x.z))), x.w = pack2f(silu_f(lo2f(x.w)), silu_f(hi2f(x.w)));
+      }
+      *reinterpret_cast<uint4*>(&dst[r][c]) = x;
+    }
+  }
+};
 
-// CTA (chunk, head): U [dim, vdim] = sum_s decay^(L-1-s) k_scale k_s v_s^T -> ws.  Warp w owns the state rows 16 w .. (and 64 further).
+// CTA (chunk, head): U [dim, vdim] = sum_s decay^(L-1-s) k_scale k_s v_s^T -> ws.  A warp takes 16 state rows x half of the columns.
 template <int DP, int VP>
-__global__ void __launch_bounds__(128) linear_chunk_state_kernel(const LinearAttnArgs a) {
+__global__ void __launch_bounds__(LT) linear_chunk_state_kernel(const LinearAttnArgs a) {
   extern __shared__ __align__(16) unsigned char lc_smem[];
   typedef bf16 KT[DP + 8];
   typedef bf16 VT[VP + 8];
   KT* Kh = reinterpret_cast<KT*>(lc_smem);
   KT* Kl = Kh + LC;
   VT* Vs = reinterpret_cast<VT*>(Kl + LC);
-  __shared__ int info[3];
   pdl_wait();
   pdl_trigger();
-  if (threadIdx.x == 0 && !find_chunk(a, blockIdx.x, info)) info[0] = -1;
-  __syncthreads();
-  if (info[0] < 0) return;
-  const int h = blockIdx.y, row0 = info[0], L = info[1], dim = a.dim, vdim = a.vdim;
-  load_tile<DP>(a.k_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Kh);
-  load_tile<VP>(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim, a.act, Vs);
-  __syncthreads();
+  int row0, L;
+  if (!find_chunk(a, blockIdx.x, &row0, &L)) return;
+  const int h = blockIdx.y, dim = a.dim, vdim = a.vdim;
   const float* pw = a.decay_pow + h * (LC + 1);
-  for (int i = threadIdx.x; i < L * DP; i += blockDim.x) {  // decayed keys as hi + lo pairs
-    const int s = i / DP, d = i - s * DP;
-    const float x = bf2f(Kh[s][d]) * (a.k_scale * pw[L - 1 - s]);
-    const bf16 hi = f2bf(x);
-    Kh[s][d] = hi;
-    Kl[s][d] = f2bf(x - bf2f(hi));
+  {
+    TileRegs<DP> k;
+    TileRegs<VP> v;
+    k.load(a.k_bf + h * dim, a.ld_bf, row0, L, dim);
+    v.load(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim);
+    v.store(Vs, a.act);
+    // decayed keys as hi + lo pairs
+#pragma unroll
+    for (int n = 0; n < TileRegs<DP>::N; ++n) {
+      const int i = threadIdx.x + n * LT, r = i / (DP / 8), c = (i % (DP / 8)) * 8;
+      const float f = r < L ? a.k_scale * pw[L - 1 - r] : 0.f;
+      const uint32_t u[4] = {k.v[n].x, k.v[n].y, k.v[n].z, k.v[n].w};
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float x0 = lo2f(u[j]), x1 = hi2f(u[j]);
+        if (a.act) {  // the activated key is a bf16 value, as in the scores
+          const uint32_t act = pack2f(silu_f(x0), silu_f(x1));
+          x0 = lo2f(act), x1 = hi2f(act);
+        }
+        x0 *= f, x1 *= f;
+        hi[j] = pack2f(x0, x1);
+        lo[j] = pack2f(x0 - lo2f(hi[j]), x1 - hi2f(hi[j]));
+      }
+      *reinterpret_cast<uint4*>(&Kh[r][c]) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(&Kl[r][c]) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
   }
-  for (int i = L * DP + threadIdx.x; i < LC * DP; i += blockDim.x) Kl[i / DP][i % DP] = f2bf(0.f);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int HB = VP / 16;  // blocks of 8 columns per half
   float* U = a.ws + ((size_t)blockIdx.x * a.heads + h) * dim * vdim;
-  for (int m0 = warp * 16; m0 < DP && m0 < dim; m0 += 64) {
-    float acc[VP / 8][4];
+  for (int u = warp; u < DP / 8; u += LT / 32) {
+    const int m0 = (u >> 1) * 16, vb0 = (u & 1) * HB;
+    if (m0 >= dim || vb0 * 8 >= vdim) continue;
+    float acc[HB][4];
 #pragma unroll
-    for (int i = 0; i < VP / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int i = 0; i < HB; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
     for (int kb = 0; kb < LC / 16; ++kb) {
       // A = K'^T: element (state row m, token k) lies at [k][m]
@@ -187,20 +217,27 @@ __global__ void __launch_bounds__(128) linear_chunk_state_kernel(const LinearAtt
       ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], smem_u32(&Kh[tok][dm]));
       ldmatrix_x4_trans(al[0], al[1], al[2], al[3], smem_u32(&Kl[tok][dm]));
 #pragma unroll
-      for (int vb = 0; vb < VP / 8; ++vb) {
+      for (int vb = 0; vb < HB; ++vb) {
         uint32_t b0, b1;
-        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][vb * 8]));
+        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][(vb0 + vb) * 8]));
         mma_bf16_16816(acc[vb], ah, b0, b1);
         mma_bf16_16816(acc[vb], al, b0, b1);
       }
     }
     const int r = m0 + (lane >> 2), c = (lane & 3) * 2;
 #pragma unroll
-    for (int vb = 0; vb < VP / 8; ++vb)
+    for (int vb = 0; vb < HB; ++vb)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int rr = r + (e >> 1) * 8, cc = vb * 8 + c + (e & 1);
-        if (rr < dim && cc < vdim) U[(size_t)rr * vdim + cc] = acc[vb][e];
+      for (int e = 0; e < 4; e += 2) {
+        const int rr = r + (e >> 1) * 8, cc = (vb0 + vb) * 8 + c;
+        if (rr >= dim || cc >= vdim) continue;
+        float* d = U + (size_t)rr * vdim + cc;
+        if (vdim % 2 == 0) {
+          *reinterpret_cast<float2*>(d) = make_float2(acc[vb][e], acc[vb][e + 1]);
+        } else {
+          d[0] = acc[vb][e];
+          if (cc + 1 < vdim) d[1] = acc[vb][e + 1];
+        }
       }
   }
 }
@@ -235,9 +272,10 @@ __global__ void __launch_bounds__(256) linear_carry_kernel(const LinearAttnArgs 
   *st = S;
 }
 
-// CTA (chunk, head): the outputs of the chunk's rows from its entry state and its own keys and values; warp w owns rows 16 w ..
+// CTA (chunk, head): the outputs of the chunk's rows from its entry state and its own keys and values; warp w owns rows
+// 16 (w % 4) .. and half w / 4 of the value columns
 template <int DP, int VP>
-__global__ void __launch_bounds__(128) linear_chunk_out_kernel(const LinearAttnArgs a) {
+__global__ void __launch_bounds__(LT) linear_chunk_out_kernel(const LinearAttnArgs a) {
   extern __shared__ __align__(16) unsigned char lc_smem[];
   typedef bf16 KT[DP + 8];
   typedef bf16 VT[VP + 8];
@@ -246,32 +284,49 @@ __global__ void __launch_bounds__(128) linear_chunk_out_kernel(const LinearAttnA
   VT* Vs = reinterpret_cast<VT*>(Ks + LC);
   VT* Sh = Vs + LC;   // [DP] entry state, hi
   VT* Sl = Sh + DP;   // lo
-  __shared__ int info[3];
   __shared__ float pw[LC + 1];
+  __shared__ float sq[2][LC];
   pdl_wait();
   pdl_trigger();
-  if (threadIdx.x == 0 && !find_chunk(a, blockIdx.x, info)) info[0] = -1;
-  __syncthreads();
-  if (info[0] < 0) return;
-  const int h = blockIdx.y, row0 = info[0], L = info[1], dim = a.dim, vdim = a.vdim, tid = threadIdx.x;
-  for (int i = tid; i <= LC; i += 128) pw[i] = a.decay_pow[h * (LC + 1) + i];
-  load_tile<DP>(a.q_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Qs);
-  load_tile<DP>(a.k_bf + h * dim, a.ld_bf, row0, L, dim, a.act, Ks);
-  load_tile<VP>(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim, a.act, Vs);
+  int row0, L;
+  if (!find_chunk(a, blockIdx.x, &row0, &L)) return;
+  const int h = blockIdx.y, dim = a.dim, vdim = a.vdim, tid = threadIdx.x;
+  {
+    TileRegs<DP> q, k;
+    TileRegs<VP> v;
+    q.load(a.q_bf + h * dim, a.ld_bf, row0, L, dim);
+    k.load(a.k_bf + h * dim, a.ld_bf, row0, L, dim);
+    v.load(a.v_bf + h * vdim, a.ld_bf, row0, L, vdim);
+    for (int i = tid; i <= LC; i += LT) pw[i] = a.decay_pow[h * (LC + 1) + i];
+    q.store(Qs, a.act);
+    k.store(Ks, a.act);
+    v.store(Vs, a.act);
+  }
   {
     const float* S = a.ws + ((size_t)blockIdx.x * a.heads + h) * dim * vdim;
     if (vdim % 4 == 0) {
-      for (int i = tid; i < DP * (VP / 4); i += 128) {
-        const int d = i / (VP / 4), c = (i % (VP / 4)) * 4;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (d < dim && c < vdim) x = *reinterpret_cast<const float4*>(S + (size_t)d * vdim + c);
-        const bf16 h0 = f2bf(x.x), h1 = f2bf(x.y), h2 = f2bf(x.z), h3 = f2bf(x.w);
-        *reinterpret_cast<uint2*>(&Sh[d][c]) = make_uint2(pack2(h0, h1), pack2(h2, h3));
-        *reinterpret_cast<uint2*>(&Sl[d][c]) =
-            make_uint2(pack2(f2bf(x.x - bf2f(h0)), f2bf(x.y - bf2f(h1))), pack2(f2bf(x.z - bf2f(h2)), f2bf(x.w - bf2f(h3))));
+      constexpr int NS = DP * (VP / 4) / LT, B = 8;
+#pragma unroll
+      for (int n0 = 0; n0 < NS; n0 += B) {  // (NS is 4, 8 or 16)
+        float4 x[B];
+#pragma unroll
+        for (int j = 0; j < B; ++j) {
+          const int i = tid + (n0 + j) * LT, d = i / (VP / 4), c = (i % (VP / 4)) * 4;
+          x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (n0 + j < NS && d < dim && c < vdim) x[j] = *reinterpret_cast<const float4*>(S + (size_t)d * vdim + c);
+        }
+#pragma unroll
+        for (int j = 0; j < B; ++j) {
+          if (n0 + j >= NS) break;
+          const int i = tid + (n0 + j) * LT, d = i / (VP / 4), c = (i % (VP / 4)) * 4;
+          const uint32_t h0 = pack2f(x[j].x, x[j].y), h1 = pack2f(x[j].z, x[j].w);
+          *reinterpret_cast<uint2*>(&Sh[d][c]) = make_uint2(h0, h1);
+          *reinterpret_cast<uint2*>(&Sl[d][c]) =
+              make_uint2(pack2f(x[j].x - lo2f(h0), x[j].y - hi2f(h0)), pack2f(x[j].z - lo2f(h1), x[j].w - hi2f(h1)));
+        }
       }
     } else {
-      for (int i = tid; i < DP * VP; i += 128) {
+      for (int i = tid; i < DP * VP; i += LT) {
         const int d = i / VP, c = i % VP;
         const float x = d < dim && c < vdim ? S[(size_t)d * vdim + c] : 0.f;
         const bf16 hi = f2bf(x);
@@ -280,87 +335,103 @@ __global__ void __launch_bounds__(128) linear_chunk_out_kernel(const LinearAttnA
     }
   }
   __syncthreads();
-  const int warp = tid >> 5, lane = tid & 31, w0 = warp * 16;
-  if (w0 >= L) return;
+  constexpr int HB = VP / 16;  // blocks of 8 columns per half
+  const int warp = tid >> 5, lane = tid & 31, w0 = (warp & 3) * 16, vb0 = (warp >> 2) * HB;
+  const bool active = w0 < L;
   const int qr = lane >> 2, qc = (lane & 3) * 2;
   const int t0 = w0 + qr, t1 = t0 + 8;  // this thread's two rows of the chunk
-  float o[VP / 8][4];
+  float o[HB][4];
 #pragma unroll
-  for (int i = 0; i < VP / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float s[LC / 8][4];
+  for (int i = 0; i < HB; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  if (active) {
+    float s[LC / 8][4];
 #pragma unroll
-  for (int i = 0; i < LC / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    for (int i = 0; i < LC / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
-  for (int kk = 0; kk < DP / 16; ++kk) {
-    uint32_t qf[4];
-    ldmatrix_x4(qf[0], qf[1], qf[2], qf[3], smem_u32(&Qs[w0 + (lane & 15)][kk * 16 + (lane >> 4) * 8]));
+    for (int kk = 0; kk < DP / 16; ++kk) {
+      uint32_t qf[4];
+      ldmatrix_x4(qf[0], qf[1], qf[2], qf[3], smem_u32(&Qs[w0 + (lane & 15)][kk * 16 + (lane >> 4) * 8]));
 #pragma unroll
-    for (int nb = 0; nb < LC / 8; ++nb) {
-      if (nb * 8 > w0 + 15) break;  // later than every row of the warp
-      uint32_t b0, b1;
-      ldmatrix_x2(b0, b1, smem_u32(&Ks[nb * 8 + (lane & 7)][kk * 16 + ((lane >> 3) & 1) * 8]));
-      mma_bf16_16816(s[nb], qf, b0, b1);
+      for (int nb = 0; nb < LC / 8; ++nb) {
+        if (nb * 8 > w0 + 15) break;  // later than every row of the warp
+        uint32_t b0, b1;
+        ldmatrix_x2(b0, b1, smem_u32(&Ks[nb * 8 + (lane & 7)][kk * 16 + ((lane >> 3) & 1) * 8]));
+        mma_bf16_16816(s[nb], qf, b0, b1);
+      }
+#pragma unroll
+      for (int vb = 0; vb < HB; ++vb) {
+        uint32_t b0, b1;
+        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sh[kk * 16 + (lane & 15)][(vb0 + vb) * 8]));
+        mma_bf16_16816(o[vb], qf, b0, b1);
+        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sl[kk * 16 + (lane & 15)][(vb0 + vb) * 8]));
+        mma_bf16_16816(o[vb], qf, b0, b1);
+      }
+    }
+    {
+      const float e0 = pw[t0 + 1], e1 = pw[t1 + 1];
+#pragma unroll
+      for (int vb = 0; vb < HB; ++vb) o[vb][0] *= e0, o[vb][1] *= e0, o[vb][2] *= e1, o[vb][3] *= e1;
     }
 #pragma unroll
-    for (int vb = 0; vb < VP / 8; ++vb) {
-      uint32_t b0, b1;
-      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sh[kk * 16 + (lane & 15)][vb * 8]));
-      mma_bf16_16816(o[vb], qf, b0, b1);
-      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Sl[kk * 16 + (lane & 15)][vb * 8]));
-      mma_bf16_16816(o[vb], qf, b0, b1);
-    }
-  }
-  {
-    const float e0 = pw[t0 + 1], e1 = pw[t1 + 1];
+    for (int kb = 0; kb < LC / 16; ++kb) {
+      if (kb * 16 > w0 + 15) break;
+      uint32_t ph[4], pl[4];
 #pragma unroll
-    for (int vb = 0; vb < VP / 8; ++vb) o[vb][0] *= e0, o[vb][1] *= e0, o[vb][2] *= e1, o[vb][3] *= e1;
-  }
+      for (int f = 0; f < 4; ++f) {
+        const int nb = 2 * kb + (f >> 1), j = nb * 8 + qc, t = (f & 1) ? t1 : t0;
+        const float x0 = j <= t ? s[nb][(f & 1) * 2] * (a.k_scale * pw[t - j]) : 0.f;
+        const float x1 = j + 1 <= t ? s[nb][(f & 1) * 2 + 1] * (a.k_scale * pw[t - j - 1]) : 0.f;
+        ph[f] = pack2f(x0, x1);
+        pl[f] = pack2f(x0 - lo2f(ph[f]), x1 - hi2f(ph[f]));
+      }
 #pragma unroll
-  for (int kb = 0; kb < LC / 16; ++kb) {
-    if (kb * 16 > w0 + 15) break;
-    uint32_t ph[4], pl[4];
-#pragma unroll
-    for (int f = 0; f < 4; ++f) {
-      const int nb = 2 * kb + (f >> 1), j = nb * 8 + qc, t = (f & 1) ? t1 : t0;
-      const float x0 = j <= t ? s[nb][(f & 1) * 2] * (a.k_scale * pw[t - j]) : 0.f;
-      const float x1 = j + 1 <= t ? s[nb][(f & 1) * 2 + 1] * (a.k_scale * pw[t - j - 1]) : 0.f;
-      const bf16 h0 = f2bf(x0), h1 = f2bf(x1);
-      ph[f] = pack2(h0, h1);
-      pl[f] = pack2(f2bf(x0 - bf2f(h0)), f2bf(x1 - bf2f(h1)));
-    }
-#pragma unroll
-    for (int vb = 0; vb < VP / 8; ++vb) {
-      uint32_t b0, b1;
-      ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][vb * 8]));
-      mma_bf16_16816(o[vb], ph, b0, b1);
-      mma_bf16_16816(o[vb], pl, b0, b1);
+      for (int vb = 0; vb < HB; ++vb) {
+        uint32_t b0, b1;
+        ldmatrix_x2_trans_la(b0, b1, smem_u32(&Vs[kb * 16 + (lane & 15)][(vb0 + vb) * 8]));
+        mma_bf16_16816(o[vb], ph, b0, b1);
+        mma_bf16_16816(o[vb], pl, b0, b1);
+      }
     }
   }
   const bool v0 = t0 < L, v1 = t1 < L;
   float n0 = 1.f, n1 = 1.f;
-  if (a.norm_gate) {  // a row of a head lies in the four threads of a quad
+  if (a.norm_gate) {  // a row of a head lies in a quad of each of the two warps that share its rows
     float q0 = 0.f, q1 = 0.f;
 #pragma unroll
-    for (int vb = 0; vb < VP / 8; ++vb) q0 = fmaf(o[vb][0], o[vb][0], fmaf(o[vb][1], o[vb][1], q0)), q1 = fmaf(o[vb][2], o[vb][2], fmaf(o[vb][3], o[vb][3], q1));
+    for (int vb = 0; vb < HB; ++vb) q0 = fmaf(o[vb][0], o[vb][0], fmaf(o[vb][1], o[vb][1], q0)), q1 = fmaf(o[vb][2], o[vb][2], fmaf(o[vb][3], o[vb][3], q1));
     q0 += __shfl_xor_sync(0xffffffffu, q0, 1), q1 += __shfl_xor_sync(0xffffffffu, q1, 1);
     q0 += __shfl_xor_sync(0xffffffffu, q0, 2), q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
-    n0 = 1.0f / sqrtf(q0 / (float)vdim + a.eps), n1 = 1.0f / sqrtf(q1 / (float)vdim + a.eps);
+    if ((lane & 3) == 0) sq[warp >> 2][t0] = q0, sq[warp >> 2][t1] = q1;
+    __syncthreads();
+    n0 = 1.0f / sqrtf((sq[0][t0] + sq[1][t0]) / (float)vdim + a.eps), n1 = 1.0f / sqrtf((sq[0][t1] + sq[1][t1]) / (float)vdim + a.eps);
   }
-#pragma unroll
-  for (int vb = 0; vb < VP / 8; ++vb)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int c = vb * 8 + qc + e;
-      if (c >= vdim) continue;
-      const size_t ra = (size_t)(row0 + t0), rb = (size_t)(row0 + t1);
-      if (a.norm_gate) {
-        if (v0) a.out_bf[ra * a.ldo_bf + h * vdim + c] = f2bf(o[vb][e] * n0 * silu_f(bf2f(a.g_bf[ra * a.ld_bf + h * vdim + c])));
-        if (v1) a.out_bf[rb * a.ldo_bf + h * vdim + c] = f2bf(o[vb][2 + e] * n1 * silu_f(bf2f(a.g_bf[rb * a.ld_bf + h * vdim + c])));
+  const bool even = vdim % 2 == 0 && (a.norm_gate ? a.ldo_bf % 2 == 0 && a.ld_bf % 2 == 0 && ((reinterpret_cast<uintptr_t>(a.out_bf) | reinterpret_cast<uintptr_t>(a.g_bf)) & 3) == 0
+                                                  : a.ldo % 2 == 0);
+  auto put = [&](int t, int c, float x, float y, float n) {  // columns c and c + 1 of row t
+    const size_t r = (size_t)(row0 + t);
+    const int hc = h * vdim + c;
+    if (a.norm_gate) {
+      if (even) {
+        const uint32_t g = *reinterpret_cast<const uint32_t*>(a.g_bf + r * a.ld_bf + hc);
+        *reinterpret_cast<uint32_t*>(a.out_bf + r * a.ldo_bf + hc) = pack2f(x * n * silu_f(lo2f(g)), y * n * silu_f(hi2f(g)));
       } else {
-        if (v0) a.out[ra * a.ldo + h * vdim + c] = o[vb][e];
-        if (v1) a.out[rb * a.ldo + h * vdim + c] = o[vb][2 + e];
+        a.out_bf[r * a.ldo_bf + hc] = f2bf(x * n * silu_f(bf2f(a.g_bf[r * a.ld_bf + hc])));
+        if (c + 1 < vdim) a.out_bf[r * a.ldo_bf + hc + 1] = f2bf(y * n * silu_f(bf2f(a.g_bf[r * a.ld_bf + hc + 1])));
       }
+    } else if (even) {
+      *reinterpret_cast<float2*>(a.out + r * a.ldo + hc) = make_float2(x, y);
+    } else {
+      a.out[r * a.ldo + hc] = x;
+      if (c + 1 < vdim) a.out[r * a.ldo + hc + 1] = y;
     }
+  };
+#pragma unroll
+  for (int vb = 0; vb < HB; ++vb) {
+    const int c = (vb0 + vb) * 8 + qc;
+    if (c >= vdim) continue;
+    if (v0) put(t0, c, o[vb][0], o[vb][1], n0);
+    if (v1) put(t1, c, o[vb][2], o[vb][3], n1);
+  }
 }
 
 template <int DP, int VP>
@@ -375,11 +446,11 @@ cudaError_t launch_chunked(const LinearAttnArgs& a, cudaStream_t st) {
     if ((r = cudaFuncSetAttribute(linear_chunk_out_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2)) != cudaSuccess) return r;
     once.done();
   }
-  cudaError_t r = launch_k(linear_chunk_state_kernel<DP, VP>, dim3(chunks, a.heads), dim3(128), s1, st, a);
+  cudaError_t r = launch_k(linear_chunk_state_kernel<DP, VP>, dim3(chunks, a.heads), dim3(LT), s1, st, a);
   if (r != cudaSuccess) return r;
   const int per = a.heads * a.dim * a.vdim;
   if ((r = launch_k(linear_carry_kernel, dim3((per + 255) / 256, a.n_seg), dim3(256), 0, st, a)) != cudaSuccess) return r;
-  return launch_k(linear_chunk_out_kernel<DP, VP>, dim3(chunks, a.heads), dim3(128), s2, st, a);
+  return launch_k(linear_chunk_out_kernel<DP, VP>, dim3(chunks, a.heads), dim3(LT), s2, st, a);
 }
 
 }  // namespace
