@@ -726,14 +726,10 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
       f0 = l0 > 0.f ? 1.0f / l0 : 0.f;
       f1 = l1 > 0.f ? 1.0f / l1 : 0.f;
     }
-    if (a.talk) {  // the heads are mixed by gqa_talk_finish_kernel
+    if (a.talk) {  // the heads are mixed by gqa_talk_mix_kernel
       const size_t rs = (size_t)(vcols + 2);
       float* w0 = a.ws + ((size_t)(row0 + wrow + qr) * a.heads + h) * rs;
       float* w1 = w0 + (size_t)8 * a.heads * rs;
-      if (blockIdx.z == 0 && (lane & 3) == 0) {
-        if (rv0) w0[0] = 0.f, w0[1] = 1.f;
-        if (rv1) w1[0] = 0.f, w1[1] = 1.f;
-      }
 #pragma unroll
       for (int vb = 0; vb < VP / 8; ++vb) {
         const int c = vb * 8 + qc;
@@ -888,10 +884,10 @@ __global__ void __launch_bounds__(128) gqa_finish_kernel(const GqaAttnArgs a, in
   for (int c = threadIdx.x; c < vd; c += blockDim.x) out[c] = o[c] * rstd;
 }
 
-// CTA of `rows` rows: merges the key splits of every head's attended values and mixes the heads.  Thread = (kv head c, value
+// CTA per row: merges the key splits of every head's attended values and mixes the heads.  Thread = (kv head c, value
 // column): out[h] = sum_g talk[h, g] a_g[c] for the heads h of kv head c, eight of them at a time.  Shared memory: the mix
 // [g][h] as fp32 | split weights [heads][n_splits]
-__global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits, int rows) {
+__global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits) {
   extern __shared__ float tf_smem[];
   pdl_wait();
   pdl_trigger();
@@ -900,9 +896,9 @@ __global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs 
   float* tk = tf_smem;
   float* wt = tk + H * H;
   for (int i = threadIdx.x; i < H * H; i += blockDim.x) tk[(i % H) * H + i / H] = bf2f(a.talk[i]);
-  for (int r = blockIdx.x * rows; r < min(a.n, (int)(blockIdx.x + 1) * rows); ++r) {
+  {
+    const int r = blockIdx.x;
     const float* rec = a.ws + (size_t)r * H * n_splits * rs;
-    __syncthreads();
     for (int g = threadIdx.x; g < H; g += blockDim.x) {
       const float* rg = rec + (size_t)g * n_splits * rs;
       float M = -INFINITY, L = 0.f;
@@ -951,6 +947,54 @@ __global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs 
   }
 }
 
+// Single normalised record per (row, head) (the prompt kernels): no split weights, up to 16 heads' values in flight per thread
+__global__ void __launch_bounds__(256) gqa_talk_mix_kernel(const GqaAttnArgs a) {
+  extern __shared__ float tf_smem[];  // the mix [g][h]
+  pdl_wait();
+  pdl_trigger();
+  const int vd = a.vdim, H = a.heads, hpg = H / a.kv_heads, ncol = a.kv_heads * vd;
+  const size_t rs = (size_t)ncol + 2;
+  const size_t r = blockIdx.x;
+  const float* rec = a.ws + r * H * rs + 2;
+  float v[16];
+  auto load = [&](int i, int g0) {
+#pragma unroll
+    for (int u = 0; u < 16; ++u) v[u] = g0 + u < H && i < ncol ? rec[(size_t)(g0 + u) * rs + i] : 0.f;
+  };
+  load(threadIdx.x, 0);  // on their way while the mix is staged
+  for (int i = threadIdx.x; i < H * H; i += blockDim.x) {
+    const int h = i / H;
+    tf_smem[(i - h * H) * H + h] = bf2f(a.talk[i]);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
+    const int c = i / vd, col = i - c * vd;
+    for (int h0 = 0; h0 < hpg; h0 += 8) {
+      float acc[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) acc[k] = 0.f;
+      for (int g0 = 0; g0 < H; g0 += 16) {
+        if (i != threadIdx.x || h0 || g0) load(i, g0);
+#pragma unroll
+        for (int u = 0; u < 16; ++u) {
+          if (g0 + u >= H) break;
+          const float* t = tf_smem + (g0 + u) * H + c * hpg + h0;
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+            if (h0 + k < hpg) acc[k] = fmaf(t[k], v[u], acc[k]);
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        if (h0 + k >= hpg) break;
+        const size_t o = (size_t)(c * hpg + h0 + k) * vd + col;
+        if (a.out_bf) a.out_bf[r * a.ldo_bf + o] = f2bf(acc[k]);
+        else a.out[r * a.ldo + o] = acc[k];
+      }
+    }
+  }
+}
+
 }  // namespace
 
 static size_t talk_smem(const TalkQueries& t) { return ((size_t)t.heads * t.dim + (size_t)t.heads * t.heads) * sizeof(float); }
@@ -994,15 +1038,17 @@ cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* 
   return launch_k(kv_pool_rows_kernel, dim3((n + POOL_ROWS - 1) / POOL_ROWS), dim3(256), 0, st, c, pos, slot, block_table, max_pages, n);
 }
 
+// splits 0: the records are normalised, one per (row, head)
 static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStream_t st) {
   const size_t smem = ((size_t)a.heads * splits + (size_t)a.heads * a.heads) * sizeof(float);
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return cudaErrorInvalidValue;
-    cudaError_t r = cudaFuncSetAttribute(gqa_talk_finish_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t r = cudaFuncSetAttribute(splits ? (const void*)gqa_talk_finish_kernel : (const void*)gqa_talk_mix_kernel,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (r != cudaSuccess) return r;
   }
-  const int rows = a.n >= 1024 ? 2 : 1;
-  return launch_k(gqa_talk_finish_kernel, dim3((a.n + rows - 1) / rows), dim3(256), smem, st, a, splits, rows);
+  if (splits == 0) return launch_k(gqa_talk_mix_kernel, dim3(a.n), dim3(256), smem, st, a);
+  return launch_k(gqa_talk_finish_kernel, dim3(a.n), dim3(256), smem, st, a, splits);
 }
 
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches) {
@@ -1020,7 +1066,7 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
   if (tc_on && gqa_talk_tc_fits(a)) {
     if (n_launches) *n_launches = 2;
     cudaError_t r = launch_gqa_talk_tc(a, st);
-    return r != cudaSuccess ? r : launch_talk_finish(a, 1, st);
+    return r != cudaSuccess ? r : launch_talk_finish(a, 0, st);
   }
   // prompt portions over a bf16 cache: the tensor-core kernel (one launch, no workspace); QIE_ATTN_MMA=0 keeps the per-row kernel (A/B)
   static const bool mma_on = [] { const char* v = getenv("QIE_ATTN_MMA"); return !(v && v[0] == '0'); }();
@@ -1032,7 +1078,7 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
     else if (a.dim <= 64) r = launch_prefill_mma_v<64>(a, a.seg_start, a.seg_slot, a.n_seg, st);
     else r = launch_prefill_mma_v<128>(a, a.seg_start, a.seg_slot, a.n_seg, st);
     if (r != cudaSuccess || !a.talk) return r;
-    return launch_talk_finish(a, 1, st);
+    return launch_talk_finish(a, 0, st);
   }
   if (a.maps < 1 || a.maps > 2 || a.heads % a.kv_heads || (a.finish == 2 && a.maps != 2) || (!a.talk && a.maps * a.vdim > ATHREADS * AMAXACC))
     return cudaErrorInvalidValue;

@@ -1,15 +1,16 @@
 // attn_gqa_tc.cu -- prompt attention over paged bf16 key/value rows on the 5th-gen tensor cores (tcgen05 + TMEM), for grouped
 // queries whose softmax weights are mixed over the heads (GqaAttnArgs::talk), a sliding window or a causal mask, and pooled
 // rows.  Mixing after the softmax is linear, so every head attends to the values of ALL kv heads -- one product with up to
-// 256 value columns, which is what the tensor cores are good at -- and gqa_talk_finish_kernel mixes the results.
+// 256 value columns, which is what the tensor cores are good at -- and gqa_talk_mix_kernel mixes the results.
 //
 // A CTA owns 128 consecutive rows of one segment, one query head and one chunk of value columns, and walks tiles of 64 keys: first
 // the tiles of pooled rows that some row sees, then the tokens from the first window's lower edge on.  20 warps:
 //   the last 3  bring the tile's key and value rows into the swizzled operand layout, a ring of stages: token rows by TMA boxes of
-//               a page, pooled rows (and token rows of pages that do not divide a tile) by cp.async
-//   warp 16     issues the products: S = Q K^T (128 x 64, two TMEM buffers, one tile ahead of the softmax) and O += P V (TMEM)
-//   warps 0-15  softmax, four threads per row: S from TMEM, mask, reference maximum, weights as bf16 hi + lo pairs into shared
-//               memory (two buffers, two products per tile, so a weight keeps ~16 bits)
+//               a page, pooled rows (and token rows of pages that do not divide a tile) by cp.async; the first pooled tiles are
+//               copied by all warps before they take their roles
+//   warp 16     issues the products: S = Q K^T (128 x 64, two TMEM buffers, one tile ahead of the softmax) and O += P V
+//   warps 0-15  softmax, four threads per row: S from TMEM, mask, reference maximum, weights as bf16 hi + lo pairs into TMEM (two
+//               buffers; the second product takes its A operand from there), two products per tile, so a weight keeps ~16 bits
 // O stays in TMEM over all tiles.  Instead of scaling it whenever a row's maximum grows, a row keeps its reference maximum until a
 // score exceeds it by RESCALE (weights then stay below 2^RESCALE); only then the warp that owns the row scales its part of O.
 // Every wait has a limit; when one runs out the CTA finishes without waiting and marks its results as not a number.
@@ -29,6 +30,7 @@ namespace {
 constexpr int TQ = 128, TK = 64;
 constexpr int NSOFT = 512, NLOAD = 96, MMA_WARP = NSOFT / 32, NTHR = NSOFT + 32 + NLOAD;
 constexpr int LROWS = NLOAD / 8, LPASS = (TK + LROWS - 1) / LROWS;  // rows a pass of the copying threads covers
+constexpr int MAX_ST = 6, TURN = 33;                                // stages at most; row pitch of the turned results
 constexpr int KBLK = TK * 128;   // [64 keys][64 columns] bf16, 8-row swizzle atoms: 8 KiB
 constexpr int QBLK = TQ * 128;   // [128 rows][64 columns]: 16 KiB
 constexpr float RESCALE = 8.0f;  // in powers of two
@@ -76,6 +78,20 @@ __device__ __forceinline__ void tmem_st16_tc(uint32_t taddr, const uint32_t (&r)
       "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
       : "memory");
 }
+__device__ __forceinline__ void tmem_st8_tc(uint32_t taddr, const uint32_t (&r)[8]) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%8], {%0,%1,%2,%3,%4,%5,%6,%7};" ::"r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]),
+               "r"(r[6]), "r"(r[7]), "r"(taddr)
+               : "memory");
+}
+// A from TMEM: row = lane, a 32-bit column holds two consecutive k
+__device__ __forceinline__ void umma_ts_tc(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(d_tmem), "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(acc)
+      : "memory");
+}
 // K-major operand, SWIZZLE_128B, 8-row atoms 1024 bytes apart
 __device__ __forceinline__ uint64_t desc_k_tc(uint32_t smem_addr) {
   return (uint64_t)((smem_addr >> 4) & 0x3FFF) | (uint64_t)1 << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
@@ -97,18 +113,28 @@ __device__ __forceinline__ float ex2_tc(float x) {  // 2^x; 2^(-inf) = 0
 __device__ __forceinline__ uint32_t blk_off(int r, int ch) { return (uint32_t)(r * 128 + ((ch ^ (r & 7)) << 4)); }
 
 struct TcLayout {  // byte offsets from the 1024-aligned base
-  int dblk, vblk, nst, q, p, st, stage, bar, total;
+  int dblk, vblk, nst, q, st, stage, bar, total;
 };
 __host__ __device__ inline TcLayout tc_layout(int dblk, int vblk, int nst) {
   TcLayout l;
   l.dblk = dblk, l.vblk = vblk, l.nst = nst;
   l.q = 0;
-  l.p = l.q + dblk * QBLK;        // P [buffer 2][hi, lo]
-  l.st = l.p + 4 * QBLK;          // stages: K blocks | V blocks
+  l.st = l.q + dblk * QBLK;       // stages: K blocks | V blocks; at the end the results are turned around there
   l.stage = (dblk + vblk) * KBLK;
-  l.bar = l.st + nst * l.stage;   // mbarriers, flags, row maxima
+  l.bar = l.st + (nst * l.stage > NSOFT * TURN * 4 ? nst * l.stage : (NSOFT * TURN * 4 + 1023) / 1024 * 1024);  // mbarriers, flags, row maxima
   l.total = l.bar + 256 + 8 * TQ * 4;
   return l;
+}
+
+// chunk ch (16 bytes) of every 64-column block of one key row and its values -> row r of the stage at `base`; null: zeros
+__device__ __forceinline__ void copy_row(const bf16* row, size_t koff, size_t voff, uint32_t base, int r, int ch, int dblk, int vblk, int dim, int nv) {
+  for (int b = 0; b < dblk + vblk; ++b) {
+    const bool isv = b >= dblk;
+    const int c = (isv ? b - dblk : b) * 64 + ch * 8;
+    const uint32_t dst = base + b * KBLK + blk_off(r, ch);
+    if (row && c < (isv ? nv : dim)) cp_async16(dst, row + (isv ? voff : koff) + c);
+    else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0u) : "memory");
+  }
 }
 
 __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc,
@@ -120,7 +146,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
-    int left = blockIdx.y, found = 0;
+    int left = gridDim.y - 1 - blockIdx.y, found = 0;  // late tiles of a segment see more keys: they start first
     for (int s = 0; s < a.n_seg && !found; ++s) {
       const int r0 = a.seg_start[s], len = a.seg_start[s + 1] - r0, nt = (len + TQ - 1) / TQ;
       if (left < nt) info[0] = r0 + left * TQ, info[1] = min(TQ, len - left * TQ), info[2] = a.seg_slot[s], found = 1;
@@ -137,7 +163,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   const uint32_t s0 = (smem_u32(smem_raw) + 1023u) & ~1023u;
   unsigned char* sg = smem_raw + (s0 - smem_u32(smem_raw));
   const uint32_t b0 = s0 + L.bar;
-  const uint32_t bar_full = b0, bar_empty = b0 + 32, bar_s = b0 + 64, bar_p = b0 + 80, bar_o = b0 + 96, tslot = b0 + 112;
+  const uint32_t bar_full = b0, bar_empty = b0 + 8 * MAX_ST, bar_s = b0 + 16 * MAX_ST, bar_p = bar_s + 16, bar_o = bar_s + 32, tslot = bar_s + 48;
   float* xmax = reinterpret_cast<float*>(sg + L.bar + 256);  // [tile parity][quarter][row]; the sums use the parity that the last tile did not
   const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), dim = a.dim;
   const int vcols = a.kv_heads * a.vdim, col0 = blockIdx.z * vc, nv = min(vc, vcols - col0);
@@ -146,7 +172,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   const int nbmax = a.c.block > 0 ? pooled_seen(pmax, a.window, a.c.block) : 0, npt = (nbmax + TK - 1) / TK;
   const int tt0 = lo_min / TK, nt = npt + pmax / TK - tt0 + 1;  // tiles: npt of pooled rows, then tokens from tile tt0 on
   if (tid == 0) {
-    for (int i = 0; i < nst; ++i) mbar_init_tc(bar_full + 8 * i, NLOAD), mbar_init_tc(bar_empty + 8 * i, 1);
+    for (int i = 0; i < nst; ++i) mbar_init_tc(bar_full + 8 * i, NLOAD / 32), mbar_init_tc(bar_empty + 8 * i, 1);
     for (int i = 0; i < 2; ++i) mbar_init_tc(bar_s + 8 * i, 1), mbar_init_tc(bar_p + 8 * i, NSOFT), mbar_init_tc(bar_o + 8 * i, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -154,38 +180,65 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tslot), "r"(512u) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
-  // Q rows as bf16, zeros beyond the head size and the last row
+  // the first tiles of pooled rows, as many as there are stages: thread = (row, 16-byte chunk of a block)
+  const int npre = min(npt, nst);
+  const size_t koff = (size_t)g * dim, voff = (size_t)a.c.kw + col0;
+  for (int t = 0; t < npre; ++t) {
+    const int r = tid >> 3, ch = tid & 7, b = t * TK + r;
+    if (r >= TK) break;
+    const bf16* row = b < nbmax ? reinterpret_cast<const bf16*>(kv_pool_ptr(a.c, a.block_table, a.max_pages, slot, b)) : nullptr;
+    copy_row(row, koff, voff, s0 + L.st + t * L.stage, r, ch, dblk, vblk, dim, nv);
+  }
+  cp_async_commit();
+  // Q rows as bf16, zeros beyond the head size and the last row (dim is a multiple of 8)
+  const bool q16 = a.ldq % 4 == 0 && (reinterpret_cast<uintptr_t>(a.q) & 15) == 0;
   for (int i = tid; i < TQ * dblk * 8; i += NTHR) {
     const int r = i / (dblk * 8), c = (i - r * dblk * 8) * 8;
-    uint32_t w[4] = {0u, 0u, 0u, 0u};
-    if (r < nrows) {
+    uint4 w = make_uint4(0u, 0u, 0u, 0u);
+    if (r < nrows && c < dim) {
       const float* q = a.q + (size_t)(row0 + r) * a.ldq + (size_t)h * dim + c;
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (c + 2 * e < dim) w[e] = pack2(f2bf(q[2 * e]), f2bf(q[2 * e + 1]));  // dim is a multiple of 8
+      if (q16) {
+        const float4 x = *reinterpret_cast<const float4*>(q), y = *reinterpret_cast<const float4*>(q + 4);
+        w = make_uint4(pack2f(x.x, x.y), pack2f(x.z, x.w), pack2f(y.x, y.y), pack2f(y.z, y.w));
+      } else {
+        w = make_uint4(pack2f(q[0], q[1]), pack2f(q[2], q[3]), pack2f(q[4], q[5]), pack2f(q[6], q[7]));
+      }
     }
-    *reinterpret_cast<uint4*>(sg + L.q + (c >> 6) * QBLK + blk_off(r, (c >> 3) & 7)) = make_uint4(w[0], w[1], w[2], w[3]);
+    *reinterpret_cast<uint4*>(sg + L.q + (c >> 6) * QBLK + blk_off(r, (c >> 3) & 7)) = w;
   }
+  cp_async_wait<0>();
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   uint32_t tmem;
   asm volatile("ld.shared.b32 %0, [%1];" : "=r"(tmem) : "r"(tslot));
-  const uint32_t t_o = tmem + 128;  // S: columns 0..127 (two buffers), O: 128 ..
+  const uint32_t t_o = tmem + 128, t_p = tmem + 384;  // S: columns 0..127 (two buffers), O: 128 .. 383, P: 384 .. (two buffers of hi | lo)
   const int vcp = vblk * 64;        // columns of O
 
   if (warp > MMA_WARP) {
     // ---- copies
-    const int lt = tid - (NSOFT + 32), ch = lt & 7, rr = lt >> 3;  // chunk of a 64-column block, rows rr + LROWS k
-    const size_t koff = (size_t)g * dim, voff = (size_t)a.c.kw + col0;
+    const int lt = tid - (NSOFT + 32), lw = warp - MMA_WARP - 1, ch = lt & 7, rr = lt >> 3;  // cp.async: chunk of a block, rows rr + LROWS k
+    // TMA: boxes of up to 64 rows of a page and 64 columns, box number 3 * lane + lw.  Rows behind the last position and columns behind
+    // a part are other cache contents: finite numbers that meet zero weights, zero queries or columns nobody reads.
+    const int br = min(a.c.page_size, TK), nbx = TK / br, boxes = nbx * (dblk + vblk), bi = 3 * lane + lw, bb = bi / nbx, pg = bi - bb * nbx;
+    const int bx = bb < dblk ? g * dim + bb * 64 : a.c.kw + col0 + (bb - dblk) * 64;
+    const uint32_t bdst = (uint32_t)(bb * KBLK + pg * br * 128), wbytes = (uint32_t)((boxes - lw + 2) / 3 * br * 128);
+    const int* bt = a.block_table + (size_t)slot * a.max_pages;
+    auto page_of = [&](int t) { return bt[min((tt0 + t - npt) * TK + pg * br, pmax) / a.c.page_size]; };
     auto announce = [&](int t) {  // the copies of tile t are complete: visible to the tensor core
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      mbar_arrive_tc(bar_full + 8 * (t % nst));
+      __syncwarp();
+      if (lane == 0) mbar_arrive_tc(bar_full + 8 * (t % nst));
     };
+    int page = use_tma && bi < boxes && npt < nt ? page_of(npt) : 0;
     bool prev_cp = false;  // the tile before was copied by cp.async and is not announced yet
     for (int t = 0; t < nt; ++t) {
       const int s = t % nst;
+      if (t < npre) {  // copied above
+        if (lane == 0) mbar_arrive_tc(bar_full + 8 * s);
+        continue;
+      }
       const bool tma = use_tma && t >= npt;
       if (prev_cp && (nst == 2 || tma)) {  // (two stages: the stage that this tile waits for is only given back behind the scores of the tile before)
         cp_async_wait<0>();
@@ -194,21 +247,14 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
       }
       if (t >= nst) mbar_wait_tc(bar_empty + 8 * s, (uint32_t)((t / nst - 1) & 1), dead);
       const uint32_t base = s0 + L.st + s * L.stage;
-      if (tma) {  // boxes of up to 64 rows of a page and 64 columns; rows behind the last position and columns behind a part are
-                  // other cache contents, finite numbers that meet zero weights, zero queries or columns nobody reads
-        if (lt == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar_full + 8 * s), "r"((uint32_t)L.stage) : "memory");
-        else mbar_arrive_tc(bar_full + 8 * s);
-        if (warp == MMA_WARP + 1) {
-          __syncwarp();
-          const int br = min(a.c.page_size, TK), nbx = TK / br, j0 = (tt0 + t - npt) * TK;
-          for (int i = lane; i < nbx * (dblk + vblk); i += 32) {
-            const int b = i / nbx, pg = i - b * nbx;
-            const int x = b < dblk ? g * dim + b * 64 : a.c.kw + col0 + (b - dblk) * 64;
-            const int page = a.block_table[(size_t)slot * a.max_pages + min(j0 + pg * br, pmax) / a.c.page_size];
-            asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
-                         ::"r"(base + b * KBLK + pg * br * 128), "l"(&rows_map), "r"(bar_full + 8 * s), "r"(x), "r"(j0 % a.c.page_size), "r"(page)
-                         : "memory");
-          }
+      if (tma) {
+        if (lane == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar_full + 8 * s), "r"(wbytes) : "memory");
+        __syncwarp();
+        if (bi < boxes) {
+          asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+                       ::"r"(base + bdst), "l"(&rows_map), "r"(bar_full + 8 * s), "r"(bx), "r"((tt0 + t - npt) * TK % a.c.page_size), "r"(page)
+                       : "memory");
+          if (t + 1 < nt) page = page_of(t + 1);
         }
         continue;
       }
@@ -225,19 +271,9 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
         }
         rowp[k] = reinterpret_cast<const bf16*>(p);
       }
-      for (int b = 0; b < dblk + vblk; ++b) {
-        const bool isv = b >= dblk;
-        const int c = (isv ? b - dblk : b) * 64 + ch * 8;
-        const bool in = c < (isv ? nv : dim);
 #pragma unroll
-        for (int k = 0; k < LPASS; ++k) {
-          const int r = rr + LROWS * k;
-          if (r >= TK) break;
-          const uint32_t dst = base + b * KBLK + blk_off(r, ch);
-          if (in && rowp[k]) cp_async16(dst, rowp[k] + (isv ? voff : koff) + c);
-          else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0u) : "memory");
-        }
-      }
+      for (int k = 0; k < LPASS; ++k)
+        if (rr + LROWS * k < TK) copy_row(rowp[k], koff, voff, base, rr + LROWS * k, ch, dblk, vblk, dim, nv);
       cp_async_commit();
       if (prev_cp) {
         cp_async_wait<1>();
@@ -268,10 +304,10 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
         if (t + 1 < nt) issue_s(t + 1);  // its buffer was read before the weights of tile t - 1 were announced
         mbar_wait_tc(bar_p + 8 * (t & 1), (uint32_t)((t >> 1) & 1), dead);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t vb = s0 + L.st + (t % nst) * L.stage + dblk * KBLK, ph = s0 + L.p + (t & 1) * 2 * QBLK;
+        const uint32_t vb = s0 + L.st + (t % nst) * L.stage + dblk * KBLK, ph = t_p + (uint32_t)((t & 1) * TK);
         for (int part = 0; part < 2; ++part)  // hi, lo
           for (int kk = 0; kk < TK / 16; ++kk)
-            umma_tc(t_o, desc_k_tc(ph + part * QBLK + kk * 32), desc_mn_tc(vb + kk * 16 * 128), id_o, t > 0 || part > 0 || kk > 0);
+            umma_ts_tc(t_o, ph + (uint32_t)(part * (TK / 2) + kk * 8), desc_mn_tc(vb + kk * 16 * 128), id_o, t > 0 || part > 0 || kk > 0);
         umma_commit_tc(bar_empty + 8 * (t % nst));
         umma_commit_tc(bar_o + 8 * (t & 1));
       }
@@ -337,15 +373,11 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
       }
       l_run += rs;
       if (t >= 2) mbar_wait_tc(bar_o + 8 * (t & 1), (uint32_t)(((t >> 1) - 1) & 1), dead);  // the product that read this P buffer
-      const uint32_t pd = s0 + L.p + (t & 1) * 2 * QBLK;
-#pragma unroll
-      for (int q8 = 0; q8 < 2; ++q8) {
-        const uint32_t o = blk_off(row, 2 * qt + q8);
-        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + o), "r"(hi[4 * q8]), "r"(hi[4 * q8 + 1]), "r"(hi[4 * q8 + 2]), "r"(hi[4 * q8 + 3]) : "memory");
-        asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(pd + QBLK + o), "r"(lo[4 * q8]), "r"(lo[4 * q8 + 1]), "r"(lo[4 * q8 + 2]), "r"(lo[4 * q8 + 3]) : "memory");
-      }
+      const uint32_t pd = t_p + lane_addr + (uint32_t)((t & 1) * TK + 8 * qt);
+      tmem_st8_tc(pd, hi);
+      tmem_st8_tc(pd + TK / 2, lo);
+      asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       mbar_arrive_tc(bar_p + 8 * (t & 1));
     }
     mbar_wait_tc(bar_o + 8 * ((nt - 1) & 1), (uint32_t)(((nt - 1) >> 1) & 1), dead);
@@ -359,19 +391,21 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
     float* rec = a.ws + ((size_t)(row0 + (warp & 3) * 32) * a.heads + h) * rs_rec;  // record of the warp's first row
     const size_t row_step = (size_t)a.heads * rs_rec;
     const int wrows = min(32, nrows - (warp & 3) * 32);
-    if (lane < wrows && qt == 0 && blockIdx.z == 0) rec[lane * row_step] = 0.f, rec[lane * row_step + 1] = 1.f;
-    float* tr = reinterpret_cast<float*>(sg + L.p) + warp * (32 * 17);  // every product is done: P is free to turn the rows around
-    for (int c = oc0; c < oc1; c += 16) {
+    float* tr = reinterpret_cast<float*>(sg + L.st) + warp * (32 * TURN);  // every product is done: the stages are free to turn the rows around
+    for (int c = oc0; c < oc1; c += 32) {
+      const int cw = min(32, oc1 - c);  // 32 or 16 columns
       uint32_t o[16];
-      tmem_ld16_tc(t_o + lane_addr + c, o);
-      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       __syncwarp();
+      for (int u = 0; u < cw; u += 16) {
+        tmem_ld16_tc(t_o + lane_addr + c + u, o);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-      for (int j = 0; j < 16; ++j) tr[lane * 17 + j] = __uint_as_float(o[j]) * inv;
+        for (int j = 0; j < 16; ++j) tr[lane * TURN + u + j] = __uint_as_float(o[j]) * inv;
+      }
       __syncwarp();
-      const int cc = c + (lane & 15);
+      const int x = lane & (cw - 1), cc = c + x, rstep = 32 / cw;
       if (cc < nv)
-        for (int i = lane >> 4; i < wrows; i += 2) rec[i * row_step + 2 + col0 + cc] = tr[i * 17 + (lane & 15)];
+        for (int i = lane / cw; i < wrows; i += rstep) rec[i * row_step + 2 + col0 + cc] = tr[i * TURN + x];
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -394,7 +428,8 @@ TcPlan tc_plan(const GqaAttnArgs& a) {
   p.nvc = (vcols + 255) / 256;
   p.vc = ((vcols + p.nvc - 1) / p.nvc + 7) / 8 * 8;
   p.vblk = (p.vc + 63) / 64;
-  p.nst = tc_layout(p.dblk, p.vblk, 3).total + 1024 <= SMEM_MAX ? 3 : 2;
+  p.nst = MAX_ST;
+  while (p.nst > 2 && tc_layout(p.dblk, p.vblk, p.nst).total + 1024 > SMEM_MAX) --p.nst;
   p.smem = (size_t)tc_layout(p.dblk, p.vblk, p.nst).total + 1024;
   return p;
 }

@@ -186,7 +186,7 @@ struct GqaAttnArgs {
 inline size_t gqa_ws_floats(int n, int heads, int maps, int vdim) { return (size_t)n * heads * maps * (vdim + 2); }
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches = nullptr);
 // the tcgen05 form of a prompt portion's attention with `talk` (attn_gqa_tc.cu), without the mix of the heads: the normalised result
-// of every head over the values of all kv heads goes to its workspace record (max 0, sum 1); launch_gqa_attention picks it
+// of every head over the values of all kv heads goes to its workspace record; launch_gqa_attention picks it
 bool gqa_talk_tc_fits(const GqaAttnArgs& a);
 cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st);
 
