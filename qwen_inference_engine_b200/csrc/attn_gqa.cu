@@ -884,66 +884,41 @@ __global__ void __launch_bounds__(128) gqa_finish_kernel(const GqaAttnArgs a, in
   for (int c = threadIdx.x; c < vd; c += blockDim.x) out[c] = o[c] * rstd;
 }
 
-// CTA per row: merges the key splits of every head's attended values and mixes the heads.  Thread = (kv head c, value
-// column): out[h] = sum_g talk[h, g] a_g[c] for the heads h of kv head c, eight of them at a time.  Shared memory: the mix
-// [g][h] as fp32 | split weights [heads][n_splits]
+// CTA (row, block of 32 value columns): merges the key splits of every head's attended values, then mixes the heads.  A warp
+// takes the heads warp, warp + 8, ...: its lanes hold the weights of the head's splits (at most 32) and then one column
+// each.  Shared memory: the mix [heads][heads] as bf16 values in fp32 | attended values [heads][32]
 __global__ void __launch_bounds__(256) gqa_talk_finish_kernel(const GqaAttnArgs a, int n_splits) {
   extern __shared__ float tf_smem[];
   pdl_wait();
   pdl_trigger();
   const int vd = a.vdim, H = a.heads, hpg = H / a.kv_heads, ncol = a.kv_heads * vd;
-  const size_t rs = (size_t)ncol + 2;
+  const size_t rs = (size_t)ncol + 2, r = blockIdx.x;
   float* tk = tf_smem;
-  float* wt = tk + H * H;
-  for (int i = threadIdx.x; i < H * H; i += blockDim.x) tk[(i % H) * H + i / H] = bf2f(a.talk[i]);
-  {
-    const int r = blockIdx.x;
-    const float* rec = a.ws + (size_t)r * H * n_splits * rs;
-    for (int g = threadIdx.x; g < H; g += blockDim.x) {
-      const float* rg = rec + (size_t)g * n_splits * rs;
-      float M = -INFINITY, L = 0.f;
-      for (int s = 0; s < n_splits; ++s) M = fmaxf(M, rg[s * rs]);
-      for (int s = 0; s < n_splits; ++s) {
-        const float ms = rg[s * rs], w = ms > -INFINITY ? expf(ms - M) : 0.f;
-        wt[g * n_splits + s] = w;
-        L = fmaf(rg[s * rs + 1], w, L);
-      }
-      for (int s = 0; s < n_splits; ++s) wt[g * n_splits + s] /= L;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
-      const int c = i / vd, col = i - c * vd;
-      const float* ri = rec + 2 + i;
-      for (int h0 = 0; h0 < hpg; h0 += 8) {
-        float acc[8];
+  float* at = tk + H * H;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = blockIdx.y * 32 + lane;
+  for (int g = warp; g < H; g += 8) {
+    const float* rg = a.ws + ((size_t)r * H + g) * n_splits * rs;
+    const float ms = lane < n_splits ? rg[lane * rs] : -INFINITY, ls = lane < n_splits ? rg[lane * rs + 1] : 0.f;
+    float x[32];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) acc[k] = 0.f;
-        for (int g0 = 0; g0 < H; g0 += 8) {  // eight heads' values in flight
-          float v[8];
+    for (int s = 0; s < 32; ++s) x[s] = s < n_splits && i < ncol ? rg[s * rs + 2 + i] : 0.f;
+    const float M = warp_max(ms), w0 = ms > -INFINITY ? expf(ms - M) : 0.f, w = w0 / warp_sum(w0 * ls);
+    float v = 0.f;
 #pragma unroll
-          for (int u = 0; u < 8; ++u) v[u] = g0 + u < H ? ri[(size_t)(g0 + u) * n_splits * rs] * wt[(g0 + u) * n_splits] : 0.f;
-          for (int s = 1; s < n_splits; ++s)
-#pragma unroll
-            for (int u = 0; u < 8; ++u)
-              if (g0 + u < H) v[u] = fmaf(ri[((size_t)(g0 + u) * n_splits + s) * rs], wt[(g0 + u) * n_splits + s], v[u]);
-#pragma unroll
-          for (int u = 0; u < 8; ++u) {
-            if (g0 + u >= H) break;
-            const float* t = tk + (g0 + u) * H + c * hpg + h0;
-#pragma unroll
-            for (int k = 0; k < 8; ++k)
-              if (h0 + k < hpg) acc[k] = fmaf(t[k], v[u], acc[k]);
-          }
-        }
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          if (h0 + k >= hpg) break;
-          const size_t o = (size_t)(c * hpg + h0 + k) * vd + col;
-          if (a.out_bf) a.out_bf[(size_t)r * a.ldo_bf + o] = f2bf(acc[k]);
-          else a.out[(size_t)r * a.ldo + o] = acc[k];
-        }
-      }
-    }
+    for (int s = 0; s < 32; ++s) v = fmaf(x[s], __shfl_sync(0xffffffffu, w, s), v);
+    at[g * 32 + lane] = v;
+  }
+  for (int j = threadIdx.x; j < H * H; j += blockDim.x) tk[j] = bf2f(a.talk[j]);
+  __syncthreads();
+  for (int j = threadIdx.x; j < hpg * 32; j += blockDim.x) {
+    const int k = j >> 5, x = j & 31, col = blockIdx.y * 32 + x;
+    if (col >= ncol) continue;
+    const int h = col / vd * hpg + k;
+    float v = 0.f;
+    for (int g = 0; g < H; ++g) v = fmaf(tk[h * H + g], at[g * 32 + x], v);
+    const size_t o = (size_t)h * vd + col % vd;
+    if (a.out_bf) a.out_bf[r * a.ldo_bf + o] = f2bf(v);
+    else a.out[r * a.ldo + o] = v;
   }
 }
 
@@ -1040,7 +1015,7 @@ cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* 
 
 // splits 0: the records are normalised, one per (row, head)
 static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStream_t st) {
-  const size_t smem = ((size_t)a.heads * splits + (size_t)a.heads * a.heads) * sizeof(float);
+  const size_t smem = ((size_t)a.heads * a.heads + (splits ? (size_t)a.heads * 32 : 0)) * sizeof(float);
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return cudaErrorInvalidValue;
     cudaError_t r = cudaFuncSetAttribute(splits ? (const void*)gqa_talk_finish_kernel : (const void*)gqa_talk_mix_kernel,
@@ -1048,7 +1023,7 @@ static cudaError_t launch_talk_finish(const GqaAttnArgs& a, int splits, cudaStre
     if (r != cudaSuccess) return r;
   }
   if (splits == 0) return launch_k(gqa_talk_mix_kernel, dim3(a.n), dim3(256), smem, st, a);
-  return launch_k(gqa_talk_finish_kernel, dim3(a.n), dim3(256), smem, st, a, splits);
+  return launch_k(gqa_talk_finish_kernel, dim3(a.n, (a.kv_heads * a.vdim + 31) / 32), dim3(256), smem, st, a, splits);
 }
 
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches) {
@@ -1092,6 +1067,10 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
   if (ctas < 2L * a.num_sms && a.max_keys > 2 * ATK) {
     splits = (int)std::min<long>((2L * a.num_sms + ctas - 1) / ctas, (a.max_keys + 2 * ATK - 1) / (2 * ATK));
     splits = std::max(1, std::min(splits, 16));
+  }
+  if (a.talk && splits > 1) {  // more value columns per key: one tile of keys per split, up to what a warp of the finishing kernel merges
+    const int keys = a.window > 0 ? std::min(a.max_keys, a.window + (a.c.block > 0 ? a.max_keys / a.c.block : 0)) : a.max_keys;
+    splits = (int)std::min<long>(std::max<long>(1, 4L * a.num_sms / ctas), std::min(32, (keys + ATK - 1) / ATK));
   }
   const size_t one = gqa_ws_floats(a.n, a.heads, a.maps, vcols);
   if (one > a.ws_floats) return cudaErrorInvalidValue;

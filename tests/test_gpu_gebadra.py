@@ -424,3 +424,37 @@ def test_bf16_linear_recurrence_in_chunks(tmp_path, dim, vdim):
         assert np.median(err) < 1e-2 and err.max() < 4e-2, (np.median(err), err.max())
     err = _row_err(steps, right[2])
     assert np.median(err) < 1e-2 and err.max() < 4e-2
+
+
+@pytest.mark.parametrize("kv_heads,dim,vdim,size,pool,page", [
+    (2, 64, 64, 100, 16, 64),    # a tile of keys is one page
+    (2, 16, 32, 90, 16, 128),    # a page is two tiles
+    (4, 40, 72, 70, 7, 16),      # 288 value columns: two chunks; blocks over page borders
+    (2, 128, 128, 130, 32, 16),  # two blocks of head columns, fewer stages
+    (1, 72, 24, 40, 16, 12),     # pages that do not divide a tile: every row by its own address
+    (2, 32, 16, 9, 1, 16),       # blocks of one token: more tiles of pooled rows than stages
+    (4, 8, 8, 500, 5, 32),       # a window longer than the prompt
+], ids=["page64", "page128", "two_value_chunks", "wide_heads", "odd_pages", "blocks_of_one", "no_block_seen"])
+def test_bf16_prompt_attention_tiles(tmp_path, kv_heads, dim, vdim, size, pool, page):
+    # the tensor-core prompt attention (portions of 128 rows and more) against the restatement, and against short portions of the
+    # same prompt through the other kernels; runs of equal tokens keep the pooled keys large, and the left half is loud
+    cfg = U.make_config([U.parallel(heads=8, kv_heads=kv_heads, dim=dim, vdim=vdim, size=size, pool=pool, scale=0.7 / np.sqrt(dim) * 2, rot_dims=dim // 4 * 2,
+                                    factor=2.0, rheads=2, rdim=8, rvdim=8)], width=64, vocab=29)
+    w = U.random_weights(cfg, seed=47, gain=1.3)
+    _sharp(cfg, w, factor=1.2, loud=3.0)
+    toks = _runs(cfg, 300, 3, 9)
+    right = _oracle_logits(cfg, w, toks)
+    other = _runs(cfg, 140, 3, 10)
+    right2 = _oracle_logits(cfg, w, other)
+    eng = _engine(tmp_path, cfg, w, dtype="bfloat16", page_size=page, max_pages=1600 // page, rows=512)
+    whole = _whole(eng, toks)
+    a, b = eng.new_sequence(), eng.new_sequence()
+    first = eng.forward_batch([(a, toks[:131])], range(131))
+    both = eng.forward_batch([(b, other), (a, toks[131:])], range(309))  # two sequences, one continues its cache
+    eng.free_sequence(a)
+    cut = _cuts(eng, toks, [60, 2, 63, 50, 1, 61, 63])
+    eng.close()
+    for got, want in ((whole, right), (np.concatenate([first, both[140:]]), right), (both[:140], right2), (cut, right)):
+        err = _row_err(got, want)
+        assert np.median(err) < 1e-2 and np.quantile(err, 0.95) < 3e-2 and err.max() < 8e-2, (np.median(err), err.max())
+    assert np.median(_row_err(_oracle_logits(cfg, w, toks[:150], fault_no_talk=True), right[:150])) > 0.1
