@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(LT) linear_chunk_state_kernel(const LinearAttn
     float acc[HB][4];
 #pragma unroll
     for (int i = 0; i < HB; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-#pragma unroll
+#pragma unroll 2
     for (int kb = 0; kb < LC / 16; ++kb) {
       // A = K'^T: element (state row m, token k) lies at [k][m]
       uint32_t ah[4], al[4];
@@ -285,7 +285,6 @@ __global__ void __launch_bounds__(LT) linear_chunk_out_kernel(const LinearAttnAr
   VT* Sh = Vs + LC;   // [DP] entry state, hi
   VT* Sl = Sh + DP;   // lo
   __shared__ float pw[LC + 1];
-  __shared__ float sq[2][LC];
   pdl_wait();
   pdl_trigger();
   int row0, L;
@@ -347,7 +346,7 @@ __global__ void __launch_bounds__(LT) linear_chunk_out_kernel(const LinearAttnAr
     float s[LC / 8][4];
 #pragma unroll
     for (int i = 0; i < LC / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-#pragma unroll
+#pragma unroll 2
     for (int kk = 0; kk < DP / 16; ++kk) {
       uint32_t qf[4];
       ldmatrix_x4(qf[0], qf[1], qf[2], qf[3], smem_u32(&Qs[w0 + (lane & 15)][kk * 16 + (lane >> 4) * 8]));
@@ -393,44 +392,56 @@ __global__ void __launch_bounds__(LT) linear_chunk_out_kernel(const LinearAttnAr
       }
     }
   }
-  const bool v0 = t0 < L, v1 = t1 < L;
-  float n0 = 1.f, n1 = 1.f;
-  if (a.norm_gate) {  // a row of a head lies in a quad of each of the two warps that share its rows
-    float q0 = 0.f, q1 = 0.f;
+  // the result goes through shared memory (everything else there has been read): four threads per row then write whole pieces
+  float (*os)[VP + 4] = reinterpret_cast<float (*)[VP + 4]>(lc_smem);
+  __syncthreads();
+  if (active) {
 #pragma unroll
-    for (int vb = 0; vb < HB; ++vb) q0 = fmaf(o[vb][0], o[vb][0], fmaf(o[vb][1], o[vb][1], q0)), q1 = fmaf(o[vb][2], o[vb][2], fmaf(o[vb][3], o[vb][3], q1));
-    q0 += __shfl_xor_sync(0xffffffffu, q0, 1), q1 += __shfl_xor_sync(0xffffffffu, q1, 1);
-    q0 += __shfl_xor_sync(0xffffffffu, q0, 2), q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
-    if ((lane & 3) == 0) sq[warp >> 2][t0] = q0, sq[warp >> 2][t1] = q1;
-    __syncthreads();
-    n0 = 1.0f / sqrtf((sq[0][t0] + sq[1][t0]) / (float)vdim + a.eps), n1 = 1.0f / sqrtf((sq[0][t1] + sq[1][t1]) / (float)vdim + a.eps);
-  }
-  const bool even = vdim % 2 == 0 && (a.norm_gate ? a.ldo_bf % 2 == 0 && a.ld_bf % 2 == 0 && ((reinterpret_cast<uintptr_t>(a.out_bf) | reinterpret_cast<uintptr_t>(a.g_bf)) & 3) == 0
-                                                  : a.ldo % 2 == 0);
-  auto put = [&](int t, int c, float x, float y, float n) {  // columns c and c + 1 of row t
-    const size_t r = (size_t)(row0 + t);
-    const int hc = h * vdim + c;
-    if (a.norm_gate) {
-      if (even) {
-        const uint32_t g = *reinterpret_cast<const uint32_t*>(a.g_bf + r * a.ld_bf + hc);
-        *reinterpret_cast<uint32_t*>(a.out_bf + r * a.ldo_bf + hc) = pack2f(x * n * silu_f(lo2f(g)), y * n * silu_f(hi2f(g)));
-      } else {
-        a.out_bf[r * a.ldo_bf + hc] = f2bf(x * n * silu_f(bf2f(a.g_bf[r * a.ld_bf + hc])));
-        if (c + 1 < vdim) a.out_bf[r * a.ldo_bf + hc + 1] = f2bf(y * n * silu_f(bf2f(a.g_bf[r * a.ld_bf + hc + 1])));
-      }
-    } else if (even) {
-      *reinterpret_cast<float2*>(a.out + r * a.ldo + hc) = make_float2(x, y);
-    } else {
-      a.out[r * a.ldo + hc] = x;
-      if (c + 1 < vdim) a.out[r * a.ldo + hc + 1] = y;
+    for (int vb = 0; vb < HB; ++vb) {
+      const int c = (vb0 + vb) * 8 + qc;
+      *reinterpret_cast<float2*>(&os[t0][c]) = make_float2(o[vb][0], o[vb][1]);
+      *reinterpret_cast<float2*>(&os[t1][c]) = make_float2(o[vb][2], o[vb][3]);
     }
-  };
+  }
+  __syncthreads();
+  const int t = tid >> 2, c0 = (tid & 3) * 4;
+  const size_t r = (size_t)(row0 + t);
+  float n = 1.f;
+  if (a.norm_gate) {
+    float q = 0.f;
+    for (int c = c0; c < vdim; c += 16)
 #pragma unroll
-  for (int vb = 0; vb < HB; ++vb) {
-    const int c = (vb0 + vb) * 8 + qc;
-    if (c >= vdim) continue;
-    if (v0) put(t0, c, o[vb][0], o[vb][1], n0);
-    if (v1) put(t1, c, o[vb][2], o[vb][3], n1);
+      for (int e = 0; e < 4; ++e)
+        if (c + e < vdim) q = fmaf(os[t][c + e], os[t][c + e], q);
+    q += __shfl_xor_sync(0xffffffffu, q, 1);
+    q += __shfl_xor_sync(0xffffffffu, q, 2);
+    n = 1.0f / sqrtf(q / (float)vdim + a.eps);
+  }
+  if (t >= L) return;
+  if (a.norm_gate) {
+    const bf16* g = a.g_bf + r * a.ld_bf + h * vdim;
+    bf16* out = a.out_bf + r * a.ldo_bf + h * vdim;
+    const bool vec = vdim % 4 == 0 && a.ld_bf % 4 == 0 && a.ldo_bf % 4 == 0 && ((reinterpret_cast<uintptr_t>(a.g_bf) | reinterpret_cast<uintptr_t>(a.out_bf)) & 7) == 0;
+#pragma unroll 2
+    for (int c = c0; c < vdim; c += 16) {
+      if (vec) {
+        const uint2 gv = *reinterpret_cast<const uint2*>(g + c);
+        const float4 x = *reinterpret_cast<const float4*>(&os[t][c]);
+        *reinterpret_cast<uint2*>(out + c) = make_uint2(pack2f(x.x * n * silu_f(lo2f(gv.x)), x.y * n * silu_f(hi2f(gv.x))),
+                                                        pack2f(x.z * n * silu_f(lo2f(gv.y)), x.w * n * silu_f(hi2f(gv.y))));
+      } else {
+        for (int e = c; e < min(c + 4, vdim); ++e) out[e] = f2bf(os[t][e] * n * silu_f(bf2f(g[e])));
+      }
+    }
+  } else {
+    float* out = a.out + r * a.ldo + h * vdim;
+    const bool vec = vdim % 4 == 0 && a.ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0;
+#pragma unroll 2
+    for (int c = c0; c < vdim; c += 16) {
+      if (vec) *reinterpret_cast<float4*>(out + c) = *reinterpret_cast<const float4*>(&os[t][c]);
+      else
+        for (int e = c; e < min(c + 4, vdim); ++e) out[e] = os[t][e];
+    }
   }
 }
 
