@@ -283,23 +283,42 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const NormGate a) {
   const size_t r = blockIdx.x;
   const int W = a.width, gs = W / a.groups, t0 = threadIdx.x * V, step = blockDim.x * V;
   float* scale = row + W;
-  for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_f32<V>(a.v + r * a.ldv + i));
-  __syncthreads();
-  group_rstd(row, W, a.groups, a.eps, red, scale);
-  for (int i = t0; i < W; i += step) {
-    Pack<V> x = ld_f32<V>(row + i), w;
-    const Pack<V> g = a.g_bf ? ld_bf16<V>(a.g_bf + r * a.ldg_bf + i) : ld_f32<V>(a.g + r * a.ldg + i);
+  auto gate_of = [&](int i) { return a.g_bf ? ld_bf16<V>(a.g_bf + r * a.ldg_bf + i) : ld_f32<V>(a.g + r * a.ldg + i); };
+  auto finish = [&](int i, Pack<V> x, const Pack<V>& g, float s0) {
+    Pack<V> w;
     if (a.w) w = ld_bf16<V>(a.w + i);
 #pragma unroll
     for (int u = 0; u < V; ++u) {
       const float sg = 1.0f / (1.0f + expf(-g.v[u]));
-      float y = x.v[u] * scale[(i + u) / gs];
+      float y = x.v[u] * (a.groups == 1 ? s0 : scale[(i + u) / gs]);
       if (a.w) y *= w.v[u];
       x.v[u] = y * (a.act == 1 ? sg : g.v[u] * sg);
     }
     if (a.out) st_f32<V>(a.out + r * a.ldo + i, x);
     if (a.out_bf) st_bf16<V>(a.out_bf + r * a.ldo_bf + i, x);
+  };
+  constexpr int NR = 2;
+  if (a.groups == 1 && W <= NR * step) {  // the row and its gate stay in registers, every load in flight at once
+    Pack<V> x[NR], g[NR];
+    float sq = 0.f;
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W) x[k] = ld_f32<V>(a.v + r * a.ldv + t0 + k * step), g[k] = gate_of(t0 + k * step);
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W)
+#pragma unroll
+        for (int u = 0; u < V; ++u) sq = fmaf(x[k].v[u], x[k].v[u], sq);
+    const float s0 = 1.0f / sqrtf(block_sum_r(sq, red) / (float)W + a.eps);
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W) finish(t0 + k * step, x[k], g[k], s0);
+    return;
   }
+  for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_f32<V>(a.v + r * a.ldv + i));
+  __syncthreads();
+  group_rstd(row, W, a.groups, a.eps, red, scale);
+  for (int i = t0; i < W; i += step) finish(i, ld_f32<V>(row + i), gate_of(i), scale[0]);
 }
 
 }  // namespace

@@ -79,6 +79,7 @@ SINGLE = {
     "lightning_one_head": ([U.lightning(heads=1, dim=7, vdim=3, decay=[1.0])], 1),
     "lightning_wide_values": ([U.lightning(heads=2, dim=3, vdim=70, decay=[0.0, 0.9], mlp=U.dense(ff=3))], 3),
     "lightning_wide_keys": ([U.lightning(heads=2, dim=130, vdim=2)], 2),
+    "lightning_long_row": ([U.lightning(heads=5, dim=4, vdim=103)], 2),
     "parallel": ([U.parallel()], 2),
     "parallel_plain": ([U.parallel(heads=3, kv_heads=3, dim=5, vdim=3, rot_dims=0, rheads=1)], 1),
     "parallel_one_kv_head": ([U.parallel(heads=8, kv_heads=1, dim=4, vdim=40, size=1, pool=1, rot_dims=4, factor=None)], 4),
