@@ -146,8 +146,8 @@ cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* 
 // shared_keys: every head scores against the WHOLE key part of the cached row (dim = kw / maps elements: the keys of all
 // kv heads side by side) while its values stay those of kv head h / (heads / kv_heads); the queries are then
 // [h][map][kw / maps] (TalkQueries builds them).
-// c.block > 0 (with a window): beside the tokens of the window a row sees the pooled rows of the blocks that lie wholly before
-// it, block b when (b + 1) * block - 1 <= pos - window, in the same softmax.
+// c.block > 0 (with a window): beside the tokens of the window a row sees the pooled rows of the blocks that end before
+// it begins, block b when (b + 1) * block - 1 <= pos - window, in the same softmax.
 // talk (optional, [heads, heads]): the heads' softmax weights are mixed, weight_h <- sum_g talk[h, g] weight_g, before they meet
 // the values of head h's own kv head.  Computed as out_h = sum_g talk[h, g] (softmax_g . values of h's kv head): every
 // head attends to the values of all kv heads, and the heads are mixed when its result is complete.

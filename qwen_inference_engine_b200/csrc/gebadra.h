@@ -37,7 +37,7 @@ namespace qie {
 //   S = decay_h S + (k_scale k_t) v_t^T,   o_t = S^T q_t          with act 1: q, k, v = silu of the rows read
 // q [n, heads * dim], k alike, v [n, heads * vdim] are columns of fp32 rows (row stride ld) or of bf16 rows (*_bf, ld_bf).
 // decay_pow: [heads][LINEAR_CHUNK + 1] the powers decay_h^0 .. decay_h^LINEAR_CHUNK on the device.
-// The result goes to fp32 rows.  With norm_gate (only where launch_linear_attention_fuses says so) each head's o is divided by
+// The result goes to fp32 rows.  With norm_gate (only where linear_attention_chunked says so) each head's o is divided by
 // sqrt(mean(o^2) + eps), multiplied by silu(g_bf[t, h * vdim + c]) and written as bf16 rows instead.
 // bf16 sources, LINEAR_CHUNK rows and more and a workspace: portions run in chunks of LINEAR_CHUNK rows on tensor cores (each chunk's own
 // contribution to the state, a carry pass over the chunks, then the outputs of all chunks side by side); else token by token.

@@ -17,7 +17,7 @@ __device__ __forceinline__ const char* kv_pool_ptr(const KvRowCache& c, const in
   const size_t off = (size_t)page * c.page_elems + c.pool_off + (size_t)(b - pi * c.page_size / c.block) * (c.kw + c.vw);
   return static_cast<const char*>(c.pool) + off * c.elt_bytes;
 }
-// blocks that lie wholly before the window of position pos: (b + 1) * block - 1 <= pos - window
+// blocks that end before the window of position pos begins: (b + 1) * block - 1 <= pos - window
 __host__ __device__ __forceinline__ int pooled_seen(int pos, int window, int block) { return block > 0 && pos >= window ? (pos - window + 1) / block : 0; }
 
 }  // namespace qie
