@@ -21,14 +21,15 @@ __global__ void xielu_kernel(float* __restrict__ z, int ld, int cols, const bf16
   }
 }
 
-__global__ void silu_glu_kernel(const float* gu, int ld, float* out, int ldo, int ff) {  // out may be gu (a thread reads its elements first)
+__global__ void silu_glu_kernel(const float* gu, int ld, float* out, int ldo, int ff, const float* __restrict__ row_w) {  // out may be gu (a thread reads its elements first)
   pdl_wait();
   pdl_trigger();
   const float* row = gu + (size_t)blockIdx.x * ld;
   float* o = out + (size_t)blockIdx.x * ldo;
+  const float rw = row_w ? row_w[blockIdx.x] : 1.0f;
   for (int i = threadIdx.x; i < ff; i += blockDim.x) {
-    const float g = row[i];
-    o[i] = g / (1.0f + expf(-g)) * row[ff + i];
+    const float g = row[i] * rw;
+    o[i] = g / (1.0f + expf(-g)) * (row[ff + i] * rw);
   }
 }
 
@@ -137,9 +138,9 @@ cudaError_t launch_xielu(float* z, int ld, int cols, const bf16* pq, int n, cuda
   return launch_k(xielu_kernel, dim3(n), dim3(256), 0, st, z, ld, cols, pq);
 }
 
-cudaError_t launch_silu_glu(const float* gu, int ld, float* out, int ldo, int ff, int n, cudaStream_t st) {
+cudaError_t launch_silu_glu(const float* gu, int ld, float* out, int ldo, int ff, int n, cudaStream_t st, const float* row_w) {
   if (n <= 0 || ff <= 0) return cudaSuccess;
-  return launch_k(silu_glu_kernel, dim3(n), dim3(256), 0, st, gu, ld, out, ldo, ff);
+  return launch_k(silu_glu_kernel, dim3(n), dim3(256), 0, st, gu, ld, out, ldo, ff, row_w);
 }
 
 }  // namespace qie

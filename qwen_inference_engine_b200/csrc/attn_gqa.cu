@@ -1,7 +1,7 @@
 // attn_gqa.cu -- grouped-query attention over paged key/value rows for the fp32-stream families (fosavik.h): the
 // store of new rows (optional unit norm of queries and keys, per head or over the whole projection; mean rows of whole
 // blocks of tokens), and an attention whose mask, sink, number of score maps and finishing step are arguments: causal or
-// sliding window with kept first tokens or with the mean rows of the blocks before it, a unit sink in the denominator, one
+// sliding window with kept first tokens or with the mean rows of the blocks before it, or the row's own chunk of positions, a unit sink in the denominator, one
 // or two softmax maps over shared values, and as the last step nothing, a sigmoid gate per head, the differential
 // combination with a unit norm per head, or a mix of the heads' softmax weights.  Softmax and accumulation are fp32; the cache rows are fp32
 // or bf16.  Keys are ALWAYS read from the cache (a row's own position is stored first), so a result does not depend
@@ -49,12 +49,12 @@ __device__ __forceinline__ void talk_queries_row(const TalkQueries& t, int r, fl
 template <typename Get, typename Put>
 __device__ __forceinline__ void norm_rope_group(const KvStoreArgs& a, int p, int lane, int d, Get get, const bf16* w, Put put) {
   float rstd = 1.f;
-  if (w) {
+  if (w || a.unit_norm) {
     float s = 0.f;
     for (int i = lane; i < d; i += 32) s = fmaf(get(i), get(i), s);
     rstd = 1.0f / sqrtf(warp_sum(s) / (float)d + a.eps);
   }
-  auto val = [&](int i) { return w ? get(i) * rstd * bf2f(w[i]) : get(i); };
+  auto val = [&](int i) { return w ? get(i) * rstd * bf2f(w[i]) : a.unit_norm ? get(i) * rstd : get(i); };
   const int dims = a.rope.dims, half = dims / 2;
   const int st1 = a.rope.half_layout ? 1 : 2, off2 = a.rope.half_layout ? half : 1;
   for (int i = lane; i < half; i += 32) {
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(128) kv_store_rows_kernel(const KvStoreArgs a)
     char* row = const_cast<char*>(kv_row_ptr(a.c, a.block_table, a.max_pages, a.slot[r], a.pos[r]));
     const float* k = a.k + (size_t)r * a.ldk;
     auto key = [&](int i) { return a.k_bias ? k[i] + bf2f(a.k_bias[i]) : k[i]; };
-    if (a.k_norm || a.rope.dims > 0) {
+    if (a.k_norm || a.unit_norm || a.rope.dims > 0) {
       const int d = a.norm_dim;
       for (int g = warp; g < a.c.kw / d; g += nw) norm_rope_group(a, a.pos[r], lane, d, [&](int i) { return key(g * d + i); }, a.k_norm,
                                                                   [&](int i, float x) { store_elt(a.c, row, g * d + i, x); });
@@ -95,7 +95,7 @@ __global__ void __launch_bounds__(128) kv_store_rows_kernel(const KvStoreArgs a)
       store_elt(a.c, row, a.c.kw + i, x);
     }
   }
-  if (a.q && (a.q_norm || a.rope.dims > 0 || a.q_bias)) {
+  if (a.q && (a.q_norm || a.unit_norm || a.rope.dims > 0 || a.q_bias)) {
     float* q = a.q + (size_t)r * a.ldq;
     const int d = a.norm_dim;
     for (int h = warp; h < a.q_heads; h += nw)
@@ -305,6 +305,90 @@ __global__ void __launch_bounds__(256) kv_store_whole_warp_kernel(const KvStoreA
   }
 }
 
+// bf16 sources, a unit norm per head (weights optional), rotary pairs (i, i + dims/2): a warp per row, lane = 16-byte pieces lane,
+// lane + 32, ... of the row's [queries | keys]; the d / 8 lanes of a head (a power of two) add up its squares, and a piece meets the piece
+// that it is rotated with through a shuffle.  NQ, NK: pieces per lane.
+template <int NQ, int NK>
+__global__ void __launch_bounds__(256) kv_store_heads_warp_kernel(const KvStoreArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= a.n) return;
+  const int p = a.pos[r], d = a.norm_dim, hp = a.rope.dims / 16, pph = d / 8;  // pieces per half of the rotated part, per head
+  const int q8 = a.q_heads * pph, k8 = a.c.kw / 8, v8 = a.c.vw / 8;
+  const uint4* qb = reinterpret_cast<const uint4*>(a.q_bf + (size_t)r * a.ld_bf);
+  const uint4* kb = reinterpret_cast<const uint4*>(a.k_bf + (size_t)r * a.ld_bf);
+  const uint4* vb = reinterpret_cast<const uint4*>(a.v_bf + (size_t)r * a.ld_bf);
+  bf16* row = reinterpret_cast<bf16*>(const_cast<char*>(kv_row_ptr(a.c, a.block_table, a.max_pages, a.slot[r], p)));
+  uint4 q[NQ], k[NK];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) q[i] = lane + 32 * i < q8 ? qb[lane + 32 * i] : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+  for (int i = 0; i < NK; ++i) k[i] = lane + 32 * i < k8 ? kb[lane + 32 * i] : make_uint4(0u, 0u, 0u, 0u);
+  for (int i = lane; i < v8; i += 32) reinterpret_cast<uint4*>(row + a.c.kw)[i] = vb[i];
+  const int pi = lane % pph;  // the lane's piece of its head, the same in every round (pph divides 32)
+  const bool first = pi < hp, turned = pi < 2 * hp;
+  const int mate = first ? lane + hp : turned ? lane - hp : lane;
+  float cs[8], sn[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) cs[j] = 1.f, sn[j] = 0.f;
+  if (turned) {
+    const size_t o = (size_t)p * (a.rope.dims / 2) + (size_t)(first ? pi : pi - hp) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; j += 4) {
+      const float4 c4 = *reinterpret_cast<const float4*>(a.rope.cos_t + o + j), s4 = *reinterpret_cast<const float4*>(a.rope.sin_t + o + j);
+      const float sg = first ? -1.f : 1.f;  // u cos - v sin for the first half, v cos + u sin for the second
+      cs[j] = c4.x, cs[j + 1] = c4.y, cs[j + 2] = c4.z, cs[j + 3] = c4.w;
+      sn[j] = sg * s4.x, sn[j + 1] = sg * s4.y, sn[j + 2] = sg * s4.z, sn[j + 3] = sg * s4.w;
+    }
+  }
+  auto weights = [&](const bf16* w, float (&f)[8]) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] = w ? bf2f(w[pi * 8 + j]) : 1.f;
+  };
+  float qw[8], kw_[8];
+  weights(a.q_norm, qw);
+  weights(a.k_norm, kw_);
+  // every lane of the warp takes part (the shuffles); y: the piece normed and rotated
+  auto turn = [&](const uint4& x, const float (&w)[8], bool norm, float (&y)[8]) {
+    const uint32_t u[4] = {x.x, x.y, x.z, x.w};
+    float f[8], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      f[2 * j] = lo2f(u[j]), f[2 * j + 1] = hi2f(u[j]);
+      s = fmaf(f[2 * j], f[2 * j], fmaf(f[2 * j + 1], f[2 * j + 1], s));
+    }
+    float rstd = 1.f;
+    if (norm) {
+      for (int o = pph >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      rstd = 1.0f / sqrtf(s / (float)d + a.eps);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float v = f[j] * rstd * w[j];
+      const float m = __shfl_sync(0xffffffffu, v, mate);
+      y[j] = fmaf(v, cs[j], m * sn[j]);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < NK; ++i) {
+    if (32 * i >= k8) break;
+    float y[8];
+    turn(k[i], kw_, a.unit_norm || a.k_norm, y);
+    if (lane + 32 * i < k8) reinterpret_cast<uint4*>(row)[lane + 32 * i] = make_uint4(pack2f(y[0], y[1]), pack2f(y[2], y[3]), pack2f(y[4], y[5]), pack2f(y[6], y[7]));
+  }
+  float* qf = a.q + (size_t)r * a.ldq;
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    if (32 * i >= q8) break;
+    float y[8];
+    turn(q[i], qw, a.unit_norm || a.q_norm, y);
+    if (lane + 32 * i >= q8) continue;
+    *reinterpret_cast<float4*>(qf + 8 * (lane + 32 * i)) = make_float4(y[0], y[1], y[2], y[3]);
+    *reinterpret_cast<float4*>(qf + 8 * (lane + 32 * i) + 4) = make_float4(y[4], y[5], y[6], y[7]);
+  }
+}
+
 // CTA (row, kv head x head chunk x value chunk, key split).  Shared memory: q [QV][dim] (scaled) | K tile [ATK][kd + 1] | V tile
 // [ATK][nv] | scores [QV][ATK] | corr [QV] | m [QV] | l [QV], QV = hpc * maps query vectors, kd = maps * dim, nv <= vc the
 // value columns of this CTA: a head's own vdim, or (talk) a chunk of the values of all kv heads.
@@ -332,9 +416,9 @@ __global__ void __launch_bounds__(ATHREADS) gqa_attention_kernel(const GqaAttnAr
   float* lrun = mrun + hpc * maps;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pos = a.pos[r], slot = a.slot[r];
-  // visible keys as one virtual range: the pooled blocks before the window, the kept first tokens below it, then the window
+  // visible keys as one virtual range: the pooled blocks before the window, the kept first tokens below it, then the window (or the chunk)
   const int npool = a.c.block > 0 ? pooled_seen(pos, a.window, a.c.block) : 0;
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = first_seen(pos, a.window, a.chunk);
   const int nfirst = a.window > 0 ? min(a.keep_first, lo) : 0;
   const int nkeys = npool + nfirst + (pos - lo + 1);
   int per = (nkeys + n_splits - 1) / n_splits;
@@ -492,8 +576,8 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   if (tid == 0) {
     // a CTA takes tile p and tile nt-1-p of a segment: under a causal mask the late tiles see many key blocks and the early
     // ones few, so every CTA gets about the same number
-    // (under a sliding window every tile sees about the same number: one tile per CTA, twice the CTAs)
-    const bool pair = a.window <= 0;
+    // (under a sliding window or in chunks every tile sees about the same number: one tile per CTA, twice the CTAs)
+    const bool pair = a.window <= 0 && a.chunk <= 0;
     int left = blockIdx.x, found = 0;
     for (int s = 0; s < n_seg && !found; ++s) {
       const int r0 = seg_start[s], len = seg_start[s + 1] - r0, nt = (len + PT_ROWS - 1) / PT_ROWS, np = pair ? (nt + 1) / 2 : nt;
@@ -519,7 +603,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   const int row0 = tile_info[0] + tile * PT_ROWS, nrows = min(PT_ROWS, tile_info[1] - tile * PT_ROWS);
   const int pos0 = a.pos[row0];                       // rows of a segment are consecutive positions
   const int pmax = pos0 + nrows - 1;
-  const int lo_min = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int lo_min = first_seen(pos0, a.window, a.chunk);
   const int nbmax = a.c.block > 0 ? pooled_seen(pmax, a.window, a.c.block) : 0, npb = (nbmax + PT_KEYS - 1) / PT_KEYS;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
   // soft cap of a scaled score: cap * tanh(s / cap) as cap * (1 - 2 / (exp(2 s / cap) + 1)); the weights become bf16 operands
@@ -530,6 +614,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
   const int wrow = warp * 16;
   const bool rv0 = wrow + qr < nrows, rv1 = wrow + qr + 8 < nrows;
   const int i0 = pos0 + wrow + qr, i1 = i0 + 8;       // positions of the thread's two rows
+  const int cl0 = a.chunk > 0 ? i0 / a.chunk * a.chunk : 0, cl1 = a.chunk > 0 ? i1 / a.chunk * a.chunk : 0;  // and where their chunks start
   // 16-byte staging when every cache row piece starts on a 16-byte boundary
   const bool vec = (a.c.page_elems % 8 == 0) && (a.c.layer_off % 8 == 0) && ((a.c.kw + a.c.vw) % 8 == 0) && (dim % 8 == 0) && (vd % 8 == 0) &&
                    (a.c.kw % 8 == 0) && (!a.c.block || a.c.pool_off % 8 == 0);
@@ -559,7 +644,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
     for (int i = 0; i < VP / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     // key blocks that some row of the tile sees: the blocks of the kept first tokens, then from the window's lower edge on
-    auto skipped = [&](int j) { return a.window > 0 && j + PT_KEYS - 1 < lo_min && j >= a.keep_first; };
+    auto skipped = [&](int j) { return (a.window > 0 || a.chunk > 0) && j + PT_KEYS - 1 < lo_min && j >= a.keep_first; };
     // a block's number j is its first position, or for the npb blocks of pooled rows -PT_KEYS * npb, ..., -PT_KEYS
     auto next_block = [&](int j) {
       j += PT_KEYS;
@@ -633,7 +718,8 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
       // mask, running maximum
       float mx0 = -INFINITY, mx1 = -INFINITY;
       // a block that every row of the warp sees whole (below the diagonal, inside the window) needs no mask
-      const bool whole = j0 >= 0 && j0 + PT_KEYS - 1 <= pos0 + wrow && (a.window <= 0 || pos0 + wrow + 15 - j0 < a.window);
+      const bool whole = j0 >= 0 && j0 + PT_KEYS - 1 <= pos0 + wrow && (a.window <= 0 || pos0 + wrow + 15 - j0 < a.window) &&
+                         (a.chunk <= 0 || j0 >= (pos0 + wrow + 15) / a.chunk * a.chunk);
       if (j0 < 0) {  // pooled rows: a prefix of the blocks, longer for later rows
         const int b0 = j0 + npb * PT_KEYS + qc, n0 = pooled_seen(i0, a.window, a.c.block), n1 = pooled_seen(i1, a.window, a.c.block);
 #pragma unroll
@@ -661,7 +747,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
           for (int e = 0; e < 4; ++e) {
             const int j = j0 + nb * 8 + qc + (e & 1);
             const int i = (e >> 1) ? i1 : i0;
-            const bool ok = j <= i && (a.window <= 0 || i - j < a.window || j < a.keep_first);
+            const bool ok = j <= i && j >= ((e >> 1) ? cl1 : cl0) && (a.window <= 0 || i - j < a.window || j < a.keep_first);
             s[nb][e] = ok ? capped(s[nb][e] * a.scale) - slope * (float)(i - j) : -INFINITY;  // the scale meets the fp32 score, not the bf16 operand
             if (e >> 1) mx1 = fmaxf(mx1, s[nb][e]);
             else mx0 = fmaxf(mx0, s[nb][e]);
@@ -805,7 +891,7 @@ __global__ void __launch_bounds__(128) gqa_prefill_mma_kernel(const GqaAttnArgs 
 
 template <int DP, int VP>
 cudaError_t launch_prefill_mma_dv(const GqaAttnArgs& a, const int* seg_start, const int* seg_slot, int n_seg, cudaStream_t st) {
-  const int per_cta = a.window <= 0 ? 2 * PT_ROWS : PT_ROWS;
+  const int per_cta = a.window <= 0 && a.chunk <= 0 ? 2 * PT_ROWS : PT_ROWS;
   // talk: the values of all kv heads in equal chunks of at most VP columns, each a multiple of 8
   const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim, nvc = (vcols + VP - 1) / VP, vc = ((vcols + nvc - 1) / nvc + 7) / 8 * 8;
   const dim3 grid((a.n + per_cta - 1) / per_cta + n_seg, a.heads, nvc), block(128);  // upper bound of the tiles / tile pairs
@@ -974,9 +1060,26 @@ __global__ void __launch_bounds__(256) gqa_talk_mix_kernel(const GqaAttnArgs a) 
 
 static size_t talk_smem(const TalkQueries& t) { return ((size_t)t.heads * t.dim + (size_t)t.heads * t.heads) * sizeof(float); }
 
+bool kv_store_heads_fits(const KvStoreArgs& a) {
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const int d = a.norm_dim;
+  return a.q_bf && a.k_bf && a.v_bf && a.q && !a.whole_norm && a.c.elt_bytes == 2 && a.c.block == 0 && d >= 8 && d <= 256 && (d & (d - 1)) == 0 && a.c.kw % d == 0 &&
+         a.rope.dims % 16 == 0 && a.rope.dims <= d && (a.rope.dims == 0 || a.rope.half_layout) && a.c.vw % 8 == 0 && a.ld_bf % 8 == 0 && a.ldq % 4 == 0 &&
+         a.c.layer_off % 8 == 0 && a.c.page_elems % 8 == 0 && a.q_heads * d <= 4096 && a.c.kw <= 2048 && !a.q_bias && !a.k_bias && !a.v_bias && !a.tq.talk &&
+         !a.v_lam && !a.v_keep && al(a.q_bf) && al(a.k_bf) && al(a.v_bf) && al(a.q) && al(a.c.pool) && al(a.rope.cos_t) && al(a.rope.sin_t);
+}
+
 cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st) {
   if (a.n <= 0) return cudaSuccess;
-  if ((a.k_norm || a.rope.dims > 0) && (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2)) return cudaErrorInvalidValue;
+  if (a.k_bf && !a.whole_norm) {
+    if (!kv_store_heads_fits(a)) return cudaErrorInvalidValue;
+    const int nq = a.q_heads * a.norm_dim;
+    const dim3 grid((a.n + 7) / 8);
+    if (nq <= 1024 && a.c.kw <= 512) return launch_k(kv_store_heads_warp_kernel<4, 2>, grid, dim3(256), 0, st, a);
+    if (nq <= 2048 && a.c.kw <= 1024) return launch_k(kv_store_heads_warp_kernel<8, 4>, grid, dim3(256), 0, st, a);
+    return launch_k(kv_store_heads_warp_kernel<16, 8>, grid, dim3(256), 0, st, a);
+  }
+  if ((a.k_norm || a.unit_norm || a.rope.dims > 0) && (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2)) return cudaErrorInvalidValue;
   if (a.c.block > 0 && !a.whole_norm) return cudaErrorInvalidValue;  // pooled rows are written by the whole-projection form
   if (a.whole_norm) {
     if (a.norm_dim <= 0 || a.c.kw % a.norm_dim || a.rope.dims > a.norm_dim || a.rope.dims % 2 || !a.c.pool || a.tq.talk || a.v_lam || a.v_keep ||
@@ -1034,14 +1137,15 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
   if (a.out_bf && a.maps != 1 && !a.out) return cudaErrorInvalidValue;  // two maps: the first one's result waits in the fp32 rows
   if (a.talk && (a.maps != 1 || a.finish || a.unit_sink || a.shared_keys)) return cudaErrorInvalidValue;
   if (a.c.block > 0 && (a.window <= 0 || a.slopes || a.shared_keys || a.maps != 1)) return cudaErrorInvalidValue;
+  if (a.chunk > 0 && (a.window > 0 || a.keep_first > 0)) return cudaErrorInvalidValue;
   const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim;
   if (a.talk && gqa_ws_floats(a.n, a.heads, 1, vcols) > a.ws_floats) return cudaErrorInvalidValue;
-  // mixed heads over a bf16 cache: the tcgen05 kernel for prompt portions (QIE_ATTN_TC=0: the kernels below)
+  // plain or mixed heads over a bf16 cache: the tcgen05 kernel for prompt portions (QIE_ATTN_TC=0: the kernels below)
   static const bool tc_on = [] { const char* v = getenv("QIE_ATTN_TC"); return !(v && v[0] == '0'); }();
-  if (tc_on && gqa_talk_tc_fits(a)) {
-    if (n_launches) *n_launches = 2;
-    cudaError_t r = launch_gqa_talk_tc(a, st);
-    return r != cudaSuccess ? r : launch_talk_finish(a, 0, st);
+  if (tc_on && gqa_tc_fits(a)) {
+    if (n_launches) *n_launches = a.talk ? 2 : 1;
+    cudaError_t r = launch_gqa_tc(a, st);
+    return r != cudaSuccess || !a.talk ? r : launch_talk_finish(a, 0, st);
   }
   // prompt portions over a bf16 cache: the tensor-core kernel (one launch, no workspace); QIE_ATTN_MMA=0 keeps the per-row kernel (A/B)
   static const bool mma_on = [] { const char* v = getenv("QIE_ATTN_MMA"); return !(v && v[0] == '0'); }();
@@ -1064,8 +1168,9 @@ cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_l
   // key splits: fill the machine when there are few rows, within the workspace
   int splits = 1;
   const long ctas = (long)a.n * a.kv_heads * chunks * nvc;
-  if (ctas < 2L * a.num_sms && a.max_keys > 2 * ATK) {
-    splits = (int)std::min<long>((2L * a.num_sms + ctas - 1) / ctas, (a.max_keys + 2 * ATK - 1) / (2 * ATK));
+  const int most = a.chunk > 0 ? std::min(a.max_keys, a.chunk) : a.max_keys;  // keys of a row
+  if (ctas < 2L * a.num_sms && most > 2 * ATK) {
+    splits = (int)std::min<long>((2L * a.num_sms + ctas - 1) / ctas, (most + 2 * ATK - 1) / (2 * ATK));
     splits = std::max(1, std::min(splits, 16));
   }
   if (a.talk && splits > 1) {  // more value columns per key: one tile of keys per split, up to what a warp of the finishing kernel merges

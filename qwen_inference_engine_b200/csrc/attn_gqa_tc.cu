@@ -1,6 +1,6 @@
 // attn_gqa_tc.cu -- prompt attention over paged bf16 key/value rows on the 5th-gen tensor cores (tcgen05 + TMEM), for grouped
-// queries whose softmax weights are mixed over the heads (GqaAttnArgs::talk), a sliding window or a causal mask, and pooled
-// rows.  Mixing after the softmax is linear, so every head attends to the values of ALL kv heads -- one product with up to
+// queries under a sliding window, a causal mask or chunks of positions, and pooled rows.  A plain head attends to the values of its kv
+// head and writes its output rows.  The softmax weights may be mixed over the heads (GqaAttnArgs::talk).  Mixing after the softmax is linear, so every head attends to the values of ALL kv heads -- one product with up to
 // 256 value columns, which is what the tensor cores are good at -- and gqa_talk_mix_kernel mixes the results.
 //
 // A CTA owns 128 consecutive rows of one segment, one query head and one chunk of value columns, and walks tiles of 64 keys: first
@@ -137,7 +137,7 @@ __device__ __forceinline__ void copy_row(const bf16* row, size_t koff, size_t vo
   }
 }
 
-__global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc,
+__global__ void __launch_bounds__(NTHR, 1) gqa_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc,
                                                                const __grid_constant__ CUtensorMap rows_map, int use_tma) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   __shared__ int info[4];  // first row, rows, slot
@@ -166,9 +166,10 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   const uint32_t bar_full = b0, bar_empty = b0 + 8 * MAX_ST, bar_s = b0 + 16 * MAX_ST, bar_p = bar_s + 16, bar_o = bar_s + 32, tslot = bar_s + 48;
   float* xmax = reinterpret_cast<float*>(sg + L.bar + 256);  // [tile parity][quarter][row]; the sums use the parity that the last tile did not
   const int h = blockIdx.x, g = h / (a.heads / a.kv_heads), dim = a.dim;
-  const int vcols = a.kv_heads * a.vdim, col0 = blockIdx.z * vc, nv = min(vc, vcols - col0);
+  // value columns: chunk blockIdx.z of those of all kv heads, or (plain heads) the columns of head h's kv head
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim, zc = blockIdx.z * vc, nv = min(vc, vcols - zc), col0 = a.talk ? zc : g * a.vdim + zc;
   const int pos0 = a.pos[row0], pmax = pos0 + nrows - 1;
-  const int lo_min = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int lo_min = first_seen(pos0, a.window, a.chunk);
   const int nbmax = a.c.block > 0 ? pooled_seen(pmax, a.window, a.c.block) : 0, npt = (nbmax + TK - 1) / TK;
   const int tt0 = lo_min / TK, nt = npt + pmax / TK - tt0 + 1;  // tiles: npt of pooled rows, then tokens from tile tt0 on
   if (tid == 0) {
@@ -316,7 +317,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
   } else {
     // ---- softmax: row (TMEM lane), quarter of the tile's keys and of O's columns
     const int row = (warp & 3) * 32 + lane, qt = warp >> 2;
-    const int my_pos = pos0 + row, my_lo = a.window > 0 ? my_pos - a.window + 1 : 0, my_seen = a.c.block > 0 ? pooled_seen(my_pos, a.window, a.c.block) : 0;
+    const int my_pos = pos0 + row, my_lo = first_seen(my_pos, a.window, a.chunk), my_seen = a.c.block > 0 ? pooled_seen(my_pos, a.window, a.c.block) : 0;
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const float sl2 = a.scale * 1.4426950408889634f;
     const int oc0 = qt * (vcp / 4), oc1 = oc0 + vcp / 4;
@@ -388,6 +389,7 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
     const float l = (xs[0] + xs[TQ]) + (xs[2 * TQ] + xs[3 * TQ]);
     const float inv = *dead ? __int_as_float(0x7fffffff) : (l > 0.f ? 1.0f / l : 0.f);
     const size_t rs_rec = (size_t)vcols + 2;
+    const int wrow0 = row0 + (warp & 3) * 32;
     float* rec = a.ws + ((size_t)(row0 + (warp & 3) * 32) * a.heads + h) * rs_rec;  // record of the warp's first row
     const size_t row_step = (size_t)a.heads * rs_rec;
     const int wrows = min(32, nrows - (warp & 3) * 32);
@@ -404,8 +406,16 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_talk_tc_kernel(const GqaAttnArgs 
       }
       __syncwarp();
       const int x = lane & (cw - 1), cc = c + x, rstep = 32 / cw;
-      if (cc < nv)
+      if (cc >= nv) continue;
+      if (a.talk) {
         for (int i = lane / cw; i < wrows; i += rstep) rec[i * row_step + 2 + col0 + cc] = tr[i * TURN + x];
+      } else {
+        const size_t oc = (size_t)h * a.vdim + zc + cc;
+        for (int i = lane / cw; i < wrows; i += rstep) {
+          if (a.out_bf) a.out_bf[(size_t)(wrow0 + i) * a.ldo_bf + oc] = f2bf(tr[i * TURN + x]);
+          else a.out[(size_t)(wrow0 + i) * a.ldo + oc] = tr[i * TURN + x];
+        }
+      }
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -423,7 +433,7 @@ struct TcPlan {
 };
 TcPlan tc_plan(const GqaAttnArgs& a) {
   TcPlan p;
-  const int vcols = a.kv_heads * a.vdim;
+  const int vcols = a.talk ? a.kv_heads * a.vdim : a.vdim;
   p.dblk = (a.dim + 63) / 64;
   p.nvc = (vcols + 255) / 256;
   p.vc = ((vcols + p.nvc - 1) / p.nvc + 7) / 8 * 8;
@@ -436,18 +446,18 @@ TcPlan tc_plan(const GqaAttnArgs& a) {
 
 }  // namespace
 
-bool gqa_talk_tc_fits(const GqaAttnArgs& a) {
-  return a.talk && a.c.elt_bytes == 2 && a.seg_start && a.n >= 128 && a.n / a.n_seg >= 64 && a.dim <= 128 && a.dim % 8 == 0 && (a.kv_heads * a.vdim) % 8 == 0 &&
-         a.maps == 1 && a.scale > 0.f && a.keep_first == 0 && a.softcap == 0.f && !a.slopes && !a.shared_keys && a.c.page_elems % 8 == 0 && a.c.layer_off % 8 == 0 &&
+bool gqa_tc_fits(const GqaAttnArgs& a) {
+  return a.c.elt_bytes == 2 && a.seg_start && a.n >= 128 && a.n / a.n_seg >= 64 && a.dim <= 128 && a.dim % 8 == 0 &&
+         (a.talk ? a.kv_heads * a.vdim : a.vdim) % 8 == 0 && a.heads % a.kv_heads == 0 && a.finish == 0 && !a.unit_sink && a.maps == 1 && a.scale > 0.f && a.keep_first == 0 && a.softcap == 0.f && !a.slopes && !a.shared_keys && a.c.page_elems % 8 == 0 && a.c.layer_off % 8 == 0 &&
          (a.c.kw + a.c.vw) % 8 == 0 && a.c.kw % 8 == 0 && (!a.c.block || (a.c.pool_off % 8 == 0 && a.window > 0)) &&
          (reinterpret_cast<uintptr_t>(a.c.pool) & 15) == 0 && a.heads <= 65535;
 }
 
-cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st) {
+cudaError_t launch_gqa_tc(const GqaAttnArgs& a, cudaStream_t st) {
   const TcPlan p = tc_plan(a);
   static PerDeviceOnce once;
   if (once.need()) {
-    cudaError_t r = cudaFuncSetAttribute(gqa_talk_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
+    cudaError_t r = cudaFuncSetAttribute(gqa_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
     if (r != cudaSuccess) return r;
     once.done();
   }
@@ -457,7 +467,7 @@ cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st) {
   const int use_tma = a.c.n_pages > 0 && row >= 64 && (ps % TK == 0 || (TK % ps == 0 && ps >= 8)) &&
                       make_tensor_map_pages(&tm, static_cast<const bf16*>(a.c.pool) + a.c.layer_off, row, ps, a.c.n_pages, a.c.page_elems,
                                             std::min(ps, TK)) == cudaSuccess;
-  return launch_k(gqa_talk_tc_kernel, dim3(a.heads, a.n / TQ + a.n_seg, p.nvc), dim3(NTHR), p.smem, st, a, p.dblk, p.vblk, p.nst, p.vc,
+  return launch_k(gqa_tc_kernel, dim3(a.heads, a.n / TQ + a.n_seg, p.nvc), dim3(NTHR), p.smem, st, a, p.dblk, p.vblk, p.nst, p.vc,
                   *reinterpret_cast<const CUtensorMap*>(&tm), use_tma);
 }
 

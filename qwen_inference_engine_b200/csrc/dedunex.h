@@ -36,11 +36,14 @@ namespace qie {
 // ---------------------------------------------------------------- grouped RMS norm around a parallel block (rmsnorm_f32.cu)
 // gnorm(v) w: v is split into `groups` equal consecutive parts, each divided by its own sqrt(mean(part^2) + eps), the
 // whole multiplied by w.  One CTA per row r, src(r) = gather ? gather[r] : r, in this order (every part optional):
-//   source  x[src] as it is, or (ids != null) gnorm(embed[ids[r]]) w_pre : the first norm of a model that norms its embedding
-//   add     x[src] += y1[src] + y2[src]       the two sublayer outputs of the block before (fp32 or dense bf16 rows)
+//   source  x[src] as it is, or (ids != null) the embedding: embed[ids[r]] * embed_scale, or with w_pre gnorm(embed[ids[r]]) w_pre
+//   add     x[src] += y1[src] + y2[src]       the sublayer outputs of the block before (fp32 or dense bf16 rows)
+//           x[src] += sum_k w_k ye[slot_k]    the experts' outputs (mix; as bf16 rows in ye_bf; without mix.top_w every w_k is 1)
 //   dump    dump[r] = x[src]                  the stream after a layer, for the parity hook
 //   step    x[src] += step                    a vector of the model (before a pass of a loop)
-//   read    h[r] = gnorm(x[src]) w_in         fp32 rows and / or dense bf16 rows
+//   again   x[src] += embed[ids[r]] * embed_scale   the embedding once more (before a pass of a loop; the source is then x itself)
+//   read    h[r] = gnorm(x[src]) (w_off + w_in)   fp32 rows and / or dense bf16 rows (w_off 1: a weight stored around zero)
+//   route   the router's logits and choice of the row just read (RouteRider)
 // x[src] is written back when it changed.
 struct GroupNormStep {
   float* x = nullptr;
@@ -49,16 +52,22 @@ struct GroupNormStep {
   const int* ids = nullptr;
   const bf16* embed = nullptr;
   const bf16* w_pre = nullptr;
+  float embed_scale = 1.f;
+  int again = 0;
   const float* y1 = nullptr;
   const float* y2 = nullptr;
   const bf16* y1_bf = nullptr;
   const bf16* y2_bf = nullptr;
+  MoeMix mix;
+  const bf16* ye_bf = nullptr;
   float* dump = nullptr;
   const bf16* step = nullptr;
   const bf16* w_in = nullptr;
+  float w_off = 0.f;
   float* h = nullptr;
   bf16* h_bf = nullptr;
   const int* gather = nullptr;
+  RouteRider route;
 };
 cudaError_t launch_group_norm_step(const GroupNormStep& a, cudaStream_t st);
 

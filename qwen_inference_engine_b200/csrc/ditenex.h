@@ -8,7 +8,7 @@
 // embedding table.  Residual stream, norms, softmax, router and the carried rows are fp32.
 //
 // The mechanisms are launchers with their constants as arguments so that another design can use them: the norms and
-// the token shift (rmsnorm_f32.cu), the activations (activations.cu), the router (moe_route.cuh), the query mixing, distance
+// the token shift (rmsnorm_f32.cu), the activations (activations.cu), the router (moe_route.cuh; RouteRider in nogatar.h), the query mixing, distance
 // slopes, shared keys and elementwise gate of the paged attention (attn_gqa.cu, fosavik.h).  ditenex_model.cu holds the
 // configuration reader, the weight loader and the launch order.  The family shares the engine's sequences, page
 // allocator, block tables, row metadata, sampler, scheduler and C ABI with the other families (engine.h, family.h).
@@ -32,19 +32,7 @@ namespace qie {
 //   add  (y != null or mix.ye != null):  x[r] += mult * rms(y[r]) w_out      (y may be the mixture-of-experts combine
 //                                        of the row, computed on the fly from `mix`; mix.z == null: shared expert ungated)
 //   read (h != null):                    h[r] = rms(x[src(r)]) w_in,  src(r) = gather ? gather[r] : r
-// Rider of the read half in front of a mixture of experts: the row's router logits z_e = w_router[e, :] . h (fp32, from the
-// normed row while it is in shared memory) and the choice (moe_route.cuh), by the same CTA:
-// s = sigmoid(z); choice score c = s + correction.  The experts form `groups` equal runs of neighbours; a group's score is
-// the sum of its two largest c; only experts of the `keep` best groups can be chosen; the `top` largest c among them
-// (lowest index first among equals) are chosen with weights s * scale (not renormalised).
-struct RouteRider {
-  const bf16* w_router = nullptr;  // [experts, width]; null: no rider
-  const bf16* correction = nullptr;
-  int experts = 0, top = 0, groups = 1, keep = 1;
-  float scale = 1.f;
-  int* top_idx = nullptr;  // [n, top]
-  float* top_w = nullptr;
-};
+// The router's logits and choice may ride the read half (RouteRider, nogatar.h).
 struct RmsStep {
   float* x = nullptr;
   int width = 0, n = 0;
@@ -88,8 +76,8 @@ cudaError_t launch_rms_shift(const RmsShiftArgs& a, cudaStream_t st);
 //   z > 0: softplus(pq[0]) z^2 + z / 2;   z <= 0: (1/2 + softplus(pq[1])) (exp(z) - 1 - z) + z / 2
 cudaError_t launch_xielu(float* z, int ld, int cols, const bf16* pq, int n, cudaStream_t st);
 cudaError_t launch_xielu_bf16(bf16* z, int ld, int cols, const bf16* pq, int n, cudaStream_t st);  // bf16 rows, fp32 arithmetic
-// out[r, c] = silu(gu[r, c]) * gu[r, ff + c]
-cudaError_t launch_silu_glu(const float* gu, int ld, float* out, int ldo, int ff, int n, cudaStream_t st);
+// out[r, c] = silu(gu[r, c]) * gu[r, ff + c]; with row_w both are first multiplied by row_w[r] (a scaled input of the two linear maps)
+cudaError_t launch_silu_glu(const float* gu, int ld, float* out, int ldo, int ff, int n, cudaStream_t st, const float* row_w = nullptr);
 cudaError_t launch_silu_glu_bf16(const bf16* gu, int ld, bf16* out, int ldo, int ff, int n, cudaStream_t st);
 
 // ---------------------------------------------------------------- the model (ditenex_model.cu)

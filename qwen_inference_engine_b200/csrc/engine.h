@@ -17,6 +17,7 @@
 #include "ditenex.h"
 #include "fosavik.h"
 #include "gebadra.h"
+#include "gubanex.h"
 #include "nogatar.h"
 #include "tp_nccl.h"
 
@@ -46,14 +47,15 @@ struct CaptureBuf {
 }  // namespace qie
 
 struct qie_engine {
-  // model family: Qwen (the members below named after its operators) unless `fam` is set (nogatar.h, fosavik.h, ditenex.h, dedunex.h, gebadra.h); sequences, pages,
+  // model family: Qwen (the members below named after its operators) unless `fam` is set (nogatar.h, fosavik.h, ditenex.h, dedunex.h, gebadra.h, gubanex.h); sequences, pages,
   // block tables, row metadata, sampling and graphs are shared by the families
-  qie::RowFamily* fam = nullptr;  // the family's interface (family.h); ng / fv / dx / dd / gb below are the same object, typed
+  qie::RowFamily* fam = nullptr;  // the family's interface (family.h); ng / fv / dx / dd / gb / gx below are the same object, typed
   qie::NgModel* ng = nullptr;
   qie::FvModel* fv = nullptr;
   qie::DxModel* dx = nullptr;
   qie::DdModel* dd = nullptr;
   qie::GbModel* gb = nullptr;
+  qie::GxModel* gx = nullptr;
   qie_config cfg{};
   qie_engine_opts opts{};
   int num_sms = 0;

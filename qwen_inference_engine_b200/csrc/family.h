@@ -1,5 +1,5 @@
-// family.h -- what the model families with a general row forward share (Nogatar, Fosavik, Ditenex, Dedunex, Gebadra): the interface the engine
-// drives them through (forward over rows, slot reset, release), the weight blob helpers (tensor layout, safetensors
+// family.h -- what the model families with a general row forward share (Nogatar, Fosavik, Ditenex, Dedunex, Gebadra, Gubanex): the
+// interface the engine drives them through (forward over rows, slot reset, release), the weight blob helpers (tensor layout, safetensors
 // reader, synthetic fill), the rotary tables and the projection helper that puts a plain GEMM on the tcgen05 kernel when
 // precision and shape allow.  A row is (sequence slot, position); rows of one sequence are consecutive and in position order
 // (a "segment"); rows of different sequences may be portions of prompts next to single decoded tokens.
@@ -7,6 +7,7 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <map>
 #include <string>
 #include <vector>
 
@@ -51,7 +52,7 @@ struct TensorSpec {
   std::string name;
   size_t rows = 0, cols = 0;  // cols 0 = vector of `rows`
   size_t off = 0;             // element offset in the blob
-  int kind = 0;               // synthetic fill: 0 matrix (uniform, variance 1/cols), 1 norm weight (about 1), 2 small vector; 3: zeros that no file holds
+  int kind = 0;               // synthetic fill: 0 matrix (uniform, variance 1/cols), 1 norm weight (about 1), 2 small vector; 3: zeros that no file holds; 4: norm weight stored around zero
   size_t elems() const { return rows * (cols ? cols : 1); }
 };
 // appends tensors to a layout; pad() starts the next group on a 256-byte boundary (tensors that one GEMM reads as a
@@ -73,22 +74,28 @@ uint16_t f32_to_bf16_bits(float f);
 void fill_synthetic_blob(const std::vector<TensorSpec>& t, uint64_t seed, std::vector<uint16_t>* blob);
 // reads every tensor of the layout from a safetensors file (BF16 only; shapes are checked by element count) -> "" or the error
 std::string load_safetensors_blob(const std::string& path, const std::vector<TensorSpec>& t, std::vector<uint16_t>* blob);
+// shapes by tensor name, for sizes that only the file gives (reads the header alone) -> "" or the error
+std::string safetensors_shapes(const std::string& path, std::map<std::string, std::vector<size_t>>* shapes);
 
 // ---------------------------------------------------------------- rotary positions
 // Rotation angles of position p: a_i = p * f_i, f_i = base^(-2i / dims), i < dims / 2.  With `scaled` (YaRN) the
 // frequencies are blended: with corr(t) = dims * ln(original / (2 pi t)) / (2 ln base), lo = max(floor(corr(fast)), 0),
 // hi = min(ceil(corr(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is
 // f_i / factor * ramp_i + f_i * (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.  `linear` divides every
-// frequency (linear position scaling).
+// frequency (linear position scaling).  With `by_wave` a frequency is scaled by its wavelength l = 2 pi / f_i: kept below
+// original / high, divided by factor above original / low, and between them blended, (1 - s) f_i / factor + s f_i with
+// s = (original / l - low) / (high - low); cos and sin keep their size.
 struct RotaryCfg {
   int dims = 0;
   double base = 10000.0;
   bool scaled = false;
   double factor = 1.0, original = 0.0, fast = 0.0, slow = 0.0;
   double linear = 1.0;
+  bool by_wave = false;  // uses factor and original
+  double low = 0.0, high = 0.0;
   bool operator==(const RotaryCfg& o) const {
     return dims == o.dims && base == o.base && scaled == o.scaled && factor == o.factor && original == o.original && fast == o.fast &&
-           slow == o.slow && linear == o.linear;
+           slow == o.slow && linear == o.linear && by_wave == o.by_wave && low == o.low && high == o.high;
   }
 };
 // cos / sin tables [context, dims / 2], worked out in double, the magnitude factor folded in

@@ -49,26 +49,51 @@ void fill_synthetic_blob(const std::vector<TensorSpec>& t, uint64_t seed, std::v
     const float a = s.kind == 0 ? sqrtf(3.0f / (float)s.cols) : 0.f;
     for (size_t i = 0; i < s.elems(); ++i) {
       const float u = hash_uniform(seed + 1315423911ull * k, i);
-      const float v = s.kind == 0 ? a * u : (s.kind == 1 ? 1.0f + 0.1f * u : 0.5f * u);
+      const float v = s.kind == 0 ? a * u : (s.kind == 1 ? 1.0f + 0.1f * u : (s.kind == 4 ? 0.1f : 0.5f) * u);
       (*blob)[s.off + i] = f32_to_bf16_bits(v);
     }
   }
 }
 
+// the header of an open safetensors file and the offset of its data -> "" or the error
+static std::string read_safetensors_header(FILE* f, const std::string& path, JsonValue* root, size_t* data0) {
+  unsigned char lenb[8];
+  if (fread(lenb, 1, 8, f) != 8) return "short safetensors file " + path;
+  uint64_t hl = 0;
+  for (int i = 7; i >= 0; --i) hl = (hl << 8) | lenb[i];
+  if (hl == 0 || hl > ((uint64_t)1 << 30)) return "bad safetensors header length in " + path;
+  std::string hdr((size_t)hl, '\0'), err;
+  if (fread(&hdr[0], 1, (size_t)hl, f) != (size_t)hl) return "short safetensors header in " + path;
+  if (!JsonReader::parse(hdr.data(), hdr.data() + hdr.size(), root, &err)) return path + ": " + err;
+  *data0 = 8 + (size_t)hl;
+  return "";
+}
+
+std::string safetensors_shapes(const std::string& path, std::map<std::string, std::vector<size_t>>* shapes) {
+  FILE* f = fopen(path.c_str(), "rb");
+  if (!f) return "cannot open " + path;
+  JsonValue root;
+  size_t data0 = 0;
+  const std::string err = read_safetensors_header(f, path, &root, &data0);
+  fclose(f);
+  if (!err.empty()) return err;
+  for (const auto& kv : root.obj) {
+    const JsonValue* sh = kv.second.have("shape");
+    if (!sh || sh->kind != JsonValue::Array) continue;
+    std::vector<size_t> v;
+    for (const JsonValue& d : sh->arr) v.push_back((size_t)llround(d.num));
+    (*shapes)[kv.first] = v;
+  }
+  return "";
+}
+
 std::string load_safetensors_blob(const std::string& path, const std::vector<TensorSpec>& t, std::vector<uint16_t>* blob) {
   FILE* f = fopen(path.c_str(), "rb");
   if (!f) return "cannot open " + path;
-  unsigned char lenb[8];
-  if (fread(lenb, 1, 8, f) != 8) return fclose(f), "short safetensors file " + path;
-  uint64_t hl = 0;
-  for (int i = 7; i >= 0; --i) hl = (hl << 8) | lenb[i];
-  if (hl == 0 || hl > ((uint64_t)1 << 30)) return fclose(f), "bad safetensors header length in " + path;
-  std::string hdr((size_t)hl, '\0');
-  if (fread(&hdr[0], 1, (size_t)hl, f) != (size_t)hl) return fclose(f), "short safetensors header in " + path;
   JsonValue root;
-  std::string err;
-  if (!JsonReader::parse(hdr.data(), hdr.data() + hdr.size(), &root, &err)) return fclose(f), path + ": " + err;
-  const size_t data0 = 8 + (size_t)hl;
+  size_t data0 = 0;
+  const std::string err = read_safetensors_header(f, path, &root, &data0);
+  if (!err.empty()) return fclose(f), err;
   for (const TensorSpec& s : t) {
     if (s.kind == 3) continue;  // not in the file: zero rows between the parts of a fused matrix
     const JsonValue* rec = root.have(s.name.c_str());
@@ -134,6 +159,15 @@ void rotary_tables(const RotaryCfg& r, int context, std::vector<float>* c, std::
       f[i] = f[i] / r.factor * ramp + f[i] * (1.0 - ramp);
     }
     mag = 0.1 * log(r.factor) + 1.0;
+  }
+  if (r.by_wave) {
+    const double PI = 3.14159265358979323846;
+    for (int i = 0; i < half; ++i) {
+      const double wave = 2.0 * PI / f[i];
+      if (wave < r.original / r.high) continue;
+      const double s = wave > r.original / r.low ? 0.0 : r.high > r.low ? (r.original / wave - r.low) / (r.high - r.low) : 1.0;
+      f[i] = (1.0 - s) * f[i] / r.factor + s * f[i];
+    }
   }
   c->resize((size_t)context * half);
   s->resize((size_t)context * half);

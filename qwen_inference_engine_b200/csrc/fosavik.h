@@ -85,9 +85,12 @@ inline int kv_pool_rows(int page_size, int block) { return block > 0 ? (page_siz
 // Optional: biases added to keys and values first; values blended with another layer's values of the same rows,
 // v = (1 - lam) v + lam v_other (lam one bf16 number on the device); the stored values also kept as fp32 rows (v_keep);
 // the head-mixed queries of the row (TalkQueries below) written in the same launch.
+// unit_norm: queries and keys are normed per `norm_dim` elements without a weight (k_norm and q_norm null).  The rotation keeps the
+// length of what it turns, so this is also the norm of the rotated vectors.
 // whole_norm: the unit RMS norm of the keys (and of the queries) goes over the row's whole key part (all its query heads)
 // at once, with weights k_norm [kw] and q_norm [q_heads * norm_dim]; norm_dim is then the head size that rotates.  In this form
-// the sources may be bf16 rows (*_bf, row stride ld_bf) and the queries go from q_bf to the fp32 rows q.
+// the sources may be bf16 rows (*_bf, row stride ld_bf) and the queries go from q_bf to the fp32 rows q; without whole_norm bf16
+// sources run a warp per row, for the shapes that kv_store_heads_fits accepts.
 // Pooled rows (c.block > 0): the row that holds a block's last position is followed by the block's mean row, in the same
 // launch when every row of the batch is another sequence's (one_each), else by launch_kv_pool_rows.
 // Rotary positions (rope.dims > 0): after the norm, the first rope.dims elements of every `norm_dim` consecutive elements
@@ -121,7 +124,7 @@ struct KvStoreArgs {
   const bf16* v_bias = nullptr;  // [vw]
   const bf16* q_bias = nullptr;  // [q_heads * norm_dim]
   RopeTable rope;
-  int whole_norm = 0, one_each = 0;
+  int whole_norm = 0, one_each = 0, unit_norm = 0;
   const bf16 *q_bf = nullptr, *k_bf = nullptr, *v_bf = nullptr;
   int ld_bf = 0;
   const bf16* v_lam = nullptr;
@@ -134,9 +137,13 @@ struct KvStoreArgs {
   int max_pages = 0, n = 0;
 };
 cudaError_t launch_kv_store_rows(const KvStoreArgs& a, cudaStream_t st);
+// bf16 sources with a unit norm per head: whole 16-byte pieces, head sizes of 8, 16, 32, 64, 128 or 256, pairs (i, i + dims/2)
+bool kv_store_heads_fits(const KvStoreArgs& a);
 // pooled rows of every block whose last position is among the n rows (their keys and values are in the cache already)
 cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st);
 // out[r, h, :] over the keys j of row r's sequence with j <= pos and (window <= 0 or pos - j < window or j < keep_first).
+// chunk > 0 (instead of a window): the positions fall into chunks of `chunk`, counted from position 0 of the sequence, and a row sees
+// the keys of its own chunk up to itself.
 // `maps` score maps per head (queries [h][map][dim], keys [g][map][dim]) share the values [g][vdim]; head h reads kv
 // head h / (heads / kv_heads).  unit_sink adds 1 to every softmax denominator (as if one more key with a zero score and nothing to contribute took part).
 // finish 0: out = a_1;  1: out = a_1 * sigmoid(gate[r, h]);  2 (maps == 2): o = a_1 - lam * a_2, out = o / sqrt(mean(o^2) + eps) * post;
@@ -162,7 +169,7 @@ struct GqaAttnArgs {
   int ldo_bf = 0;
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0, maps = 1;
   float scale = 1.f, softcap = 0.f;
-  int window = 0, keep_first = 0, unit_sink = 0;
+  int window = 0, chunk = 0, keep_first = 0, unit_sink = 0;
   int finish = 0;
   const float* gate = nullptr;
   int ldg = 0;
@@ -185,10 +192,10 @@ struct GqaAttnArgs {
 // (vdim: with `talk` the value elements of all kv heads together)
 inline size_t gqa_ws_floats(int n, int heads, int maps, int vdim) { return (size_t)n * heads * maps * (vdim + 2); }
 cudaError_t launch_gqa_attention(const GqaAttnArgs& a, cudaStream_t st, int* n_launches = nullptr);
-// the tcgen05 form of a prompt portion's attention with `talk` (attn_gqa_tc.cu), without the mix of the heads: the normalised result
-// of every head over the values of all kv heads goes to its workspace record; launch_gqa_attention picks it
-bool gqa_talk_tc_fits(const GqaAttnArgs& a);
-cudaError_t launch_gqa_talk_tc(const GqaAttnArgs& a, cudaStream_t st);
+// the tcgen05 form of a prompt portion's attention (attn_gqa_tc.cu): plain heads, or with `talk` without the mix of the heads (the
+// normalised result of every head over the values of all kv heads goes to its workspace record); launch_gqa_attention picks it
+bool gqa_tc_fits(const GqaAttnArgs& a);
+cudaError_t launch_gqa_tc(const GqaAttnArgs& a, cudaStream_t st);
 
 // ---------------------------------------------------------------- short convolution and recurrences (recurrent.cu)
 // Causal per-channel convolution over the rows of each segment: out[t, c] = act(b[c] + sum_i w[c, i] * in(t - (taps-1-i), c)),

@@ -32,29 +32,44 @@ struct qie_engine;
 
 namespace qie {
 
-// ---------------------------------------------------------------- linear attention with a fixed decay (linear_attn.cu)
+// ---------------------------------------------------------------- linear attention with a fixed or a gated decay (linear_attn.cu)
 // Per head h over the rows of each segment, state S [dim, vdim] of slot s at state + s * slot_stride + h * dim * vdim (fp32, carried):
-//   S = decay_h S + (k_scale k_t) v_t^T,   o_t = S^T q_t          with act 1: q, k, v = silu of the rows read
+//   S = diag(decay) S + (k_scale k_t) v_t^T,   o_t = S^T (q_scale q_t)          with act 1: q, k, v = silu of the rows read
 // q [n, heads * dim], k alike, v [n, heads * vdim] are columns of fp32 rows (row stride ld) or of bf16 rows (*_bf, ld_bf).
-// decay_pow: [heads][LINEAR_CHUNK + 1] the powers decay_h^0 .. decay_h^LINEAR_CHUNK on the device.
-// The result goes to fp32 rows.  With norm_gate (only where linear_attention_chunked says so) each head's o is divided by
-// sqrt(mean(o^2) + eps), multiplied by silu(g_bf[t, h * vdim + c]) and written as bf16 rows instead.
+// The decay is one fixed number per head, or (gate.a2 != null) one per key channel that every token gates:
+//   decay_pow: [heads][LINEAR_CHUNK + 1] the powers decay_h^0 .. decay_h^LINEAR_CHUNK on the device
+//   gate:      decay_t[h, d] = sigmoid(z)^inv_tau, z = a2[h * dim + d, :] . low_t + bias[h * dim + d], low_t the token's low-rank row
+// The result goes to fp32 rows.  With norm_gate (only where linear_attention_norm_fits says so) each head's o is divided by
+// sqrt(mean(o^2) + eps), multiplied by norm_w (null: 1) and silu(g_bf[t, h * vdim + c]) and written as bf16 rows instead.
 // bf16 sources, LINEAR_CHUNK rows and more and a workspace: portions run in chunks of LINEAR_CHUNK rows on tensor cores (each chunk's own
 // contribution to the state, a carry pass over the chunks, then the outputs of all chunks side by side); else token by token.
 constexpr int LINEAR_CHUNK = 64;
+struct GatedDecay {
+  const float* low = nullptr;  // [n, rank] columns of fp32 rows (row stride LinearAttnArgs::ld) or of bf16 rows (low_bf, ld_bf)
+  const bf16* low_bf = nullptr;
+  int rank = 0;
+  const bf16* a2 = nullptr;    // [heads * dim, rank]
+  const bf16* bias = nullptr;  // [heads * dim]
+  float inv_tau = 1.f;
+  float* cum = nullptr;  // workspace of the chunked form, gated_decay_floats(): log2 of the decays, summed up inside every chunk
+};
+__host__ __device__ inline int gated_decay_pitch(int dim) { return (dim + 3) / 4 * 4; }  // floats per head and row
+inline size_t gated_decay_floats(size_t rows, int heads, int dim) { return rows * heads * gated_decay_pitch(dim); }
 struct LinearAttnArgs {
   const float *q = nullptr, *k = nullptr, *v = nullptr;
   int ld = 0;
   const bf16 *q_bf = nullptr, *k_bf = nullptr, *v_bf = nullptr;
   int ld_bf = 0;
   int act = 0;
-  float k_scale = 1.f;
+  float k_scale = 1.f, q_scale = 1.f;
   int heads = 0, dim = 0, vdim = 0;
   const float* decay_pow = nullptr;
+  GatedDecay gate;
   float* out = nullptr;
   int ldo = 0;
   int norm_gate = 0;
   const bf16* g_bf = nullptr;  // row stride ld_bf
+  const bf16* norm_w = nullptr;  // [vdim], the same for every head
   float eps = 0.f;
   bf16* out_bf = nullptr;
   int ldo_bf = 0;
@@ -69,12 +84,14 @@ struct LinearAttnArgs {
 inline size_t linear_ws_floats(size_t rows, size_t segs, int heads, int dim, int vdim) {
   return (rows / LINEAR_CHUNK + segs + 1) * heads * (size_t)dim * vdim;
 }
-// does the chunked form run (and so can norm_gate be asked for)?
+// does the chunked form run, and can norm_gate be asked for (one CTA holds a head's values whole)?
 bool linear_attention_chunked(const LinearAttnArgs& a);
+bool linear_attention_norm_fits(const LinearAttnArgs& a);
 cudaError_t launch_linear_attention(const LinearAttnArgs& a, cudaStream_t st, int* n_launches = nullptr);
 
 // ---------------------------------------------------------------- norm, then gate (rmsnorm_f32.cu)
-// out[r, c] = v[r, c] / sqrt(mean_group(v[r]^2) + eps) * w[c] * act(g[r, c]);  `groups` equal parts of `width`; w null: 1;
+// out[r, c] = v[r, c] / sqrt(mean_group(v[r]^2) + eps) * w[c] * act(g[r, c]);  `groups` equal parts of `width`; w null: 1
+// (w_shared: w holds one part's weights, the same for every part);
 // act 0: silu, 1: sigmoid.  g: fp32 rows or bf16 rows; the result goes to fp32 rows and / or bf16 rows.
 struct NormGate {
   const float* v = nullptr;
@@ -84,7 +101,7 @@ struct NormGate {
   const bf16* g_bf = nullptr;
   int ldg_bf = 0;
   const bf16* w = nullptr;
-  int width = 0, groups = 1, act = 0, n = 0;
+  int width = 0, groups = 1, act = 0, n = 0, w_shared = 0;
   float eps = 0.f;
   float* out = nullptr;
   int ldo = 0;

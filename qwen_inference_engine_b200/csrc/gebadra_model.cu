@@ -435,7 +435,7 @@ cudaError_t GbModel::forward(qie_engine* e, int n, int n_seg, int n_out, int max
       a.seg_start = segs, a.seg_slot = seg_sl, a.n_seg = n_seg, a.n_rows = n;
       a.ws = m->scan_ws, a.ws_floats = m->scan_ws_floats;
       // retention's norm covers one head, which a chunk's CTA holds whole
-      const bool fused = L.type == 1 && tc_lo && linear_attention_chunked(a);
+      const bool fused = L.type == 1 && tc_lo && linear_attention_norm_fits(a);
       if (fused) a.norm_gate = 1, a.out_bf = m->rb, a.ldo_bf = nv;
       int nl = 0;
       FAM_TRY(KK_LINEAR_ATTN, launch_linear_attention(a, st, &nl));

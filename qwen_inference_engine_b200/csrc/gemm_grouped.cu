@@ -105,11 +105,12 @@ __global__ void __launch_bounds__(256) grouped_gemm_bf16_kernel(const GroupedGem
       for (int u = 0; u < 4; ++u) {
         const int m = m0 + wm + mt * 16 + gq + (u >> 1) * 8;
         if (m >= Mz) continue;
+        const float rw = g.row_w ? g.row_w[row_base + m] : 1.f;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
           const int col = cw + nt * 8 + 2 * tq + (u & 1);
           if (col >= n_out) continue;
-          const float gate = acc[mt][nt][u], up = acc[mt][nt + 2][u];
+          const float gate = acc[mt][nt][u] * rw, up = acc[mt][nt + 2][u] * rw;
           g.out_bf[(size_t)(row_base + m) * g.ldo + col] = f2bf(gate / (1.0f + expf(-gate)) * up);
         }
       }
@@ -120,11 +121,14 @@ __global__ void __launch_bounds__(256) grouped_gemm_bf16_kernel(const GroupedGem
       for (int u = 0; u < 4; ++u) {
         const int m = m0 + wm + mt * 16 + gq + (u >> 1) * 8;
         if (m >= Mz) continue;
+        const float rw = g.row_w ? g.row_w[row_base + m] : 1.f;
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
           const int col = c0 + wn + nt * 8 + 2 * tq + (u & 1);
           if (col >= g.N) continue;
-          g.out[(size_t)(row_base + m) * g.ldo + col] = acc[mt][nt][u];
+          const float v = acc[mt][nt][u] * rw;
+          if (g.out_bf) g.out_bf[(size_t)(row_base + m) * g.ldo + col] = f2bf(v);
+          else g.out[(size_t)(row_base + m) * g.ldo + col] = v;
         }
       }
   }
@@ -139,7 +143,7 @@ bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g) {
 
 cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st) {
   if (g.rows <= 0 || g.groups <= 0) return cudaSuccess;
-  if (!grouped_gemm_bf16_fits(g) || !g.grp_off || (g.gated ? !g.out_bf : !g.out)) return cudaErrorInvalidValue;
+  if (!grouped_gemm_bf16_fits(g) || !g.grp_off || (g.gated ? !g.out_bf : !(g.out || g.out_bf))) return cudaErrorInvalidValue;
   const size_t smem = (size_t)2 * STAGES * BM * BKP * sizeof(bf16);  // 60 KB
   static PerDeviceOnce set;
   if (set.need()) {

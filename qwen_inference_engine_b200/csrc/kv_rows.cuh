@@ -17,6 +17,11 @@ __device__ __forceinline__ const char* kv_pool_ptr(const KvRowCache& c, const in
   const size_t off = (size_t)page * c.page_elems + c.pool_off + (size_t)(b - pi * c.page_size / c.block) * (c.kw + c.vw);
   return static_cast<const char*>(c.pool) + off * c.elt_bytes;
 }
+// the first position that a row at pos sees below itself: its window's edge or its chunk's start (kept first tokens aside)
+__host__ __device__ __forceinline__ int first_seen(int pos, int window, int chunk) {
+  if (chunk > 0) return pos / chunk * chunk;
+  return window > 0 && pos >= window ? pos - window + 1 : 0;
+}
 // blocks that end before the window of position pos begins: (b + 1) * block - 1 <= pos - window
 __host__ __device__ __forceinline__ int pooled_seen(int pos, int window, int block) { return block > 0 && pos >= window ? (pos - window + 1) / block : 0; }
 

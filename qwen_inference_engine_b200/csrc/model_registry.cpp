@@ -25,6 +25,7 @@ const Row kRegistry[] = {
     {"Ditenex", FAMILY_DITENEX},
     {"Dedunex", FAMILY_DEDUNEX},
     {"Gebadra", FAMILY_GEBADRA},
+    {"Gubanex", FAMILY_GUBANEX},
     {"Qwen2ForCausalLM", FAMILY_QWEN},
     {"Qwen3ForCausalLM", FAMILY_QWEN},
 };

@@ -67,7 +67,8 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int ldz, int exper
 
 // one CTA; warp w serves experts w, w + nw, ...: an ordered compaction of the assignments that chose the expert
 __global__ void __launch_bounds__(1024) moe_group_kernel(const int* top_idx, int n_assign, int top, int experts, int* grp_off,
-                                                         int* __restrict__ perm_row, int* __restrict__ slot_of, int in_smem) {
+                                                         int* __restrict__ perm_row, int* __restrict__ slot_of, const float* __restrict__ top_w,
+                                                         float* __restrict__ perm_w, int in_smem) {
   extern __shared__ int s_idx[];  // the assignments, when they fit (in_smem)
   pdl_wait();
   pdl_trigger();
@@ -106,6 +107,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* top_idx, int
         const int s = base + __popc(b & ((1u << lane) - 1u));
         perm_row[s] = i / top;
         slot_of[i] = s;
+        if (perm_w) perm_w[s] = top_w[i];
       }
       base += __popc(b);
     }
@@ -117,7 +119,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* top_idx, int
 // (expert, warp) gives every warp its first slot per expert, pass 2 hands out the slots: ascending assignment order within
 // an expert, exactly as the kernel above.  Shared memory: base [32][experts] ints.
 __global__ void __launch_bounds__(1024) moe_group_chunked_kernel(const int* __restrict__ top_idx, int n_assign, int top, int experts,
-                                                                 int* __restrict__ grp_off, int* __restrict__ perm_row, int* __restrict__ slot_of) {
+                                                                 int* __restrict__ grp_off, int* __restrict__ perm_row, int* __restrict__ slot_of,
+                                                                 const float* __restrict__ top_w, float* __restrict__ perm_w) {
   extern __shared__ int base[];  // [32][experts]
   pdl_wait();
   pdl_trigger();
@@ -172,6 +175,7 @@ __global__ void __launch_bounds__(1024) moe_group_chunked_kernel(const int* __re
       const int slot = mine[e] + __popc(peers & ((1u << lane) - 1u));
       perm_row[slot] = i / top;
       slot_of[i] = slot;
+      if (perm_w) perm_w[slot] = top_w[i];
     }
     __syncwarp();
     if (on && (peers & ((1u << lane) - 1u)) == 0) mine[e] += __popc(peers);
@@ -206,15 +210,18 @@ cudaError_t launch_moe_route(const float* z, int ldz, int experts, int top, int*
                   top, top_idx, top_w, n);
 }
 
-cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int experts, int* grp_off, int* perm_row, int* slot_of, cudaStream_t st) {
+cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int experts, int* grp_off, int* perm_row, int* slot_of, cudaStream_t st,
+                             const float* top_w, float* perm_w) {
   if (n_assign <= 0) return cudaSuccess;
+  if (perm_w && !top_w) return cudaErrorInvalidValue;
   if (n_assign >= 1024 && experts <= 1024) {  // many assignments: chunks over the warps instead of a warp per expert over all of them
     const size_t smem = (size_t)32 * experts * sizeof(int);
     if (smem > 48 * 1024) {
       cudaError_t r = cudaFuncSetAttribute(moe_group_chunked_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
       if (r != cudaSuccess) return r;
     }
-    return launch_k(moe_group_chunked_kernel, dim3(1), dim3(1024), smem, st, top_idx, n_assign, top, experts, grp_off, perm_row, slot_of);
+    return launch_k(moe_group_chunked_kernel, dim3(1), dim3(1024), smem, st, top_idx, n_assign, top, experts, grp_off, perm_row, slot_of,
+                    top_w, perm_w);
   }
   int threads = 32 * experts;
   threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
@@ -225,7 +232,7 @@ cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int expe
     if (r != cudaSuccess) return r;
   }
   return launch_k(moe_group_kernel, dim3(1), dim3(threads), in_smem ? bytes : 0, st, top_idx, n_assign, top, experts, grp_off, perm_row, slot_of,
-                  in_smem);
+                  top_w, perm_w, in_smem);
 }
 
 cudaError_t launch_moe_combine(const float* ye, const int* slot_of, const float* top_w, int top, const float* ys, const float* z, int ldz,

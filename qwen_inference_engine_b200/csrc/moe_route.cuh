@@ -1,7 +1,8 @@
-// moe_route.cuh -- the choice of a sigmoid router with a correction and group-limited top-k for ONE row, by one warp
-// (ditenex.h: RouteRider, the rider of the norm in front of a mixture of experts, rmsnorm_f32.cu).
+// moe_route.cuh -- the choice of a sigmoid router with a correction and group-limited top-k for ONE row, by one warp, and the rider of
+// a norm in front of a mixture of experts (RouteRider, nogatar.h) that works out the row's logits first.
 #pragma once
 #include "common.cuh"
+#include "nogatar.h"
 
 namespace qie {
 
@@ -35,7 +36,8 @@ __device__ __forceinline__ void route_sigmoid_row(const float* z, float* scratch
   for (int e = lane; e < experts; e += 32) {
     const float v = 1.0f / (1.0f + expf(-z[e]));
     s[e] = v;
-    c[e] = v + (correction ? bf2f(correction[e]) : 0.f);
+    // the choice scores; where nothing is added to a score its logit orders the experts alike, also where the sigmoid saturates
+    c[e] = correction ? v + bf2f(correction[e]) : keep < groups ? v : z[e];
   }
   __syncwarp();
   if (keep < groups) {
@@ -72,6 +74,34 @@ __device__ __forceinline__ void route_sigmoid_row(const float* z, float* scratch
     }
     __syncwarp();
   }
+}
+
+// the rider of a norm kernel (RouteRider): the CTA of row r holds the normed row h [W] in shared memory (complete) and works out the
+// router's logits, a warp per expert, lanes striding the width (16-byte weight loads when the rows allow it); warp 0 then chooses.
+// zl: experts + route_scratch_floats() floats of shared memory
+__device__ __forceinline__ void route_rider_row(const RouteRider& rt, int r, const float* h, int W, float* zl) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const bool vec = W % 8 == 0 && (reinterpret_cast<uintptr_t>(rt.w_router) & 15) == 0;
+  for (int e = warp; e < rt.experts; e += nw) {
+    const bf16* wr = rt.w_router + (size_t)e * W;
+    float acc = 0.f;
+    if (vec) {
+      for (int i = lane * 8; i < W; i += 256) {
+        const uint4 p = *reinterpret_cast<const uint4*>(wr + i);
+        const float* x = h + i;
+        acc = fmaf(x[0], lo2f(p.x), acc), acc = fmaf(x[1], hi2f(p.x), acc), acc = fmaf(x[2], lo2f(p.y), acc), acc = fmaf(x[3], hi2f(p.y), acc);
+        acc = fmaf(x[4], lo2f(p.z), acc), acc = fmaf(x[5], hi2f(p.z), acc), acc = fmaf(x[6], lo2f(p.w), acc), acc = fmaf(x[7], hi2f(p.w), acc);
+      }
+    } else {
+      for (int i = lane; i < W; i += 32) acc = fmaf(h[i], bf2f(wr[i]), acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) zl[e] = acc;
+  }
+  __syncthreads();
+  if (warp == 0)
+    route_sigmoid_row(zl, zl + rt.experts, rt.experts, rt.top, rt.groups, rt.keep, rt.correction, rt.scale, rt.top_idx + (size_t)r * rt.top,
+                      rt.top_w + (size_t)r * rt.top, lane);
 }
 
 }  // namespace qie

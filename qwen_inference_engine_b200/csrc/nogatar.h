@@ -50,7 +50,7 @@ cudaError_t launch_embed_scale_f32(float* x, const bf16* table, const int* ids, 
 // out[r, :] = (res ? res[r, :] : 0) + mult * LN(y[src(r), :]) * w, LN = (y - mean) / sqrt(mean((y - mean)^2) + eps);
 // src(r) = gather ? gather[r] : r.  out may alias res.
 // With `mix` (y == nullptr) the normed vector is the mixture-of-experts combine of row r, computed on the fly:
-// sum_k top_w[r,k] * ye[slot_of[r,k]] (+ sigmoid(z[r, gate_col]) * ys[r]).
+// sum_k top_w[r,k] * ye[slot_of[r,k]] (+ sigmoid(z[r, gate_col]) * ys[r]); top_w null: every weight is 1 (it scaled the experts' inputs).
 struct MoeMix {
   const float* ye = nullptr;
   const int* slot_of = nullptr;
@@ -62,8 +62,8 @@ struct MoeMix {
 };
 cudaError_t launch_layernorm_f32(const float* y, const bf16* w, float* out, const float* res, const int* gather, int width, int n,
                                  float eps, float mult, cudaStream_t st, const MoeMix& mix = MoeMix());
-// z = cap * tanh(z / cap) in place
-cudaError_t launch_softcap_f32(float* z, size_t n, float cap, cudaStream_t st);
+// z *= scale, then (cap > 0) z = cap * tanh(z / cap), in place
+cudaError_t launch_softcap_f32(float* z, size_t n, float cap, cudaStream_t st, float scale = 1.0f);
 cudaError_t launch_cast_f32_bf16(const float* in, bf16* out, size_t n, cudaStream_t st);
 // operand / result conversion around a bf16 tensor-core GEMM: strided fp32 rows (optionally gathered) <-> dense bf16 rows
 cudaError_t launch_rows_f32_to_bf16(const float* in, int ld_in, const int* row_idx, bf16* out, int cols, int n, cudaStream_t st);
@@ -150,15 +150,30 @@ cudaError_t launch_mlstm_scan(const MlstmArgs& a, cudaStream_t st);
 // route: scores = softmax(z[r, 0:experts]); the `top` largest (lowest index first among equals) with weights
 // score / (sum of the chosen + 1e-20).  group: rows sorted by expert: grp_off[experts + 1], perm_row[n*top] (source
 // row of each slot), slot_of[n*top] (slot of assignment (r, k)).  combine: y[r] = sum_k w[r,k] * ye[slot_of[r,k]]
-// (+ sigmoid(z[r, gate_col]) * ys[r] with a shared expert).
+// (+ sigmoid(z[r, gate_col]) * ys[r] with a shared expert).  group with top_w: perm_w[slot] = the weight of the slot's assignment.
+// Rider of a norm in front of a mixture of experts: the row's router logits z_e = w_router[e, :] . h (fp32, from the
+// normed row while it is in shared memory) and the choice (moe_route.cuh), by the same CTA:
+// s = sigmoid(z); choice score c = s + correction.  The experts form `groups` equal runs of neighbours; a group's score is
+// the sum of its two largest c; only experts of the `keep` best groups can be chosen; the `top` largest c among them
+// (lowest index first among equals) are chosen with weights s * scale (not renormalised).
+struct RouteRider {
+  const bf16* w_router = nullptr;  // [experts, width]; null: no rider
+  const bf16* correction = nullptr;
+  int experts = 0, top = 0, groups = 1, keep = 1;
+  float scale = 1.f;
+  int* top_idx = nullptr;  // [n, top]
+  float* top_w = nullptr;
+};
 cudaError_t launch_moe_route(const float* z, int ldz, int experts, int top, int* top_idx, float* top_w, int n, cudaStream_t st);
-cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int experts, int* grp_off, int* perm_row, int* slot_of, cudaStream_t st);
+cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int experts, int* grp_off, int* perm_row, int* slot_of, cudaStream_t st,
+                             const float* top_w = nullptr, float* perm_w = nullptr);
 cudaError_t launch_moe_combine(const float* ye, const int* slot_of, const float* top_w, int top, const float* ys, const float* z, int ldz,
                                int gate_col, float* y, int width, int n, cudaStream_t st);
 
 // Expert GEMMs on tensor cores over bf16 rows (gemm_grouped.cu): C[row, :] = A[src(row), :] W_z^T for the rows
 // grp_off[z] .. grp_off[z + 1] - 1 of expert z, src(row) = row_idx ? row_idx[row] : row; W_z = W + z * w_batch, [N, K] row-major.
-// gated: W_z = [gate rows | up rows] (N = 2 ff) and out_bf[row, c] = bf16(silu(gate_c) * up_c), c < ff; else out[row, n] fp32.
+// gated: W_z = [gate rows | up rows] (N = 2 ff) and out_bf[row, c] = bf16(silu(gate_c) * up_c), c < ff; else out[row, n] fp32 or out_bf.
+// row_w (per row of the groups): the input row is scaled by it, which both linear maps let through: gate and up (or the result) times row_w.
 struct GroupedGemmBf16 {
   const bf16* A = nullptr;
   int lda = 0;
@@ -167,6 +182,7 @@ struct GroupedGemmBf16 {
   const bf16* W = nullptr;
   long w_batch = 0;
   int N = 0, K = 0, groups = 0;
+  const float* row_w = nullptr;
   int rows = 0;  // rows over all groups (bounds the grid)
   int gated = 0;
   float* out = nullptr;

@@ -453,11 +453,13 @@ __global__ void gemv_trans_f32_kernel(const GemmF32 g) {
   g.C[(size_t)z * g.c_batch + (size_t)m * g.ldc + n] = acc;
 }
 
-__global__ void softcap_kernel(float* z, size_t n, float cap) {
+__global__ void softcap_kernel(float* z, size_t n, float cap, float scale) {
   pdl_wait();
   pdl_trigger();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) z[i] = cap * tanhf(z[i] / cap);
+  if (i >= n) return;
+  const float v = z[i] * scale;
+  z[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
 }
 
 __global__ void cast_f32_bf16_kernel(const float* in, bf16* out, size_t n) {
@@ -613,9 +615,9 @@ cudaError_t launch_layernorm_f32(const float* y, const bf16* w, float* out, cons
   return launch_k(layernorm_f32_kernel, dim3(n), dim3(256), smem, st, y, w, out, res, gather, width, eps, mult, mix);
 }
 
-cudaError_t launch_softcap_f32(float* z, size_t n, float cap, cudaStream_t st) {
+cudaError_t launch_softcap_f32(float* z, size_t n, float cap, cudaStream_t st, float scale) {
   if (n == 0) return cudaSuccess;
-  return launch_k(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, z, n, cap);
+  return launch_k(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, z, n, cap, scale);
 }
 
 cudaError_t launch_cast_f32_bf16(const float* in, bf16* out, size_t n, cudaStream_t st) {

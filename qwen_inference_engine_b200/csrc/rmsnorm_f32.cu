@@ -2,7 +2,8 @@
 // into the residual add together with the next sublayer's input norm, and the input norm of a mixer that reads a blend
 // of each row with the row before it (token shift) with one carried row per sequence slot; and the grouped RMS norm of a
 // model of parallel blocks (dedunex.h): the residual add of the two sublayer outputs and the next block's norm in one kernel;
-// and the grouped norm with a gate behind it (gebadra.h).
+// and the grouped norm with a gate behind it (gebadra.h).  A model with one group and a router in front of its experts (gubanex.h) uses
+// the grouped step with the router's rider.
 // All fp32, one CTA per row, every reduction in a fixed order per row, so a row's result does not depend on the rows it
 // shares a launch with.
 #include "dedunex.h"
@@ -92,32 +93,8 @@ __global__ void __launch_bounds__(256) rms_step_kernel(const RmsStep a) {
     st_f32<V>(row + i, o);
   }
   if (!a.route.w_router) return;
-  // router logits of the row: a warp per expert, lanes stride the width (16-byte weight loads when the rows allow it)
-  const RouteRider& rt = a.route;
-  float* zl = row + W;  // [experts] logits, then the router's scratch
-  __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const bool vec = W % 8 == 0 && (reinterpret_cast<uintptr_t>(rt.w_router) & 15) == 0;
-  for (int e = warp; e < rt.experts; e += nw) {
-    const bf16* wr = rt.w_router + (size_t)e * W;
-    float acc = 0.f;
-    if (vec) {
-      for (int i = lane * 8; i < W; i += 256) {
-        const uint4 p = *reinterpret_cast<const uint4*>(wr + i);
-        const float* h = row + i;
-        acc = fmaf(h[0], lo2f(p.x), acc), acc = fmaf(h[1], hi2f(p.x), acc), acc = fmaf(h[2], lo2f(p.y), acc), acc = fmaf(h[3], hi2f(p.y), acc);
-        acc = fmaf(h[4], lo2f(p.z), acc), acc = fmaf(h[5], hi2f(p.z), acc), acc = fmaf(h[6], lo2f(p.w), acc), acc = fmaf(h[7], hi2f(p.w), acc);
-      }
-    } else {
-      for (int i = lane; i < W; i += 32) acc = fmaf(row[i], bf2f(wr[i]), acc);
-    }
-    acc = warp_sum(acc);
-    if (lane == 0) zl[e] = acc;
-  }
-  __syncthreads();
-  if (warp == 0)
-    route_sigmoid_row(zl, zl + rt.experts, rt.experts, rt.top, rt.groups, rt.keep, rt.correction, rt.scale, rt.top_idx + (size_t)r * rt.top,
-                      rt.top_w + (size_t)r * rt.top, lane);
+  __syncthreads();  // the normed row is complete
+  route_rider_row(a.route, r, row, W, row + W);
 }
 
 // one CTA per row.  The CTA of a segment's first row also moves the segment's last normed row into the carried row:
@@ -196,9 +173,10 @@ __device__ __forceinline__ void group_rstd(const float* row, int W, int groups, 
   __syncthreads();
 }
 
-template <int V>
+// NR > 0: one group, the row stays in NR packs of registers per thread; NR = 0: any number of groups, the row in shared memory
+template <int V, int NR>
 __global__ void __launch_bounds__(256) group_norm_step_kernel(const GroupNormStep a) {
-  extern __shared__ __align__(16) float row[];  // [width], then [groups] scales
+  extern __shared__ __align__(16) float row[];  // [width], then [groups] scales, then the router's logits and scratch
   __shared__ float red[32];
   pdl_wait();
   pdl_trigger();
@@ -207,71 +185,104 @@ __global__ void __launch_bounds__(256) group_norm_step_kernel(const GroupNormSte
   const int t0 = threadIdx.x * V, step = blockDim.x * V;
   const int src = a.gather ? a.gather[r] : r;
   float* xr = a.x + (size_t)src * W;
-  bool changed = false;
-  if (a.ids) {  // the embedding row, normed
-    const bf16* er = a.embed + (size_t)a.ids[r] * W;
-    for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_bf16<V>(er + i));
+  const bf16* entry = a.ids ? a.embed + (size_t)a.ids[src] * W : nullptr;
+  const bool fresh = a.ids && !a.again, normed = fresh && a.w_pre;
+  const bool has1 = a.y1 || a.y1_bf, has2 = a.y2 || a.y2_bf, mixed = a.mix.ye || a.ye_bf;
+  const bool changed = a.ids || has1 || has2 || mixed || a.step;
+  if (normed) {  // the embedding row, normed
+    for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_bf16<V>(entry + i));
     __syncthreads();
     group_rstd(row, W, a.groups, a.eps, red, scale);
-    for (int i = t0; i < W; i += step) {
-      Pack<V> v = ld_f32<V>(row + i);
+  }
+  auto entry_at = [&](int i) {
+    Pack<V> v = ld_bf16<V>(entry + i);
+#pragma unroll
+    for (int u = 0; u < V; ++u) v.v[u] *= a.embed_scale;
+    return v;
+  };
+  // elements i .. i + V - 1 of the stream after every addition; a thread touches only its own elements of the row
+  auto value = [&](int i) {
+    Pack<V> v;
+    if (normed) {
+      v = ld_f32<V>(row + i);
       const Pack<V> w = ld_bf16<V>(a.w_pre + i);
 #pragma unroll
       for (int u = 0; u < V; ++u) v.v[u] = v.v[u] * scale[(i + u) / gs] * w.v[u];
-      st_f32<V>(row + i, v);
+    } else {
+      v = fresh ? entry_at(i) : ld_f32<V>(xr + i);
     }
-    changed = true;
-  } else {
-    for (int i = t0; i < W; i += step) st_f32<V>(row + i, ld_f32<V>(xr + i));
-  }
-  // every thread touches only its own elements of the row until the norm below
-  if (a.y1 || a.y1_bf || a.y2 || a.y2_bf) {
-    for (int i = t0; i < W; i += step) {
-      Pack<V> v = ld_f32<V>(row + i);
-      if (a.y1 || a.y1_bf) {
-        const Pack<V> y = a.y1_bf ? ld_bf16<V>(a.y1_bf + (size_t)src * W + i) : ld_f32<V>(a.y1 + (size_t)src * W + i);
-        if (a.y2 || a.y2_bf) {
-          const Pack<V> z = a.y2_bf ? ld_bf16<V>(a.y2_bf + (size_t)src * W + i) : ld_f32<V>(a.y2 + (size_t)src * W + i);
+    if (has1 || has2) {
+      Pack<V> y, z;
+      if (has1) y = a.y1_bf ? ld_bf16<V>(a.y1_bf + (size_t)src * W + i) : ld_f32<V>(a.y1 + (size_t)src * W + i);
+      if (has2) z = a.y2_bf ? ld_bf16<V>(a.y2_bf + (size_t)src * W + i) : ld_f32<V>(a.y2 + (size_t)src * W + i);
 #pragma unroll
-          for (int u = 0; u < V; ++u) v.v[u] += y.v[u] + z.v[u];
-        } else {
+      for (int u = 0; u < V; ++u) v.v[u] += has1 && has2 ? y.v[u] + z.v[u] : has1 ? y.v[u] : z.v[u];
+    }
+    if (mixed) {
+      Pack<V> s;
 #pragma unroll
-          for (int u = 0; u < V; ++u) v.v[u] += y.v[u];
-        }
-      } else {
-        const Pack<V> z = a.y2_bf ? ld_bf16<V>(a.y2_bf + (size_t)src * W + i) : ld_f32<V>(a.y2 + (size_t)src * W + i);
+      for (int u = 0; u < V; ++u) s.v[u] = 0.f;
+      for (int k = 0; k < a.mix.top; ++k) {
+        const size_t at = (size_t)src * a.mix.top + k, o = (size_t)a.mix.slot_of[at] * W + i;
+        const float wk = a.mix.top_w ? a.mix.top_w[at] : 1.0f;
+        const Pack<V> e = a.ye_bf ? ld_bf16<V>(a.ye_bf + o) : ld_f32<V>(a.mix.ye + o);
 #pragma unroll
-        for (int u = 0; u < V; ++u) v.v[u] += z.v[u];
+        for (int u = 0; u < V; ++u) s.v[u] = fmaf(wk, e.v[u], s.v[u]);
       }
-      st_f32<V>(row + i, v);
+#pragma unroll
+      for (int u = 0; u < V; ++u) v.v[u] += s.v[u];
     }
-    changed = true;
-  }
-  if (a.dump)
-    for (int i = t0; i < W; i += step) st_f32<V>(a.dump + (size_t)r * W + i, ld_f32<V>(row + i));
-  if (a.step) {
-    for (int i = t0; i < W; i += step) {
-      Pack<V> v = ld_f32<V>(row + i);
+    if (a.dump) st_f32<V>(a.dump + (size_t)r * W + i, v);
+    if (a.step) {
       const Pack<V> s = ld_bf16<V>(a.step + i);
 #pragma unroll
       for (int u = 0; u < V; ++u) v.v[u] += s.v[u];
-      st_f32<V>(row + i, v);
     }
-    changed = true;
-  }
-  if (changed)
-    for (int i = t0; i < W; i += step) st_f32<V>(xr + i, ld_f32<V>(row + i));
-  if (!a.h && !a.h_bf) return;
-  __syncthreads();
-  group_rstd(row, W, a.groups, a.eps, red, scale);
-  for (int i = t0; i < W; i += step) {
-    const Pack<V> x = ld_f32<V>(row + i), w = ld_bf16<V>(a.w_in + i);
+    if (a.again) {
+      const Pack<V> s = entry_at(i);
+#pragma unroll
+      for (int u = 0; u < V; ++u) v.v[u] += s.v[u];
+    }
+    if (changed) st_f32<V>(xr + i, v);
+    return v;
+  };
+  const bool read = a.h || a.h_bf;
+  auto emit = [&](int i, const Pack<V>& x, const Pack<V>& w, float s0) {
     Pack<V> o;
 #pragma unroll
-    for (int u = 0; u < V; ++u) o.v[u] = x.v[u] * scale[(i + u) / gs] * w.v[u];
+    for (int u = 0; u < V; ++u) o.v[u] = x.v[u] * (NR > 0 ? s0 : scale[(i + u) / gs]) * (a.w_off + w.v[u]);
     if (a.h) st_f32<V>(a.h + (size_t)r * W + i, o);
     if (a.h_bf) st_bf16<V>(a.h_bf + (size_t)r * W + i, o);
+    if (a.route.w_router) st_f32<V>(row + i, o);
+  };
+  if (!read) {
+    for (int i = t0; i < W; i += step) value(i);
+    return;
   }
+  if constexpr (NR > 0) {
+    Pack<V> x[NR], w[NR];
+    float sq = 0.f;
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W) x[k] = value(t0 + k * step), w[k] = ld_bf16<V>(a.w_in + t0 + k * step);
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W)
+#pragma unroll
+        for (int u = 0; u < V; ++u) sq = fmaf(x[k].v[u], x[k].v[u], sq);
+    const float s0 = 1.0f / sqrtf(block_sum_r(sq, red) / (float)W + a.eps);
+#pragma unroll
+    for (int k = 0; k < NR; ++k)
+      if (t0 + k * step < W) emit(t0 + k * step, x[k], w[k], s0);
+  } else {
+    for (int i = t0; i < W; i += step) st_f32<V>(row + i, value(i));
+    __syncthreads();
+    group_rstd(row, W, a.groups, a.eps, red, scale);
+    for (int i = t0; i < W; i += step) emit(i, ld_f32<V>(row + i), ld_bf16<V>(a.w_in + i), 0.f);
+  }
+  if (!a.route.w_router) return;
+  __syncthreads();  // the normed row is complete
+  route_rider_row(a.route, r, row, W, scale + a.groups);
 }
 
 template <int V>
@@ -286,7 +297,7 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const NormGate a) {
   auto gate_of = [&](int i) { return a.g_bf ? ld_bf16<V>(a.g_bf + r * a.ldg_bf + i) : ld_f32<V>(a.g + r * a.ldg + i); };
   auto finish = [&](int i, Pack<V> x, const Pack<V>& g, float s0) {
     Pack<V> w;
-    if (a.w) w = ld_bf16<V>(a.w + i);
+    if (a.w) w = ld_bf16<V>(a.w + (a.w_shared ? i % gs : i));
 #pragma unroll
     for (int u = 0; u < V; ++u) {
       const float sg = 1.0f / (1.0f + expf(-g.v[u]));
@@ -328,7 +339,7 @@ cudaError_t launch_norm_gate(const NormGate& a, cudaStream_t st) {
   if (a.width <= 0 || a.groups <= 0 || a.width % a.groups || !a.v || !(a.g || a.g_bf) || !(a.out || a.out_bf)) return cudaErrorInvalidValue;
   const size_t smem = ((size_t)a.width + a.groups) * sizeof(float);
   auto al = [](const void* p, size_t b) { return (reinterpret_cast<uintptr_t>(p) & (b - 1)) == 0; };
-  const bool vec = a.width % 4 == 0 && a.ldv % 4 == 0 && a.ldg % 4 == 0 && a.ldg_bf % 4 == 0 && a.ldo % 4 == 0 && a.ldo_bf % 4 == 0 && al(a.v, 16) &&
+  const bool vec = a.width % 4 == 0 && (!a.w_shared || a.width / a.groups % 4 == 0) && a.ldv % 4 == 0 && a.ldg % 4 == 0 && a.ldg_bf % 4 == 0 && a.ldo % 4 == 0 && a.ldo_bf % 4 == 0 && al(a.v, 16) &&
                    al(a.g, 16) && al(a.g_bf, 8) && al(a.w, 8) && al(a.out, 16) && al(a.out_bf, 8);
   auto* kern = vec ? norm_gate_kernel<4> : norm_gate_kernel<1>;
   if (smem > 48 * 1024) {
@@ -339,15 +350,26 @@ cudaError_t launch_norm_gate(const NormGate& a, cudaStream_t st) {
   return launch_k(kern, dim3(a.n), dim3(256), smem, st, a);
 }
 
+static bool route_ok(const RouteRider& rt) {
+  return rt.experts > 0 && rt.top > 0 && rt.top <= rt.experts && rt.groups > 0 && rt.experts % rt.groups == 0 && rt.keep > 0 && rt.keep <= rt.groups && rt.top_idx &&
+         rt.top_w;
+}
+
 cudaError_t launch_group_norm_step(const GroupNormStep& a, cudaStream_t st) {
   if (a.n <= 0) return cudaSuccess;
   const bool read = a.h || a.h_bf;
-  if (a.width <= 0 || a.groups <= 0 || a.width % a.groups || (read && !a.w_in) || (a.ids && (!a.embed || !a.w_pre || a.gather))) return cudaErrorInvalidValue;
-  const size_t smem = ((size_t)a.width + a.groups) * sizeof(float);
+  if (a.width <= 0 || a.groups <= 0 || a.width % a.groups || (read && !a.w_in) || (a.ids && (!a.embed || a.gather)) || (a.again && (!a.ids || a.w_pre))) return cudaErrorInvalidValue;
+  size_t smem = ((size_t)a.width + a.groups) * sizeof(float);
+  if (a.route.w_router) {
+    if (!read || a.gather || !route_ok(a.route)) return cudaErrorInvalidValue;
+    smem += ((size_t)a.route.experts + route_scratch_floats(a.route.experts, a.route.groups)) * sizeof(float);
+  }
   auto al = [](const void* p, size_t b) { return (reinterpret_cast<uintptr_t>(p) & (b - 1)) == 0; };
-  const bool vec = a.width % 4 == 0 && al(a.x, 16) && al(a.y1, 16) && al(a.y2, 16) && al(a.y1_bf, 8) && al(a.y2_bf, 8) && al(a.dump, 16) && al(a.h, 16) &&
-                   al(a.h_bf, 8) && al(a.w_in, 8) && al(a.w_pre, 8) && al(a.step, 8) && al(a.embed, 8);
-  auto* kern = vec ? group_norm_step_kernel<4> : group_norm_step_kernel<1>;
+  const bool vec = a.width % 4 == 0 && al(a.x, 16) && al(a.y1, 16) && al(a.y2, 16) && al(a.y1_bf, 8) && al(a.y2_bf, 8) && al(a.mix.ye, 16) && al(a.ye_bf, 8) &&
+                   al(a.dump, 16) && al(a.h, 16) && al(a.h_bf, 8) && al(a.w_in, 8) && al(a.w_pre, 8) && al(a.step, 8) && al(a.embed, 8);
+  const bool regs = vec && a.groups == 1 && !(a.ids && a.w_pre);
+  auto* kern = !vec ? group_norm_step_kernel<1, 0> : !regs ? group_norm_step_kernel<4, 0> : a.width <= 1024 ? group_norm_step_kernel<4, 1>
+               : a.width <= 2048 ? group_norm_step_kernel<4, 2> : a.width <= 4096 ? group_norm_step_kernel<4, 4> : group_norm_step_kernel<4, 0>;
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return cudaErrorInvalidValue;
     cudaError_t r = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -363,9 +385,7 @@ cudaError_t launch_rms_step(const RmsStep& a, cudaStream_t st) {
   size_t smem = (size_t)a.width * sizeof(float);
   if (a.route.w_router) {
     const RouteRider& rt = a.route;
-    if (!read || a.gather || rt.experts <= 0 || rt.top <= 0 || rt.top > rt.experts || rt.groups <= 0 || rt.experts % rt.groups || rt.keep <= 0 ||
-        rt.keep > rt.groups || !rt.top_idx || !rt.top_w)
-      return cudaErrorInvalidValue;
+    if (!read || a.gather || !route_ok(rt)) return cudaErrorInvalidValue;
     smem += ((size_t)rt.experts + route_scratch_floats(rt.experts, rt.groups)) * sizeof(float);
   }
   // 16-byte accesses when every row starts on a 16-byte boundary (cudaMalloc'd buffers, width a multiple of 4)
