@@ -552,6 +552,34 @@ def gebadra_macs_per_token(cfg):
     return mac
 
 
+def gubanex_config(z, vocab=32000):
+    """two layers, four layer runs (a loop of two passes): chunked attention on four kv heads with unit-normed queries and keys, gated
+    linear attention; mixtures of experts whose chosen experts have the width of the compared Qwen model's feed-forward"""
+    W = z["width"]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] + z["sff"] // z["top"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    att = {"dim": 64, "heads": W // 64, "kv_heads": 4, "mask": {"size": z["window"]}, "scale": 0.125, "vdim": 64,
+           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 2048}}}
+    lin = {"dim": 64, "heads": W // 128, "rank": 16, "tau": 16.0, "vdim": 128}
+    layers = [{"type": "attention", "mixer": att, "mlp": moe}, {"type": "gla", "mixer": lin, "mlp": moe}]
+    return {"architecture": "Gubanex", "embedding": {"scale": W ** 0.5}, "layers": layers, "logit_scale": 0.25, "logit_softcap": 30.0,
+            "loop": {"start": 0, "stop": 2, "times": 2}, "norm": {"eps": 1e-6}, "vocab": vocab, "width": W}
+
+
+def gubanex_macs_per_token(cfg):
+    """multiply-adds of the projections of one token over all layer runs (attention scores and the recurrence not counted)"""
+    W, mac, lp = cfg["width"], 0, cfg["loop"]
+    for i, ly in enumerate(cfg["layers"]):
+        mx, mlp = ly["mixer"], ly["mlp"]
+        H, d, vd = mx["heads"], mx["dim"], mx["vdim"]
+        if ly["type"] == "attention":
+            one = W * (H * d + mx["kv_heads"] * (d + vd) + H * vd)
+        else:
+            one = W * (H * (2 * d + 3 * vd) + mx["rank"]) + mx["rank"] * H * d
+        one += 3 * W * mlp["router"]["top"] * mlp["expert"]["ff"] + W * mlp["router"]["experts"]
+        mac += one * (lp["times"] if lp["start"] <= i < lp["stop"] else 1)
+    return mac
+
+
 def run_family_compare(args):
     import numpy as np
     import torch
@@ -642,12 +670,17 @@ def run_family_compare(args):
             dd_cfg = json.dumps(dd)
             rec["dedunex"] = measure(lambda rows, seqs: q.Engine(config_json=dd_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
                                                                  max_seqs=seqs, max_batch_tokens=rows, context=8192), vocab, False)
-        if args.family == "gebadra":
+        if args.family == "gubanex":
+            gx = gubanex_config(z, vocab)
+            gx_cfg = json.dumps(gx)
+            rec["gubanex"] = measure(lambda rows, seqs: q.Engine(config_json=gx_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
+                                                                 max_seqs=seqs, max_batch_tokens=rows, context=8192), vocab, False)
+        if args.family in ("gebadra", "gubanex"):
             gb = gebadra_config(z, vocab)
             gb_cfg = json.dumps(gb)
             rec["gebadra"] = measure(lambda rows, seqs: q.Engine(config_json=gb_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
                                                                  max_seqs=seqs, max_batch_tokens=rows, context=8192), vocab, False)
-        if args.family == "ditenex":
+        if args.family in ("ditenex", "gubanex"):
             dx = ditenex_config(z, vocab)
             dx_cfg = json.dumps(dx)
             rec["ditenex"] = measure(lambda rows, seqs: q.Engine(config_json=dx_cfg, seed=7, dtype="bfloat16", page_size=16, max_pages=pages,
@@ -669,13 +702,16 @@ def run_family_compare(args):
         if args.family == "dedunex":
             rec["macs_per_token"]["dedunex"] = dedunex_macs_per_token(dd)
             fams.append(("dedunex", rec["macs_per_token"]["dedunex"]))
-        if args.family == "gebadra":
+        if args.family == "gubanex":
+            rec["macs_per_token"]["gubanex"] = gubanex_macs_per_token(gx)
+            fams.append(("gubanex", rec["macs_per_token"]["gubanex"]))
+        if args.family in ("gebadra", "gubanex"):
             rec["macs_per_token"]["gebadra"] = gebadra_macs_per_token(gb)
             fams.append(("gebadra", rec["macs_per_token"]["gebadra"]))
         if args.family in ("fosavik", "dedunex", "gebadra"):
             rec["macs_per_token"]["fosavik"] = fosavik_macs_per_token(fv)
             fams.append(("fosavik", rec["macs_per_token"]["fosavik"]))
-        if args.family == "ditenex":
+        if args.family in ("ditenex", "gubanex"):
             rec["macs_per_token"]["ditenex"] = ditenex_macs_per_token(dx)
             fams.append(("ditenex", rec["macs_per_token"]["ditenex"]))
         for fam, mac in fams:
@@ -704,9 +740,10 @@ def main():
     ap.add_argument("--family-compare", action="store_true",
                     help="side measurement (not the contract line): prefill / decode throughput of the Nogatar family beside the "
                          "Qwen family at equal size, with per-kernel-class device times")
-    ap.add_argument("--family", default="nogatar", choices=["nogatar", "fosavik", "ditenex", "dedunex", "gebadra"],
+    ap.add_argument("--family", default="nogatar", choices=["nogatar", "fosavik", "ditenex", "dedunex", "gebadra", "gubanex"],
                     help="with --family-compare: which fp32-stream family is measured beside the Qwen family (fosavik and ditenex also run "
-                         "nogatar; dedunex and gebadra also run fosavik, the family whose mixers are closest to their own)")
+                         "nogatar; dedunex and gebadra also run fosavik, the family whose mixers are closest to their own; gubanex also runs "
+                         "gebadra and ditenex)")
     ap.add_argument("--family-size", default="", help="one of " + ", ".join(FAMILY_SIZES) + " (default: all)")
     ap.add_argument("--family-tokens", type=int, default=2048)
     ap.add_argument("--family-ctx", type=int, default=1024)
