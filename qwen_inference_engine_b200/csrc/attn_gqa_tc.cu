@@ -137,6 +137,18 @@ __device__ __forceinline__ void copy_row(const bf16* row, size_t koff, size_t vo
   }
 }
 
+// Tiles of a segment in ascending order of how deep in its chunk a tile lies, which is how many keys it sees: number i of nt.  m tiles make
+// about one chunk; a tile's depth is its number modulo m, counted from where the segment's first row (position p0) lies in its chunk.
+__device__ __forceinline__ int by_work(int i, int nt, int p0, int chunk) {
+  const int m = min((chunk + TQ - 1) / TQ, nt), off = p0 % chunk / TQ % m;
+  for (int r = 0; r < m; ++r) {
+    const int first = (r - off + m) % m, count = first < nt ? (nt - first + m - 1) / m : 0;
+    if (i < count) return first + i * m;
+    i -= count;
+  }
+  return 0;  // not reached: the counts add up to nt
+}
+
 __global__ void __launch_bounds__(NTHR, 1) gqa_tc_kernel(const GqaAttnArgs a, int dblk, int vblk, int nst, int vc,
                                                                const __grid_constant__ CUtensorMap rows_map, int use_tma) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -149,7 +161,10 @@ __global__ void __launch_bounds__(NTHR, 1) gqa_tc_kernel(const GqaAttnArgs a, in
     int left = gridDim.y - 1 - blockIdx.y, found = 0;  // late tiles of a segment see more keys: they start first
     for (int s = 0; s < a.n_seg && !found; ++s) {
       const int r0 = a.seg_start[s], len = a.seg_start[s + 1] - r0, nt = (len + TQ - 1) / TQ;
-      if (left < nt) info[0] = r0 + left * TQ, info[1] = min(TQ, len - left * TQ), info[2] = a.seg_slot[s], found = 1;
+      if (left >= 0 && left < nt) {
+        const int t = a.chunk > 0 ? by_work(left, nt, a.pos[r0], a.chunk) : left;
+        info[0] = r0 + t * TQ, info[1] = min(TQ, len - t * TQ), info[2] = a.seg_slot[s], found = 1;
+      }
       left -= nt;
     }
     if (!found) info[1] = 0;

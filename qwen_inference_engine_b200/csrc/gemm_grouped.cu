@@ -6,6 +6,8 @@
 // rows interleaved in runs of 16 with the 64 up rows of the same columns, so that a thread holds silu's argument and
 // its factor side by side and writes silu(gate) * up as bf16 -- the [gate | up] rows never go to memory.
 // k ascends per output whatever the tile, so a row's result does not depend on the rows around it.
+#include <algorithm>
+
 #include "launch.h"
 #include "nogatar.h"
 
@@ -21,13 +23,32 @@ __global__ void __launch_bounds__(256) grouped_gemm_bf16_kernel(const GroupedGem
   Tile* Bs = reinterpret_cast<Tile*>(gg_smem + STAGES * sizeof(Tile));
   __shared__ int a_row[BM];  // source row of each tile row (clamped to a valid one: rows past the group are computed and dropped)
   __shared__ int b_row[BN];  // weight row of each tile column
+  __shared__ int tile_at[2];  // group and first row of the CTA's row tile (group -1: there is no such tile)
   pdl_wait();
   pdl_trigger();
-  const int z = blockIdx.z;
-  const int row_base = g.grp_off[z], Mz = g.grp_off[z + 1] - row_base;
-  const int m0 = blockIdx.y * BM;
-  if (m0 >= Mz) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (warp == 0) {  // row tile number blockIdx.y of all groups: 32 groups at a time, a scan over their tile counts
+    int left = blockIdx.y, found = -1, m = 0;
+    for (int z0 = 0; z0 < g.groups && found < 0; z0 += 32) {
+      const int zz = z0 + lane, cnt = zz < g.groups ? (g.grp_off[zz + 1] - g.grp_off[zz] + BM - 1) / BM : 0;
+      int inc = cnt;
+      for (int o = 1; o < 32; o <<= 1) {
+        const int t = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= o) inc += t;
+      }
+      const unsigned hit = __ballot_sync(0xffffffffu, left < inc);
+      if (hit) {
+        const int l = __ffs(hit) - 1;
+        found = z0 + l, m = left - __shfl_sync(0xffffffffu, inc - cnt, l);
+      }
+      left -= __shfl_sync(0xffffffffu, inc, 31);
+    }
+    if (lane == 0) tile_at[0] = found, tile_at[1] = m * BM;
+  }
+  __syncthreads();
+  const int z = tile_at[0], m0 = tile_at[1];
+  if (z < 0) return;
+  const int row_base = g.grp_off[z], Mz = g.grp_off[z + 1] - row_base;
   const int n_out = g.gated ? g.N / 2 : g.N;                      // output columns
   const int c0 = blockIdx.x * (g.gated ? BN / 2 : BN);            // first output column of the tile
   if (tid < BM) {
@@ -152,7 +173,7 @@ cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st) 
     set.done();
   }
   const int n_out = g.gated ? g.N / 2 : g.N, per = g.gated ? BN / 2 : BN;
-  const dim3 grid((n_out + per - 1) / per, (g.rows + BM - 1) / BM, g.groups);  // rows: the upper bound of any group; empty tiles leave at once
+  const dim3 grid((n_out + per - 1) / per, g.rows / BM + std::min(g.rows, g.groups));  // row tiles of all groups: an upper bound, empty ones leave at once
   return launch_k(grouped_gemm_bf16_kernel, grid, dim3(256), smem, st, g);
 }
 

@@ -503,22 +503,24 @@ __global__ void __launch_bounds__(LT) linear_chunk_out_kernel(const LinearAttnAr
 }
 
 // ---------------------------------------------------------------- gated channels
-// CTA (chunk, 128 channels): log2 of the decays of the chunk's rows, summed up row by row -> cum [n, heads, pitch].  A thread walks the
-// rows of one channel; RMAX: the low-rank map's row in registers (0: any rank, from memory)
+// CTA (chunk, 64 channels): log2 of the decays of the chunk's rows, summed up row by row -> cum [n, heads, pitch].  A thread walks a block of
+// 16 rows of one channel, the blocks' sums meet in shared memory; RMAX: the low-rank map's row in registers (0: any rank, from memory)
+constexpr int GD_CH = 64, GD_ROWS = 16, GD_PARTS = LC / GD_ROWS;
 template <int RMAX>
-__global__ void __launch_bounds__(128) gated_decay_kernel(const LinearAttnArgs a) {
+__global__ void __launch_bounds__(GD_CH * GD_PARTS) gated_decay_kernel(const LinearAttnArgs a) {
   extern __shared__ __align__(16) float gd_low[];  // [LC][RP] low-rank rows, zeros beyond the rank
+  __shared__ float sums[GD_PARTS][GD_CH];
   pdl_wait();
   pdl_trigger();
   int row0, L;
   if (!find_chunk(a, blockIdx.x, &row0, &L)) return;
   const GatedDecay& g = a.gate;
   const int rank = g.rank, RP = RMAX > 0 ? RMAX : rank, pitch = gated_decay_pitch(a.dim);
-  for (int i = threadIdx.x; i < L * RP; i += 128) {
+  for (int i = threadIdx.x; i < L * RP; i += GD_CH * GD_PARTS) {
     const int t = i / RP, j = i - t * RP;
     gd_low[i] = j >= rank ? 0.f : g.low_bf ? bf2f(g.low_bf[(size_t)(row0 + t) * a.ld_bf + j]) : g.low[(size_t)(row0 + t) * a.ld + j];
   }
-  const int at = blockIdx.y * 128 + threadIdx.x, h = at / pitch, d = at - h * pitch;
+  const int c = threadIdx.x % GD_CH, part = threadIdx.x / GD_CH, at = blockIdx.y * GD_CH + c, h = at / pitch, d = at - h * pitch;
   const bool live = h < a.heads && d < a.dim;
   const int ch = live ? h * a.dim + d : 0;
   float w[RMAX > 0 ? RMAX : 1];
@@ -528,24 +530,36 @@ __global__ void __launch_bounds__(128) gated_decay_kernel(const LinearAttnArgs a
   }
   const float bias = bf2f(g.bias[ch]);
   __syncthreads();
+  float b[GD_ROWS], sum = 0.f;  // running sums of the thread's rows
+#pragma unroll
+  for (int k = 0; k < GD_ROWS; ++k) {
+    const int t = part * GD_ROWS + k;
+    float z = bias;
+    if (t < L) {
+      const float* low = gd_low + t * RP;
+      if constexpr (RMAX > 0) {
+#pragma unroll
+        for (int j = 0; j < RMAX; j += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(low + j);
+          z = fmaf(w[j], x.x, z), z = fmaf(w[j + 1], x.y, z), z = fmaf(w[j + 2], x.z, z), z = fmaf(w[j + 3], x.w, z);
+        }
+      } else {
+        for (int j = 0; j < rank; ++j) z = fmaf(bf2f(g.a2[(size_t)ch * rank + j]), low[j], z);
+      }
+      if (live) sum += log2_sigmoid_pow(z, g.inv_tau);
+    }
+    b[k] = sum;
+  }
+  sums[part][c] = sum;
+  __syncthreads();
+  float before = 0.f;
+  for (int p = 0; p < part; ++p) before += sums[p][c];
   if (h >= a.heads) return;
   float* out = g.cum + (size_t)row0 * a.heads * pitch + at;
-  float sum = 0.f;
-#pragma unroll 4
-  for (int t = 0; t < L; ++t) {
-    float z = bias;
-    const float* low = gd_low + t * RP;
-    if constexpr (RMAX > 0) {
 #pragma unroll
-      for (int j = 0; j < RMAX; j += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(low + j);
-        z = fmaf(w[j], x.x, z), z = fmaf(w[j + 1], x.y, z), z = fmaf(w[j + 2], x.z, z), z = fmaf(w[j + 3], x.w, z);
-      }
-    } else {
-      for (int j = 0; j < rank; ++j) z = fmaf(bf2f(g.a2[(size_t)ch * rank + j]), low[j], z);
-    }
-    if (live) sum += log2_sigmoid_pow(z, g.inv_tau);
-    out[(size_t)t * a.heads * pitch] = sum;
+  for (int k = 0; k < GD_ROWS; ++k) {
+    const int t = part * GD_ROWS + k;
+    if (t < L) out[(size_t)t * a.heads * pitch] = before + b[k];
   }
 }
 
@@ -648,6 +662,7 @@ __global__ void __launch_bounds__(LT) gated_chunk_out_kernel(const LinearAttnArg
       const int i = tid + n * LT, r = i / (DP / 4), c = (i % (DP / 4)) * 4;
       b[n] = c < pitch ? *reinterpret_cast<const float4*>(cum + (size_t)min(r, L - 1) * crow + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    load_entry_state<DP, VP>(a, h, v0, Sh, Sl);  // on its way together with the tiles
     q.store(Qs, a.act);
     k.store(Ks, a.act);
     v.store(Vs, a.act);
@@ -657,7 +672,6 @@ __global__ void __launch_bounds__(LT) gated_chunk_out_kernel(const LinearAttnArg
       *reinterpret_cast<float4*>(&Bs[i / (DP / 4)][(i % (DP / 4)) * 4]) = b[n];
     }
   }
-  load_entry_state<DP, VP>(a, h, v0, Sh, Sl);
   __syncthreads();
   for (int i = tid; i < LC / 16 * DP; i += LT) {
     const int blk = i / DP, c = i - blk * DP;
@@ -822,9 +836,9 @@ cudaError_t launch_gated_chunked(const LinearAttnArgs& a, cudaStream_t st) {
     once.done();
   }
   const int rank = a.gate.rank, RP = rank <= 16 ? 16 : rank <= 32 ? 32 : rank;
-  const dim3 dgrid(chunks, (a.heads * gated_decay_pitch(a.dim) + 127) / 128);
+  const dim3 dgrid(chunks, (a.heads * gated_decay_pitch(a.dim) + GD_CH - 1) / GD_CH);
   auto* decay = rank <= 16 ? gated_decay_kernel<16> : rank <= 32 ? gated_decay_kernel<32> : gated_decay_kernel<0>;
-  if ((r = launch_k(decay, dgrid, dim3(128), (size_t)LC * RP * sizeof(float), st, a)) != cudaSuccess) return r;
+  if ((r = launch_k(decay, dgrid, dim3(GD_CH * GD_PARTS), (size_t)LC * RP * sizeof(float), st, a)) != cudaSuccess) return r;
   if ((r = launch_k(gated_chunk_state_kernel<DP, VP>, dim3(chunks, a.heads, nvb), dim3(LT), s1, st, a)) != cudaSuccess) return r;
   const int per = a.heads * a.dim * a.vdim;
   if ((r = launch_k(linear_carry_kernel<true>, dim3((per + 255) / 256, a.n_seg), dim3(256), 0, st, a)) != cudaSuccess) return r;
@@ -855,7 +869,7 @@ cudaError_t launch_chunked(const LinearAttnArgs& a, cudaStream_t st) {
 bool linear_attention_chunked(const LinearAttnArgs& a) {
   const bool gated = a.gate.a2 != nullptr;
   return a.q_bf && a.k_bf && a.v_bf && a.n_rows >= LC && a.dim <= 128 && a.ws && linear_ws_floats(a.n_rows, a.n_seg, a.heads, a.dim, a.vdim) <= a.ws_floats &&
-         (gated ? a.gate.cum && a.gate.low_bf && a.gate.rank <= 512 : a.vdim <= 128 && a.q_scale == 1.f);
+         (gated ? a.gate.cum && a.gate.low_bf && a.gate.rank <= 160 : a.vdim <= 128 && a.q_scale == 1.f);
 }
 
 bool linear_attention_norm_fits(const LinearAttnArgs& a) { return linear_attention_chunked(a) && a.vdim <= 128; }

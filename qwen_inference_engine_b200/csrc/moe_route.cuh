@@ -77,26 +77,33 @@ __device__ __forceinline__ void route_sigmoid_row(const float* z, float* scratch
 }
 
 // the rider of a norm kernel (RouteRider): the CTA of row r holds the normed row h [W] in shared memory (complete) and works out the
-// router's logits, a warp per expert, lanes striding the width (16-byte weight loads when the rows allow it); warp 0 then chooses.
+// router's logits, a warp per two experts, lanes striding the width (four elements at a time when the rows allow it); warp 0 then chooses.  h is
+// 16-byte aligned.
 // zl: experts + route_scratch_floats() floats of shared memory
 __device__ __forceinline__ void route_rider_row(const RouteRider& rt, int r, const float* h, int W, float* zl) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const bool vec = W % 8 == 0 && (reinterpret_cast<uintptr_t>(rt.w_router) & 15) == 0;
-  for (int e = warp; e < rt.experts; e += nw) {
-    const bf16* wr = rt.w_router + (size_t)e * W;
-    float acc = 0.f;
+  const bool vec = W % 4 == 0 && (reinterpret_cast<uintptr_t>(rt.w_router) & 7) == 0;
+  for (int e = warp; e < rt.experts; e += 2 * nw) {  // two experts at a time share the reads of the row
+    const int e2 = e + nw;
+    const bool two = e2 < rt.experts;
+    const bf16 *wa = rt.w_router + (size_t)e * W, *wb = rt.w_router + (size_t)(two ? e2 : e) * W;
+    float acc = 0.f, acc2 = 0.f;
     if (vec) {
-      for (int i = lane * 8; i < W; i += 256) {
-        const uint4 p = *reinterpret_cast<const uint4*>(wr + i);
-        const float* x = h + i;
-        acc = fmaf(x[0], lo2f(p.x), acc), acc = fmaf(x[1], hi2f(p.x), acc), acc = fmaf(x[2], lo2f(p.y), acc), acc = fmaf(x[3], hi2f(p.y), acc);
-        acc = fmaf(x[4], lo2f(p.z), acc), acc = fmaf(x[5], hi2f(p.z), acc), acc = fmaf(x[6], lo2f(p.w), acc), acc = fmaf(x[7], hi2f(p.w), acc);
+#pragma unroll 8
+      for (int i = lane * 4; i < W; i += 128) {
+        const uint2 p = *reinterpret_cast<const uint2*>(wa + i), q = *reinterpret_cast<const uint2*>(wb + i);
+        const float4 x = *reinterpret_cast<const float4*>(h + i);
+        acc = fmaf(x.x, lo2f(p.x), acc), acc = fmaf(x.y, hi2f(p.x), acc), acc = fmaf(x.z, lo2f(p.y), acc), acc = fmaf(x.w, hi2f(p.y), acc);
+        acc2 = fmaf(x.x, lo2f(q.x), acc2), acc2 = fmaf(x.y, hi2f(q.x), acc2), acc2 = fmaf(x.z, lo2f(q.y), acc2), acc2 = fmaf(x.w, hi2f(q.y), acc2);
       }
     } else {
-      for (int i = lane; i < W; i += 32) acc = fmaf(h[i], bf2f(wr[i]), acc);
+      for (int i = lane; i < W; i += 32) acc = fmaf(h[i], bf2f(wa[i]), acc), acc2 = fmaf(h[i], bf2f(wb[i]), acc2);
     }
-    acc = warp_sum(acc);
-    if (lane == 0) zl[e] = acc;
+    acc = warp_sum(acc), acc2 = warp_sum(acc2);
+    if (lane == 0) {
+      zl[e] = acc;
+      if (two) zl[e2] = acc2;
+    }
   }
   __syncthreads();
   if (warp == 0)
