@@ -6,6 +6,8 @@
 // rows interleaved in runs of 16 with the 64 up rows of the same columns, so that a thread holds silu's argument and
 // its factor side by side and writes silu(gate) * up as bf16 -- the [gate | up] rows never go to memory.
 // k ascends per output whatever the tile, so a row's result does not depend on the rows around it.
+#include <stdlib.h>
+
 #include <algorithm>
 
 #include "launch.h"
@@ -162,9 +164,16 @@ bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g) {
          (reinterpret_cast<uintptr_t>(g.W) & 15) == 0 && g.N > 0 && (!g.gated || g.N % 2 == 0);
 }
 
-cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st) {
+cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st, int num_sms, int* n_launches) {
+  if (n_launches) *n_launches = 0;
   if (g.rows <= 0 || g.groups <= 0) return cudaSuccess;
   if (!grouped_gemm_bf16_fits(g) || !g.grp_off || (g.gated ? !g.out_bf : !(g.out || g.out_bf))) return cudaErrorInvalidValue;
+  static const bool tc_on = [] { const char* v = getenv("QIE_GROUPED_TC"); return !(v && v[0] == '0'); }();  // 0: the kernel above (A/B)
+  if (n_launches) *n_launches = 1;
+  if (tc_on && grouped_gemm_tc_fits(g)) {
+    if (n_launches) *n_launches = g.row_idx ? 2 : 1;
+    return launch_grouped_gemm_tc(g, num_sms, st);
+  }
   const size_t smem = (size_t)2 * STAGES * BM * BKP * sizeof(bf16);  // 60 KB
   static PerDeviceOnce set;
   if (set.need()) {

@@ -87,9 +87,9 @@ struct GxModel : RowFamily {
   float *top_w = nullptr, *perm_w = nullptr, *he = nullptr, *hg = nullptr, *ye = nullptr;
   int *top_idx = nullptr, *grp_off = nullptr, *perm_row = nullptr, *slot_of = nullptr;
   TcProjector tc;
-  // bf16 rows between the producers and consumers of tensor-core GEMMs: hb normed input, mb mixer output, yb projected mixer output, hgb
-  // gated hidden rows of the experts, yeb their outputs
-  bf16 *hb = nullptr, *mb = nullptr, *yb = nullptr, *hgb = nullptr, *yeb = nullptr;
+  // bf16 rows between the producers and consumers of tensor-core GEMMs: hb normed input, mb mixer output, yb projected mixer output, hgr
+  // normed rows in the experts' order, hgb gated hidden rows of the experts, yeb their outputs
+  bf16 *hb = nullptr, *mb = nullptr, *yb = nullptr, *hgr = nullptr, *hgb = nullptr, *yeb = nullptr;
   float* attn_ws = nullptr;
   size_t attn_ws_floats = 0;
   float* scan_ws = nullptr;  // chunk states of the linear attention

@@ -289,6 +289,7 @@ std::string finish_setup(qie_engine* e, const std::vector<TensorSpec>& t, const 
     CUS(bbuf(&m->hb, R * W));
     CUS(bbuf(&m->mb, R * w1));
     CUS(bbuf(&m->yb, R * W));
+    CUS(bbuf(&m->hgr, max_experts ? R * w_top * W : 1));
     CUS(bbuf(&m->hgb, max_experts ? R * w_he / 2 : 1));
     CUS(bbuf(&m->yeb, max_experts ? R * w_top * W : 1));
   }
@@ -354,7 +355,7 @@ std::string gubanex_create_synthetic(qie_engine* e, const std::string& cfg_json,
 
 void GxModel::release() {
   void* dev[] = {blob, kv_pool, state, x, hn, p0, p1, p3, y, xo, top_w, perm_w, he, hg, ye, top_idx, perm_row, slot_of, grp_off, attn_ws, scan_ws, decay_ws,
-                 hb, mb, yb, hgb, yeb};
+                 hb, mb, yb, hgr, hgb, yeb};
   tc.release();
   release_row_buffers();
   for (void* p : dev)
@@ -491,7 +492,7 @@ cudaError_t GxModel::forward(qie_engine* e, int n, int n_seg, int n_out, int max
     bool tc_ex = false;
     if (!m->f32 && n * top > 16 * 16) {  // more rows than the GEMV serves
       eg.A = m->hb, eg.lda = W, eg.row_idx = m->perm_row, eg.grp_off = m->grp_off, eg.W = L.w_egu, eg.w_batch = (long)2 * ff * W;
-      eg.N = 2 * ff, eg.K = W, eg.groups = E, eg.rows = n * top, eg.gated = 1, eg.out_bf = m->hgb, eg.ldo = ff, eg.row_w = m->perm_w;
+      eg.N = 2 * ff, eg.K = W, eg.groups = E, eg.rows = n * top, eg.gated = 1, eg.out_bf = m->hgb, eg.ldo = ff, eg.row_w = m->perm_w, eg.a_rows = m->hgr;
       ed.A = m->hgb, ed.lda = ff, ed.grp_off = m->grp_off, ed.W = L.w_edown, ed.w_batch = (long)W * ff;
       ed.N = W, ed.K = ff, ed.groups = E, ed.rows = n * top, ed.out_bf = m->yeb, ed.ldo = W;
       tc_ex = grouped_gemm_bf16_fits(eg) && grouped_gemm_bf16_fits(ed);
@@ -506,8 +507,10 @@ cudaError_t GxModel::forward(qie_engine* e, int n, int n_seg, int n_out, int max
     }
     FAM_TRY(KK_MOE_ROUTE, launch_moe_group(m->top_idx, n * top, top, E, m->grp_off, m->perm_row, m->slot_of, st, m->top_w, m->perm_w));
     if (tc_ex) {
-      FAM_TRY(KK_MOE_EXPERTS, launch_grouped_gemm_bf16(eg, st));
-      FAM_TRY(KK_MOE_EXPERTS, launch_grouped_gemm_bf16(ed, st));
+      int nl = 0;
+      FAM_TRY(KK_MOE_EXPERTS, launch_grouped_gemm_bf16(eg, st, e->num_sms, &nl));
+      e->launches += nl > 0 ? nl - 1 : 0;
+      FAM_TRY(KK_MOE_EXPERTS, launch_grouped_gemm_bf16(ed, st, e->num_sms));
     } else {
       GemmF32 g;  // [gate | up] of every assignment, rows grouped by expert and gathered from hn
       g.A = m->hn, g.lda = W, g.W = L.w_egu, g.ldw = W, g.w_batch = (long)2 * ff * W, g.C = m->he, g.ldc = 2 * ff;

@@ -170,7 +170,7 @@ cudaError_t launch_moe_group(const int* top_idx, int n_assign, int top, int expe
 cudaError_t launch_moe_combine(const float* ye, const int* slot_of, const float* top_w, int top, const float* ys, const float* z, int ldz,
                                int gate_col, float* y, int width, int n, cudaStream_t st);
 
-// Expert GEMMs on tensor cores over bf16 rows (gemm_grouped.cu): C[row, :] = A[src(row), :] W_z^T for the rows
+// Expert GEMMs on tensor cores over bf16 rows (gemm_grouped_tc.cu on tcgen05, gemm_grouped.cu for the shapes it does not take): C[row, :] = A[src(row), :] W_z^T for the rows
 // grp_off[z] .. grp_off[z + 1] - 1 of expert z, src(row) = row_idx ? row_idx[row] : row; W_z = W + z * w_batch, [N, K] row-major.
 // gated: W_z = [gate rows | up rows] (N = 2 ff) and out_bf[row, c] = bf16(silu(gate_c) * up_c), c < ff; else out[row, n] fp32 or out_bf.
 // row_w (per row of the groups): the input row is scaled by it, which both linear maps let through: gate and up (or the result) times row_w.
@@ -183,6 +183,7 @@ struct GroupedGemmBf16 {
   long w_batch = 0;
   int N = 0, K = 0, groups = 0;
   const float* row_w = nullptr;
+  bf16* a_rows = nullptr;  // [rows, K]: room for the gathered rows of the tcgen05 form
   int rows = 0;  // rows over all groups (bounds the grid)
   int gated = 0;
   float* out = nullptr;
@@ -190,7 +191,9 @@ struct GroupedGemmBf16 {
   int ldo = 0;
 };
 bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g);  // K a multiple of 32, 16-byte aligned rows
-cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st);
+cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st, int num_sms = 148, int* n_launches = nullptr);
+bool grouped_gemm_tc_fits(const GroupedGemmBf16& g);
+cudaError_t launch_grouped_gemm_tc(const GroupedGemmBf16& g, int num_sms, cudaStream_t st);
 
 // ---------------------------------------------------------------- the model (nogatar_model.cu)
 typedef RotaryCfg NgRot;
