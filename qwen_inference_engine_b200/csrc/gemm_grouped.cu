@@ -159,7 +159,14 @@ __global__ void __launch_bounds__(256) grouped_gemm_bf16_kernel(const GroupedGem
 
 }  // namespace
 
+// QIE_GROUPED_TC=0: the kernel above for every shape (A/B)
+static bool tc_takes(const GroupedGemmBf16& g) {
+  static const bool on = [] { const char* v = getenv("QIE_GROUPED_TC"); return !(v && v[0] == '0'); }();
+  return on && grouped_gemm_tc_fits(g);
+}
+
 bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g) {
+  if (tc_takes(g)) return true;
   return g.K >= BK && g.K % BK == 0 && g.lda % 8 == 0 && g.w_batch % 8 == 0 && (reinterpret_cast<uintptr_t>(g.A) & 15) == 0 &&
          (reinterpret_cast<uintptr_t>(g.W) & 15) == 0 && g.N > 0 && (!g.gated || g.N % 2 == 0);
 }
@@ -168,9 +175,8 @@ cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st, 
   if (n_launches) *n_launches = 0;
   if (g.rows <= 0 || g.groups <= 0) return cudaSuccess;
   if (!grouped_gemm_bf16_fits(g) || !g.grp_off || (g.gated ? !g.out_bf : !(g.out || g.out_bf))) return cudaErrorInvalidValue;
-  static const bool tc_on = [] { const char* v = getenv("QIE_GROUPED_TC"); return !(v && v[0] == '0'); }();  // 0: the kernel above (A/B)
   if (n_launches) *n_launches = 1;
-  if (tc_on && grouped_gemm_tc_fits(g)) {
+  if (tc_takes(g)) {
     if (n_launches) *n_launches = g.row_idx ? 2 : 1;
     return launch_grouped_gemm_tc(g, num_sms, st);
   }

@@ -190,7 +190,7 @@ struct GroupedGemmBf16 {
   bf16* out_bf = nullptr;
   int ldo = 0;
 };
-bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g);  // K a multiple of 32, 16-byte aligned rows
+bool grouped_gemm_bf16_fits(const GroupedGemmBf16& g);  // the tcgen05 form, or K a multiple of 32 and 16-byte aligned rows
 cudaError_t launch_grouped_gemm_bf16(const GroupedGemmBf16& g, cudaStream_t st, int num_sms = 148, int* n_launches = nullptr);
 bool grouped_gemm_tc_fits(const GroupedGemmBf16& g);
 cudaError_t launch_grouped_gemm_tc(const GroupedGemmBf16& g, int num_sms, cudaStream_t st);

@@ -417,6 +417,30 @@ def test_bf16_chosen_experts(tmp_path):
         assert np.median(err) < 1e-2 and np.quantile(err, 0.8) < 2e-2, (np.median(err), err.max())
 
 
+@pytest.mark.parametrize("width,ff,experts,top,n", [
+    (128, 128, 3, 3, 150),   # every expert has every row: a whole tile of rows and a short one
+    (160, 136, 2, 2, 200),   # k no multiple of a stage, a tile of output columns that ends early
+    (192, 64, 40, 6, 130),   # many experts with few rows each, one stage-wide hidden rows (the down product on the other kernel)
+    (256, 320, 5, 1, 700),   # more row tiles than one per expert, two and more tiles of output columns
+    (384, 192, 260, 2, 300), # most experts have no row, more of them than a scan's step takes
+], ids=["all", "ragged", "many", "tall", "empty_groups"])
+def test_bf16_expert_tiles(tmp_path, width, ff, experts, top, n):
+    # the grouped expert GEMMs on tcgen05 against the restatement and against portions that take the GEMV; a router's close call may
+    # come out otherwise at bf16 precision, so where not every expert is chosen most rows are asked for, not all
+    cfg = U.make_config([U.gla(heads=1, dim=8, vdim=8, mlp=U.moe(experts=experts, top=top, ff=ff))], width=width, vocab=29, softcap=30.0)
+    w = U.random_weights(cfg, seed=51)
+    U.set_values(w, "l0.mlp.router", 0.3 * w["l0.mlp.router"][1])  # scores well below 1, also the best of many
+    toks = _tokens(cfg, n, 6)
+    right = _oracle_logits(cfg, w, toks)
+    assert np.median(_row_err(_oracle_logits(cfg, w, toks[:40], mlp={"fault_output_weight": True}), right[:40])) > 4e-2
+    eng = _engine(tmp_path, cfg, w, dtype="bfloat16", page_size=16, max_pages=100, rows=768)
+    whole, cut = _whole(eng, toks), _cuts(eng, toks, [n - 33, 1, 32])
+    eng.close()
+    for got in (whole, cut):
+        err = _row_err(got, right)
+        assert np.median(err) < 1e-2 and np.quantile(err, 1.0 if top == experts else 0.8) < 2e-2, (np.median(err), err.max())
+
+
 def test_bf16_other_sizes(tmp_path):
     # bf16 serving precision away from the tensor-core shapes: a width that is no multiple of 64, head sizes beyond the tensor-core
     # kernels' tiles, portions against the whole
