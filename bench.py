@@ -558,10 +558,10 @@ def gubanex_config(z, vocab=32000):
     W = z["width"]
     moe = {"kind": "moe", "expert": {"ff": z["ff"] + z["sff"] // z["top"]}, "router": {"experts": z["experts"], "top": z["top"]}}
     att = {"dim": 64, "heads": W // 64, "kv_heads": 4, "mask": {"size": z["window"]}, "scale": 0.125, "vdim": 64,
-           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 2048}}}
-    lin = {"dim": 64, "heads": W // 128, "rank": 16, "tau": 16.0, "vdim": 128}
+           "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 2048}}}
+    lin = {"dim": 64, "heads": W // 128, "rank": 16, "tau": 8.0, "vdim": 128}
     layers = [{"type": "attention", "mixer": att, "mlp": moe}, {"type": "gla", "mixer": lin, "mlp": moe}]
-    return {"architecture": "Gubanex", "embedding": {"scale": W ** 0.5}, "layers": layers, "logit_scale": 0.25, "logit_softcap": 30.0,
+    return {"architecture": "Gubanex", "embedding": {"scale": W ** 0.5}, "layers": layers, "logit_scale": 0.5, "logit_softcap": 50.0,
             "loop": {"start": 0, "stop": 2, "times": 2}, "norm": {"eps": 1e-6}, "vocab": vocab, "width": W}
 
 

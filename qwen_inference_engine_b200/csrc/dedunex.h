@@ -42,7 +42,7 @@ namespace qie {
 //   dump    dump[r] = x[src]                  the stream after a layer, for the parity hook
 //   step    x[src] += step                    a vector of the model (before a pass of a loop)
 //   again   x[src] += embed[ids[r]] * embed_scale   the embedding once more (before a pass of a loop; the source is then x itself)
-//   read    h[r] = gnorm(x[src]) (w_off + w_in)   fp32 rows and / or dense bf16 rows (w_off 1: a weight stored around zero)
+//   read    h[r] = gnorm(x[src]) (w_off + w_in)   fp32 rows and / or dense bf16 rows (w_off 1: a zero-centred weight)
 //   route   the router's logits and choice of the row just read (RouteRider)
 // x[src] is written back when it changed.
 struct GroupNormStep {

@@ -52,7 +52,7 @@ struct TensorSpec {
   std::string name;
   size_t rows = 0, cols = 0;  // cols 0 = vector of `rows`
   size_t off = 0;             // element offset in the blob
-  int kind = 0;               // synthetic fill: 0 matrix (uniform, variance 1/cols), 1 norm weight (about 1), 2 small vector; 3: zeros that no file holds; 4: norm weight stored around zero
+  int kind = 0;               // synthetic fill: 0 matrix (uniform, variance 1/cols), 1 norm weight (about 1), 2 small vector; 3: zeros that no file holds; 4: zero-centred norm weight
   size_t elems() const { return rows * (cols ? cols : 1); }
 };
 // appends tensors to a layout; pad() starts the next group on a 256-byte boundary (tensors that one GEMM reads as a

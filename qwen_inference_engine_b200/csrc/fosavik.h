@@ -142,7 +142,7 @@ bool kv_store_heads_fits(const KvStoreArgs& a);
 // pooled rows of every block whose last position is among the n rows (their keys and values are in the cache already)
 cudaError_t launch_kv_pool_rows(const KvRowCache& c, const int* pos, const int* slot, const int* block_table, int max_pages, int n, cudaStream_t st);
 // out[r, h, :] over the keys j of row r's sequence with j <= pos and (window <= 0 or pos - j < window or j < keep_first).
-// chunk > 0 (instead of a window): the positions fall into chunks of `chunk`, counted from position 0 of the sequence, and a row sees
+// chunk > 0 (instead of a window): the positions fall into chunks of `chunk` (the first one begins with the sequence), and a row sees
 // the keys of its own chunk up to itself.
 // `maps` score maps per head (queries [h][map][dim], keys [g][map][dim]) share the values [g][vdim]; head h reads kv
 // head h / (heads / kv_heads).  unit_sink adds 1 to every softmax denominator (as if one more key with a zero score and nothing to contribute took part).

@@ -1,4 +1,4 @@
-// gubanex.h -- the Gubanex model family: a decoder with one fp32 residual stream and RMS norms whose weights are stored around zero,
+// gubanex.h -- the Gubanex model family: a decoder with one fp32 residual stream and RMS norms with zero-centred weights,
 // x += mixer(norm1(x)), x += ff(norm2(x)).  A layer's mixer is one of
 //  * chunked attention: grouped queries, partial rotary positions in the "rotate half" pairing with frequencies scaled by their
 //    wavelength, queries and keys normed without a weight after the rotation, a softmax over the keys of the row's own chunk of positions;
@@ -9,7 +9,7 @@
 // pass); the embedding is added to the stream again before every pass but the first.  Logits are scaled and soft-capped.
 //
 // New mechanisms are options of launchers that other families use, or stand beside the ones they resemble: chunks and unit norms of the
-// paged attention (attn_gqa.cu, attn_gqa_tc.cu), the gated decay of the linear attention (linear_attn.cu), weights around zero, the repeated
+// paged attention (attn_gqa.cu, attn_gqa_tc.cu), the gated decay of the linear attention (linear_attn.cu), zero-centred weights, the repeated
 // embedding and the router's rider of the norm step (rmsnorm_f32.cu), scaled expert inputs (moe.cu, gemm_grouped.cu,
 // activations.cu), frequencies scaled by wavelength (family.h).  gubanex_model.cu holds the configuration reader, the weight loader and
 // the launch order.  The family shares the engine's sequences, page allocator, block tables, row metadata, sampler, scheduler and

@@ -26,7 +26,7 @@ def unit_rms(x, eps):
 
 
 def zero_centred_norm(x, weight, eps, fault_plain_weight=False):
-    """an RMS norm whose weight is stored around zero: the factor is 1 + weight"""
+    """an RMS norm with a zero-centred weight: the factor is 1 + weight"""
     return unit_rms(x, eps) * (weight if fault_plain_weight else 1.0 + weight)
 
 

@@ -75,7 +75,7 @@ def random_weights(cfg, seed=0, gain=1.0, rank=3):
         elif name.endswith("mix.norm"):
             a = 1.0 + 0.2 * rng.standard_normal(shape)
         else:
-            a = 0.2 * rng.standard_normal(shape)  # stored around zero
+            a = 0.2 * rng.standard_normal(shape)  # zero-centred
         out[name] = bf16_round(np.asarray(a, np.float32))
     return out
 

@@ -238,7 +238,7 @@ def test_far_key_among_hundreds(tmp_path):
 def test_what_tame_weights_hide(tmp_path):
     # each of these would go unnoticed with tame weights: pairing and scaling of the rotation, the norm behind it, the order of the head
     # groups, tau, a decay per channel, what the decay acts on, the query scale, where the router's weight enters, a state of its own
-    # per pass, the embedding before a pass, weights around zero, the logits' scale and cap
+    # per pass, the embedding before a pass, zero-centred weights, the logits' scale and cap
     layers = [U.attention(heads=4, kv_heads=2, dim=8, vdim=6, size=30, scale=1.0, rot_dims=8, base=50.0, mlp=U.moe(experts=4, top=2)),
               U.gla(heads=2, dim=6, vdim=5, tau=3.0, mlp=U.moe(experts=5, top=1))]
     cfg = U.make_config(layers, width=16, vocab=23, loop=(0, 2, 2))
